@@ -14,12 +14,17 @@ LIB_PATH = os.path.join(_HERE, "libdoppler_b200.so")
 # status codes / dtypes of include/doppler_b200.h
 OK, ERR_INVALID, ERR_CUDA, ERR_OOM, ERR_UNSUPPORTED, ERR_TIMEOUT, ERR_STATE, ERR_COMM = range(8)
 STATUS_NAMES = ["ok", "invalid", "cuda", "oom", "unsupported", "timeout", "state", "comm"]
-F32, F16, Q4K, I32 = 0, 1, 2, 3
-DTYPE_CODES = {"f32": F32, "f16": F16, "q4k": Q4K, "i32": I32}
+F32, F16, Q4K, I32, BF16 = 0, 1, 2, 3, 4
+DTYPE_CODES = {"f32": F32, "f16": F16, "q4k": Q4K, "i32": I32, "bf16": BF16}
 DTYPE_NAMES = {v: k for k, v in DTYPE_CODES.items()}
-DTYPE_BYTES = {"f32": 4, "f16": 2, "i32": 4}
+DTYPE_BYTES = {"f32": 4, "f16": 2, "i32": 4, "bf16": 2}
 
 W_Q, W_K, W_V, W_O, W_GATE, W_UP, W_DOWN, W_IN_NORM, W_POST_NORM, W_Q_NORM, W_K_NORM = range(11)
+
+# decoders described layer by layer: mixers and tensor ids
+MIXER_ATTENTION, MIXER_MAMBA2 = 0, 1
+(T_EMBED, T_FINAL_NORM, T_NORM1, T_NORM2, T_CONV1, T_CONV2, T_HC1_IN, T_HC1_OUT, T_HC1_MIX, T_HC2_IN, T_HC2_OUT, T_HC2_MIX, T_Q, T_K, T_V, T_GATE_HEADS,
+ T_O, T_SSM_IN, T_SSM_CONV, T_SSM_CONV_B, T_SSM_DT_BIAS, T_SSM_A_LOG, T_SSM_D, T_SSM_NORM, T_FF_GATE, T_FF_UP, T_FF_DOWN) = range(27)
 
 
 class DopplerError(RuntimeError):
@@ -76,6 +81,17 @@ class ModelCfg(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("n_layers", "hidden", "n_heads", "n_kv_heads", "head_dim", "inter", "vocab",
                                         "max_seq")] + [("eps", C.c_float), ("rope_theta", C.c_float),
                                                        ("max_batch", C.c_int), ("tp_rank", C.c_int), ("tp_size", C.c_int)]
+
+
+class LayerCfg(C.Structure):
+    _fields_ = ([(n, C.c_int) for n in ("mixer", "heads", "vdim", "kv_heads", "dim", "chunk", "unit_rms_qk", "head_gate")] + [("scale", C.c_float)]
+                + [(n, C.c_int) for n in ("state", "groups", "conv_taps", "norm_groups", "ff")]
+                + [(n, C.c_float) for n in ("ff_limit", "ff_slope", "ff_shift")])
+
+
+class StackCfg(C.Structure):
+    _fields_ = ([(n, C.c_int) for n in ("n_layers", "width", "vocab", "max_seq", "max_batch", "streams", "norm_groups", "input_taps")]
+                + [("eps", C.c_float), ("embed_scale", C.c_float), ("act_dtype", C.c_int), ("max_rows", C.c_int)])
 
 
 _vp, _sz, _i, _f, _u32, _u64, _dbl = C.c_void_p, C.c_size_t, C.c_int, C.c_float, C.c_uint32, C.c_uint64, C.c_double
@@ -157,6 +173,11 @@ SIGNATURES = {
     "dp_model_reset": (_i, [_vp]),
     "dp_model_prefill": (_i, [_vp, _i, _vp, _i, C.POINTER(C.c_int32)]),
     "dp_model_decode": (_i, [_vp, _i, _vp, _i, _vp]),
+    "dp_model_extend": (_i, [_vp, _i, _vp, _i, _vp, _i, _vp]),
+    "dp_model_release": (_i, [_vp, _i]),
+    "dp_model_create_stack": (_i, [_vp, C.POINTER(StackCfg), C.POINTER(LayerCfg), C.POINTER(_vp)]),
+    "dp_model_load_tensor": (_i, [_vp, _i, _i, _vp, _i, _i]),
+    "dp_model_state_bytes": (_sz, [_vp]),
     "dp_model_last_decode_ms": (_dbl, [_vp]),
     "dp_model_read_logits": (_i, [_vp, _vp, _i]),
     "dp_model_read_hidden": (_i, [_vp, _vp, _i]),

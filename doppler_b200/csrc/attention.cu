@@ -12,6 +12,7 @@
 // for D=128); each 8-lane group keeps its own running max / sum / output and the
 // groups are merged at the end (warp shuffles, then shared memory).  Split
 // partials (m, l, o) go to a scratch buffer and a second kernel merges them.
+#include "attn_out.cuh"
 #include "common.h"
 #include "pdl.cuh"
 
@@ -20,27 +21,6 @@
 
 #define ATT_THREADS 256
 #define ATT_GROUPS (ATT_THREADS / 8)
-
-struct AttnRange { int lo, hi; };
-
-// keys visible to query row qi: [lo, hi) in cache positions
-__device__ __forceinline__ AttnRange attn_range(int kv_len, int causal, int start_pos, int qi, int sliding_window,
-                                                int kv_start) {
-  AttnRange r;
-  r.lo = 0;
-  r.hi = kv_len;
-  const int abs_q = start_pos + qi;
-  if (causal) {
-    int lim = abs_q - kv_start + 1;  // abs_key <= abs_q
-    if (lim < r.hi) r.hi = lim;
-  }
-  if (sliding_window > 0 && abs_q >= sliding_window) {
-    int first = abs_q - sliding_window + 1 - kv_start;  // abs_key >= abs_q - window + 1
-    if (first > r.lo) r.lo = first;
-  }
-  if (r.hi < r.lo) r.hi = r.lo;
-  return r;
-}
 
 // LPK lanes share a key (each owns DPL = D/LPK dims).  More lanes per key = fewer registers per
 // thread (q and the output accumulators shrink), which is what lets two CTAs share an SM.
@@ -61,7 +41,7 @@ __global__ void __launch_bounds__(ATT_THREADS, LPK == 16 ? 2 : 1) attn_split_ker
   const int h0 = kvh * G + ht * GT;  // first query head of this CTA
 
   int kv_len = p.kv_lens ? min(max(p.kv_lens[b], 0), p.kv_len) : p.kv_len;  // the host checked the cache for p.kv_len keys
-  const AttnRange r = attn_range(kv_len, p.causal, p.start_pos, qi, p.sliding_window, p.kv_start);
+  const AttnRange r = attn_range(p, kv_len, qi);
   const int n_keys = r.hi - r.lo;
   const int per_split = (n_keys + splits - 1) / splits;
   const int k_begin = r.lo + split * per_split;
@@ -192,7 +172,7 @@ __global__ void __launch_bounds__(ATT_THREADS, LPK == 16 ? 2 : 1) attn_split_ker
     }
     const int h = h0 + g;
     if (splits == 1) {
-      p.out[((size_t)z * p.num_heads + h) * D + d] = ll > 0.0f ? acc / ll : 0.0f;
+      attn_store(p, z, h, D, d, ll > 0.0f ? acc / ll : 0.0f);
     } else {
       float *pp = part + (((size_t)z * p.num_heads + h) * splits + split) * (D + 2);
       pp[d] = acc;
@@ -201,18 +181,19 @@ __global__ void __launch_bounds__(ATT_THREADS, LPK == 16 ? 2 : 1) attn_split_ker
   }
 }
 
-// Any head_dim <= 512 and any GQA ratio: one CTA per (split, query head, row),
-// lanes over dims.  Used for shapes outside the fast kernel.
+// Any query/key size and any value size up to 512, any GQA ratio, f16 or f32 caches: one CTA per (split, query
+// head, row), lanes over dims.  Used for shapes outside the fast kernels.
+template <typename KT>
 __global__ void __launch_bounds__(128) attn_split_generic_kernel(dpk_attn_params p, float *__restrict__ part, int splits) {
   pdl_launch();
   pdl_wait();
-  const int D = p.head_dim;
+  const int D = p.head_dim, V = p.v_dim ? p.v_dim : D;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int split = blockIdx.x, h = blockIdx.y, z = blockIdx.z;
   const int b = z / p.seq_len, qi = z % p.seq_len;
   const int kvh = h / (p.num_heads / p.num_kv_heads);
   int kv_len = p.kv_lens ? min(max(p.kv_lens[b], 0), p.kv_len) : p.kv_len;  // the host checked the cache for p.kv_len keys
-  const AttnRange r = attn_range(kv_len, p.causal, p.start_pos, qi, p.sliding_window, p.kv_start);
+  const AttnRange r = attn_range(p, kv_len, qi);
   const int n_keys = r.hi - r.lo;
   const int per_split = (n_keys + splits - 1) / splits;
   const int k_begin = r.lo + split * per_split;
@@ -225,13 +206,13 @@ __global__ void __launch_bounds__(128) attn_split_generic_kernel(dpk_attn_params
 #pragma unroll
   for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; q[i] = d < D ? qp[d] * p.scale : 0.0f; o[i] = 0.0f; }
   float m = -FLT_MAX, l = 0.0f;
-  const size_t row_stride = (size_t)p.num_kv_heads * D;
-  const __half *kb = p.k + (size_t)b * p.kv_batch_stride + (size_t)kvh * D;
-  const __half *vb = p.v + (size_t)b * p.kv_batch_stride + (size_t)kvh * D;
+  const size_t k_stride = (size_t)p.num_kv_heads * D, v_stride = (size_t)p.num_kv_heads * V;
+  const KT *kb = reinterpret_cast<const KT *>(p.k) + (size_t)b * p.kv_batch_stride + (size_t)kvh * D;
+  const KT *vb = reinterpret_cast<const KT *>(p.v) + (size_t)b * (p.v_batch_stride ? p.v_batch_stride : p.kv_batch_stride) + (size_t)kvh * V;
   for (int key = k_begin + warp; key < k_end; key += 4) {
     float a = 0.0f;
 #pragma unroll
-    for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; if (d < D) a = fmaf(q[i], __half2float(kb[(size_t)key * row_stride + d]), a); }
+    for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; if (d < D) a = fmaf(q[i], (float)kb[(size_t)key * k_stride + d], a); }
 #pragma unroll
     for (int s = 16; s > 0; s >>= 1) a += __shfl_xor_sync(0xffffffffu, a, s);
     if (p.softcap > 0.0f) a = tanhf(a / p.softcap) * p.softcap;
@@ -246,15 +227,15 @@ __global__ void __launch_bounds__(128) attn_split_generic_kernel(dpk_attn_params
     const float pr = exp2f(a - m);
     l += pr;
 #pragma unroll
-    for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; if (d < D) o[i] = fmaf(pr, __half2float(vb[(size_t)key * row_stride + d]), o[i]); }
+    for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; if (d < V) o[i] = fmaf(pr, (float)vb[(size_t)key * v_stride + d], o[i]); }
   }
   __shared__ float sm_o[4][512];
   __shared__ float sm_m[4], sm_l[4];
 #pragma unroll
-  for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; if (d < D) sm_o[warp][d] = o[i]; }
+  for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; if (d < V) sm_o[warp][d] = o[i]; }
   if (lane == 0) { sm_m[warp] = m; sm_l[warp] = l; }
   __syncthreads();
-  for (int d = tid; d < D; d += 128) {
+  for (int d = tid; d < V; d += 128) {
     float mm = -FLT_MAX;
     for (int w = 0; w < 4; w++) mm = fmaxf(mm, sm_m[w]);
     float ll = 0.0f, acc = 0.0f;
@@ -264,38 +245,42 @@ __global__ void __launch_bounds__(128) attn_split_generic_kernel(dpk_attn_params
       acc = fmaf(sm_o[w][d], c, acc);
     }
     if (splits == 1) {
-      p.out[((size_t)z * p.num_heads + h) * D + d] = ll > 0.0f ? acc / ll : 0.0f;
+      attn_store(p, z, h, V, d, ll > 0.0f ? acc / ll : 0.0f);
     } else {
-      float *pp = part + (((size_t)z * p.num_heads + h) * splits + split) * (D + 2);
+      float *pp = part + (((size_t)z * p.num_heads + h) * splits + split) * (V + 2);
       pp[d] = acc;
-      if (d == 0) { pp[D] = mm; pp[D + 1] = ll; }
+      if (d == 0) { pp[V] = mm; pp[V + 1] = ll; }
     }
   }
 }
 
 // merge the split partials of one (row, head)
-__global__ void attn_combine_kernel(const float *__restrict__ part, float *__restrict__ out, int D, int splits) {
+__global__ void attn_combine_kernel(dpk_attn_params p, const float *__restrict__ part, int splits) {
   pdl_launch();
   pdl_wait();
   const size_t rh = blockIdx.x;
-  const float *pp = part + rh * splits * (D + 2);
+  const int V = p.v_dim ? p.v_dim : p.head_dim;
+  const float *pp = part + rh * splits * (V + 2);
   float mm = -FLT_MAX;
-  for (int s = 0; s < splits; s++) mm = fmaxf(mm, pp[s * (D + 2) + D]);
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+  for (int s = 0; s < splits; s++) mm = fmaxf(mm, pp[s * (V + 2) + V]);
+  for (int d = threadIdx.x; d < V; d += blockDim.x) {
     float ll = 0.0f, acc = 0.0f;
 #pragma unroll 4
     for (int s = 0; s < splits; s++) {
-      const float ms = pp[s * (D + 2) + D];
+      const float ms = pp[s * (V + 2) + V];
       const float c = (ms == -FLT_MAX) ? 0.0f : exp2f(ms - mm);
-      ll = fmaf(pp[s * (D + 2) + D + 1], c, ll);
-      acc = fmaf(pp[s * (D + 2) + d], c, acc);
+      ll = fmaf(pp[s * (V + 2) + V + 1], c, ll);
+      acc = fmaf(pp[s * (V + 2) + d], c, acc);
     }
-    out[rh * D + d] = ll > 0.0f ? acc / ll : 0.0f;
+    attn_store(p, rh / p.num_heads, (int)(rh % p.num_heads), V, d, ll > 0.0f ? acc / ll : 0.0f);
   }
 }
 
+// caches the f16 kernels of one head size can read
+static bool f16_square(const dpk_attn_params &p) { return !p.kv_f32 && (p.v_dim == 0 || p.v_dim == p.head_dim); }
+
 static bool fast_shape(const dpk_attn_params &p, int *gt) {
-  if (p.head_dim != 128 && p.head_dim != 64) return false;
+  if ((p.head_dim != 128 && p.head_dim != 64) || !f16_square(p)) return false;
   const int G = p.num_heads / p.num_kv_heads;
   if (G == 1 || G == 2 || G == 4) { *gt = G; return true; }
   if (G % 4 == 0) { *gt = 4; return true; }
@@ -312,7 +297,7 @@ dp_status dpk_attention_tc_split(dp_ctx *ctx, const dpk_attn_params &p, float *s
 static bool use_tc(dp_ctx *ctx, const dpk_attn_params &p, int *gt) {
   (void)ctx;
   static const int mode = [] { const char *e = getenv("DP_ATTN_TC"); return e ? atoi(e) : 1; }();
-  return mode && dpk_attention_tc_eligible(p, gt);
+  return mode && f16_square(p) && dpk_attention_tc_eligible(p, gt);
 }
 
 // whether a call with these parameters runs on the tensor-core kernel (the decode schedule asks before it
@@ -322,6 +307,9 @@ bool dpk_attention_uses_tc(dp_ctx *ctx, const dpk_attn_params &p) {
   return use_tc(ctx, p, &gt);
 }
 
+// the most keys one query row sees
+static long row_keys(const dpk_attn_params &p) { return p.chunk > 0 && p.chunk < p.kv_len ? p.chunk : p.kv_len; }
+
 // splits for the tensor-core kernel: fewest whole waves of (two CTAs per SM) x keys per CTA
 static int tc_splits(dp_ctx *ctx, const dpk_attn_params &p, int gt) {
   const int G = p.num_heads / p.num_kv_heads;
@@ -329,7 +317,7 @@ static int tc_splits(dp_ctx *ctx, const dpk_attn_params &p, int gt) {
   const long slots = (long)ctx->sm_count * 2;
   long best = 1, best_cost = -1;
   for (long s = 1; s <= 32; s++) {
-    const long keys = (p.kv_len + s - 1) / s;
+    const long keys = (row_keys(p) + s - 1) / s;
     // at least two rounds of the CTA's four warps per split: finer splits only lengthen the merge that
     // follows (9B-shaped decode at context 1024, cache of 1450 keys: 4 / 6 / 8 / 11 / 16 splits 1.962 / 1.944 / 1.966 /
     // 1.989 / 2.046 ms per step)
@@ -355,14 +343,14 @@ size_t dpk_attention_scratch_bytes(dp_ctx *ctx, const dpk_attn_params &p, int *s
   const long target = (long)ctx->sm_count * 4;
   long splits = (target + base_ctas - 1) / base_ctas;
   const int keys_per_cta_min = fast ? 128 : 32;
-  long max_splits = (p.kv_len + keys_per_cta_min - 1) / keys_per_cta_min;
+  long max_splits = (row_keys(p) + keys_per_cta_min - 1) / keys_per_cta_min;
   if (max_splits < 1) max_splits = 1;
   if (splits > max_splits) splits = max_splits;
   if (splits < 1) splits = 1;
   if (splits > 32) splits = 32;
   *splits_out = (int)splits;
   if (splits == 1) return 0;
-  return (size_t)rows * p.num_heads * splits * (p.head_dim + 2) * sizeof(float);
+  return (size_t)rows * p.num_heads * splits * ((p.v_dim ? p.v_dim : p.head_dim) + 2) * sizeof(float);
 }
 
 template <int DPL, int GT, int LPK>
@@ -393,7 +381,7 @@ static dp_status attention_impl(dp_ctx *ctx, const dpk_attn_params &p, float *sc
   int gt = 1;
   // several causal query rows: one CTA per tile of query positions shares each K / V tile (DP_ATTN_TC=0: off)
   static const int tc_mode = [] { const char *e = getenv("DP_ATTN_TC"); return e ? atoi(e) : 1; }();
-  if (tc_mode && combine && dpk_attention_prefill_eligible(p)) return dpk_attention_prefill(ctx, p);
+  if (tc_mode && combine && f16_square(p) && dpk_attention_prefill_eligible(p)) return dpk_attention_prefill(ctx, p);
   if (use_tc(ctx, p, &gt)) {
     DP_TRY(dpk_attention_tc_split(ctx, p, scratch, splits));
   } else if (fast_shape(p, &gt)) {
@@ -408,12 +396,15 @@ static dp_status attention_impl(dp_ctx *ctx, const dpk_attn_params &p, float *sc
     }
   } else {
     dim3 grid(splits, p.num_heads, p.batch * p.seq_len);
-    DP_LAUNCH(ctx, attn_split_generic_kernel, grid, 128, 0, p, scratch, splits);
+    if (p.head_dim > 512 || p.v_dim > 512) return dp_fail(ctx, DP_ERR_UNSUPPORTED, "attention: head sizes above 512");
+    if (p.kv_f32) DP_LAUNCH(ctx, attn_split_generic_kernel<float>, grid, 128, 0, p, scratch, splits);
+    else DP_LAUNCH(ctx, attn_split_generic_kernel<__half>, grid, 128, 0, p, scratch, splits);
   }
   if (splits > 1 && combine) {
     const unsigned rows = (unsigned)((long)p.batch * p.seq_len * p.num_heads);
-    int threads = p.head_dim < 128 ? ((p.head_dim + 31) / 32) * 32 : 128;
-    DP_LAUNCH(ctx, attn_combine_kernel, rows, threads, 0, scratch, p.out, p.head_dim, splits);
+    const int V = p.v_dim ? p.v_dim : p.head_dim;
+    int threads = V < 128 ? ((V + 31) / 32) * 32 : 128;
+    DP_LAUNCH(ctx, attn_combine_kernel, rows, threads, 0, p, (const float *)scratch, splits);
   }
   return DP_OK;
 }

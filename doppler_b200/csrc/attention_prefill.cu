@@ -69,6 +69,10 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
   const int cta_keys = min(kv_len, p.start_pos + last_q + 1);
   const int warp_keys = min(kv_len, p.start_pos + min(q0 + 15, p.seq_len - 1) + 1);  // beyond this every key is masked for the warp
   const int n_tiles = (cta_keys + APF_KT - 1) / APF_KT;
+  // chunked attention: a row sees no key before its own chunk, a CTA (a warp) none before its first row's chunk
+  const int loA = p.chunk > 0 ? posA / p.chunk * p.chunk : 0, loB = p.chunk > 0 ? posB / p.chunk * p.chunk : 0;
+  const int tile0 = p.chunk > 0 ? (p.start_pos + qtile * QT) / p.chunk * p.chunk / APF_KT : 0;
+  const int warp_lo = p.chunk > 0 ? (p.start_pos + q0) / p.chunk * p.chunk : 0;
 
   const __half *kbase = p.k + (size_t)b * p.kv_batch_stride + (size_t)kvh * APF_D;
   const __half *vbase = p.v + (size_t)b * p.kv_batch_stride + (size_t)kvh * APF_D;
@@ -122,12 +126,12 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
   for (int j = 0; j < 16; j++) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f; }
   float mA = -INFINITY, mB = -INFINITY, lA = 0.0f, lB = 0.0f;  // running max (log2 units) and this lane's share of the running sum
 
-  if (n_tiles > 0) issue_tile(0);
-  for (int tile = 0; tile < n_tiles; tile++) {
+  if (tile0 < n_tiles) issue_tile(tile0);
+  for (int tile = tile0; tile < n_tiles; tile++) {
     if (tile + 1 < n_tiles) { issue_tile(tile + 1); apf_wait<1>(); } else { apf_wait<0>(); }
     __syncthreads();
     const int key0 = tile * APF_KT;
-    if (key0 < warp_keys) {  // (warp-uniform) later tiles are masked for all of this warp's rows
+    if (key0 < warp_keys && key0 + APF_KT > warp_lo) {  // (warp-uniform) other tiles are masked for all of this warp's rows
       const unsigned char *sK = apf_smem + (tile & 1) * APF_STAGE;
       const uint32_t sV = smem0 + (uint32_t)(tile & 1) * APF_STAGE + APF_TILE;
       // ---- S = (scale * Q) K^T for 16 rows x 32 keys ----
@@ -152,7 +156,7 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
         for (int e = 0; e < 4; e++) {
           const int key = key0 + nt * 8 + 2 * t + (e & 1);
           const int pos = e < 2 ? posA : posB;
-          if (key > pos || key >= kv_len) sc[nt][e] = -INFINITY;
+          if (key > pos || key >= kv_len || key < (e < 2 ? loA : loB)) sc[nt][e] = -INFINITY;
         }
         tmA = fmaxf(tmA, fmaxf(sc[nt][0], sc[nt][1]));
         tmB = fmaxf(tmB, fmaxf(sc[nt][2], sc[nt][3]));
@@ -202,16 +206,23 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
   // ---- normalise and store ----
   lA += __shfl_xor_sync(0xffffffffu, lA, 1); lA += __shfl_xor_sync(0xffffffffu, lA, 2);
   lB += __shfl_xor_sync(0xffffffffu, lB, 1); lB += __shfl_xor_sync(0xffffffffu, lB, 2);
-  const float iA = lA > 0.0f ? 1.0f / lA : 0.0f, iB = lB > 0.0f ? 1.0f / lB : 0.0f;
-  if (rowA < p.seq_len) {
-    float *dst = p.out + (((size_t)b * p.seq_len + rowA) * p.num_heads + h) * APF_D + 2 * t;
 #pragma unroll
-    for (int j = 0; j < 16; j++) *reinterpret_cast<float2 *>(dst + 8 * j) = make_float2(o[j][0] * iA, o[j][1] * iA);
-  }
-  if (rowB < p.seq_len) {
-    float *dst = p.out + (((size_t)b * p.seq_len + rowB) * p.num_heads + h) * APF_D + 2 * t;
+  for (int half = 0; half < 2; half++) {
+    const int row = half ? rowB : rowA;
+    if (row >= p.seq_len) continue;
+    const float l = half ? lB : lA;
+    const size_t z = (size_t)b * p.seq_len + row;
+    float inv = l > 0.0f ? 1.0f / l : 0.0f;
+    if (p.gate) inv *= 1.0f / (1.0f + expf(-p.gate[z * p.gate_stride + h]));
+    if (p.out_bf16) {
+      __nv_bfloat16 *dst = p.out_bf16 + z * p.out_stride + (size_t)h * APF_D + 2 * t;
 #pragma unroll
-    for (int j = 0; j < 16; j++) *reinterpret_cast<float2 *>(dst + 8 * j) = make_float2(o[j][2] * iB, o[j][3] * iB);
+      for (int j = 0; j < 16; j++) *reinterpret_cast<__nv_bfloat162 *>(dst + 8 * j) = __floats2bfloat162_rn(o[j][2 * half] * inv, o[j][2 * half + 1] * inv);
+    } else {
+      float *dst = p.out + (z * p.num_heads + h) * APF_D + 2 * t;
+#pragma unroll
+      for (int j = 0; j < 16; j++) *reinterpret_cast<float2 *>(dst + 8 * j) = make_float2(o[j][2 * half] * inv, o[j][2 * half + 1] * inv);
+    }
   }
 }
 
@@ -224,6 +235,7 @@ bool dpk_attention_prefill_eligible(const dpk_attn_params &p) {
   if (G != 1 && G != 2 && G != 4 && G != 8) return false;
   if (p.sliding_window > 0 || p.softcap > 0.0f || p.kv_start != 0) return false;
   if (p.kv_batch_stride % 8 || (((uintptr_t)p.k | (uintptr_t)p.v) & 15) || ((uintptr_t)p.q & 7) || ((uintptr_t)p.out & 7)) return false;
+  if (p.out_bf16 && (p.out_stride % 2 || ((uintptr_t)p.out_bf16 & 3))) return false;
   return true;
 }
 

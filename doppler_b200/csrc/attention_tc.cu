@@ -18,6 +18,7 @@
 // with cp.async (16 B per lane, rows XOR-swizzled so that ldmatrix is conflict free), so warps
 // never wait for one another inside the key loop.  K fragments come from ldmatrix, V^T fragments
 // from ldmatrix.trans.  Two CTAs of four warps per SM keep 128 KB of KV reads in flight per SM.
+#include "attn_out.cuh"
 #include "common.h"
 #include "pdl.cuh"
 
@@ -74,13 +75,8 @@ __global__ void __launch_bounds__(ATC_THREADS, 2) attn_tc_kernel(dpk_attn_params
   const int h0 = kvh * G + ht * gt;
 
   int kv_len = p.kv_lens ? min(max(p.kv_lens[b], 0), p.kv_len) : p.kv_len;  // the host checked the cache for p.kv_len keys
-  int lo = 0, hi = kv_len;
-  {
-    const int abs_q = p.start_pos + qi;
-    if (p.causal) { const int lim = abs_q - p.kv_start + 1; if (lim < hi) hi = lim; }
-    if (p.sliding_window > 0 && abs_q >= p.sliding_window) { const int first = abs_q - p.sliding_window + 1 - p.kv_start; if (first > lo) lo = first; }
-    if (hi < lo) hi = lo;
-  }
+  const AttnRange range = attn_range(p, kv_len, qi);
+  const int lo = range.lo, hi = range.hi;
   const int n_keys = hi - lo;
   const int per_split = (n_keys + splits - 1) / splits;
   const int k_begin = lo + split * per_split;
@@ -94,11 +90,12 @@ __global__ void __launch_bounds__(ATC_THREADS, 2) attn_tc_kernel(dpk_attn_params
   // A fragments of Q for every k-step: rows g (hi) and g+8 (lo).  This lane owns dims 16ks + 2t + {0,1,8,9}.
   const bool fused = p.fuse.qkv != nullptr;
   const int new_pos = fused ? p.fuse.pos[b] : -1;  // the key that is not in the cache yet
+  const size_t fuse_stride = p.fuse.row_stride ? p.fuse.row_stride : (size_t)(p.fuse.nh + 2 * p.fuse.nkv) * D;
   uint32_t qa[KS][4];
   {
     float x[KS][4];
     if (g < gt) {
-      const float *qrow = fused ? p.fuse.qkv + ((size_t)b * (p.fuse.nh + 2 * p.fuse.nkv) + h0 + g) * D
+      const float *qrow = fused ? p.fuse.qkv + (size_t)b * fuse_stride + (size_t)(h0 + g) * D
                                 : p.q + ((size_t)z * p.num_heads + h0 + g) * D;
 #pragma unroll
       for (int ks = 0; ks < KS; ks++) {
@@ -129,10 +126,16 @@ __global__ void __launch_bounds__(ATC_THREADS, 2) attn_tc_kernel(dpk_attn_params
 #pragma unroll
           for (int j = 0; j < 4; j++) {
             const int d = 16 * ks + 2 * t + (j & 1) + (j >> 1) * 8;
-            const float a = x[ks][j] * inv * p.fuse.q_norm[d], bb = x[ks + KS / 2][j] * inv * p.fuse.q_norm[d + HALF];
-            const float c = p.fuse.cos_t[(size_t)new_pos * HALF + d], sn = p.fuse.sin_t[(size_t)new_pos * HALF + d];
-            x[ks][j] = a * c - bb * sn;
-            x[ks + KS / 2][j] = a * sn + bb * c;
+            float a = x[ks][j] * inv, bb = x[ks + KS / 2][j] * inv;
+            if (p.fuse.q_norm) { a *= p.fuse.q_norm[d]; bb *= p.fuse.q_norm[d + HALF]; }
+            if (p.fuse.cos_t) {
+              const float c = p.fuse.cos_t[(size_t)new_pos * HALF + d], sn = p.fuse.sin_t[(size_t)new_pos * HALF + d];
+              const float ra = a * c - bb * sn;
+              bb = a * sn + bb * c;
+              a = ra;
+            }
+            x[ks][j] = a;
+            x[ks + KS / 2][j] = bb;
           }
       }
     }
@@ -201,8 +204,7 @@ __global__ void __launch_bounds__(ATC_THREADS, 2) attn_tc_kernel(dpk_attn_params
       // rounded to f16 as the cache write does) and V row, put them into the stage and, once per KV head,
       // append them to the cache (kv_cache_write_f32_to_f16.wgsl:19).
       constexpr int HALF = D / 2, PER = HALF / 32;
-      const int heads_all = p.fuse.nh + 2 * p.fuse.nkv;
-      const float *ksrc = p.fuse.qkv + ((size_t)b * heads_all + p.fuse.nh + kvh) * D;
+      const float *ksrc = p.fuse.qkv + (size_t)b * fuse_stride + (size_t)(p.fuse.nh + kvh) * D;
       const float *vsrc = ksrc + (size_t)p.fuse.nkv * D;
       float k0[PER], k1[PER], v0[PER], v1[PER];
       float ss = 0.0f;
@@ -222,9 +224,15 @@ __global__ void __launch_bounds__(ATC_THREADS, 2) attn_tc_kernel(dpk_attn_params
 #pragma unroll
       for (int e = 0; e < PER; e++) {
         const int d = lane + 32 * e;
-        const float a = k0[e] * inv * p.fuse.k_norm[d], bb = k1[e] * inv * p.fuse.k_norm[d + HALF];
-        const float c = p.fuse.cos_t[(size_t)new_pos * HALF + d], sn = p.fuse.sin_t[(size_t)new_pos * HALF + d];
-        const __half ka = __float2half_rn(a * c - bb * sn), kb = __float2half_rn(a * sn + bb * c);
+        float a = k0[e] * inv, bb = k1[e] * inv;
+        if (p.fuse.k_norm) { a *= p.fuse.k_norm[d]; bb *= p.fuse.k_norm[d + HALF]; }
+        if (p.fuse.cos_t) {
+          const float c = p.fuse.cos_t[(size_t)new_pos * HALF + d], sn = p.fuse.sin_t[(size_t)new_pos * HALF + d];
+          const float ra = a * c - bb * sn;
+          bb = a * sn + bb * c;
+          a = ra;
+        }
+        const __half ka = __float2half_rn(a), kb = __float2half_rn(bb);
         const __half va = __float2half_rn(v0[e]), vb = __float2half_rn(v1[e]);
         const int d2 = d + HALF;
         *reinterpret_cast<__half *>(rowK + ((((d >> 3) ^ rsw)) << 4) + (d & 7) * 2) = ka;
@@ -341,7 +349,7 @@ __global__ void __launch_bounds__(ATC_THREADS, 2) attn_tc_kernel(dpk_attn_params
     }
     const int h = h0 + hh;
     if (splits == 1) {
-      p.out[((size_t)z * p.num_heads + h) * D + d] = ll > 0.0f ? acc / ll : 0.0f;
+      attn_store(p, z, h, D, d, ll > 0.0f ? acc / ll : 0.0f);
     } else {
       float *pp = part + (((size_t)z * p.num_heads + h) * splits + split) * (D + 2);
       pp[d] = acc;

@@ -2,6 +2,7 @@
 #pragma once
 
 #include <cuda_runtime.h>
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 
 #include <cstdarg>
@@ -138,6 +139,7 @@ static inline size_t dp_dtype_size(dp_dtype t) {
     case DP_F32: return 4;
     case DP_F16: return 2;
     case DP_I32: return 4;
+    case DP_BF16: return 2;
     default: return 0;
   }
 }
@@ -148,6 +150,7 @@ static inline const char *dp_dtype_name(dp_dtype t) {
     case DP_F16: return "f16";
     case DP_Q4K: return "q4k";
     case DP_I32: return "i32";
+    case DP_BF16: return "bf16";
   }
   return "?";
 }
@@ -218,7 +221,9 @@ struct dpk_attn_fuse {
   __half *kc = nullptr, *vc = nullptr;
   float eps = 0.0f;
   int nh = 0, nkv = 0;
+  size_t row_stride = 0;     // floats between the rows of two sequences in qkv (0: (nh + 2 nkv) * head_dim)
 };
+// (q_norm / k_norm null: heads divided by their root mean square without a weight; cos_t null: no rotation)
 struct dpk_attn_params {
   dpk_attn_fuse fuse;
   const float *q;
@@ -229,6 +234,15 @@ struct dpk_attn_params {
   int causal, start_pos, sliding_window, kv_start;
   size_t kv_batch_stride;
   const int *kv_lens;
+  int chunk = 0;             // > 0: a query at position i sees only the keys j with floor(j / chunk) == floor(i / chunk)
+  int v_dim = 0;             // value size per head (0: head_dim); other sizes, and f32 caches, run on the generic kernel
+  bool kv_f32 = false;       // k and v point at f32 caches
+  size_t v_batch_stride = 0; // elements between the sequences of v (0: kv_batch_stride)
+  // output gate: row r's head h times sigmoid(gate[r * gate_stride + h]); null: none (kernels that write `out` only)
+  const float *gate = nullptr;
+  int gate_stride = 0;
+  __nv_bfloat16 *out_bf16 = nullptr;  // rows of out_stride elements, written instead of `out`
+  int out_stride = 0;
 };
 dp_status dpk_attention(dp_ctx *ctx, const dpk_attn_params &p);
 bool dpk_attention_uses_tc(dp_ctx *ctx, const dpk_attn_params &p);

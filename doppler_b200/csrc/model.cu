@@ -20,6 +20,7 @@
 #include "tp_exchange.h"
 #include "gemv_exchange.h"
 #include "handoff.cuh"
+#include "model.h"
 
 #include <cfloat>
 #include <cmath>
@@ -47,51 +48,6 @@ bool dp_tp_ready(dp_ctx *ctx);
 dp_tp_exchange *dp_tp_exchange_desc(dp_ctx *ctx);
 bool dp_tp_exchange_view(dp_ctx *ctx, int *rank, int *size, uint2 **areas);
 dp_status dp_take_dev_status(dp_ctx *ctx);
-
-struct LayerW {
-  dp_buf qkv = nullptr, o = nullptr, gateup = nullptr, down = nullptr;
-  float *in_norm = nullptr, *post_norm = nullptr, *q_norm = nullptr, *k_norm = nullptr;
-};
-
-struct dp_model {
-  dp_ctx *ctx;
-  dp_model_cfg cfg;
-  int nh, nkv, qdim, kvdim, inter, vocab_l, vocab0;  // this rank's share
-  int T;                                              // rows of the activation buffers
-  std::vector<LayerW> layers;
-  dp_buf norms = nullptr, embed = nullptr, lm_head = nullptr;
-  float *final_norm = nullptr;
-  std::vector<dp_buf> kc, vc;
-  dp_buf rope = nullptr;
-  float *rope_cos = nullptr, *rope_sin = nullptr;
-  dp_buf act = nullptr;  // one slab for all activations
-  float *h, *n, *qkv, *q, *att, *gu, *actv, *partial, *logits;
-  float *hbuf[3];       // tensor-parallel single-token decode: the residual stream rotates over three buffers (hbuf[0] == h);
-                        // a kernel reads one and its CTAs write their shares of the next, so none overwrites what another still reads
-  float *h_last;        // where the last forward pass left the hidden state
-  unsigned *d_ticket = nullptr;   // device counter of decode steps ever run on this CONTEXT (its exchange area outlives a model):
-                                  // hand-off tickets derive from it and never repeat
-  dp_buf state = nullptr;  // device ints: pos[B], kvlen[B], tok[B], step, then argmax scratch
-  int *d_pos, *d_kvlen, *d_tok, *d_step;
-  float *am_vals; int *am_idx; float *am_best; int *am_pair_i; float *am_gather;
-  dp_buf out_tokens = nullptr;
-  int out_tokens_cap = 0;
-  int *pin_state = nullptr;   // page-locked staging of the per-call state block (1024 words) + the status word read back
-  int *pin_out = nullptr;     // page-locked staging of the decoded tokens (out_tokens_cap words)
-  dp_buf attn_scratch = nullptr;
-  dp_buf actq = nullptr;  // fixed-point activation digits of the decode GEMV (sized for the largest K)
-  int attn_splits_decode = 1;
-  bool recording_decode = false;  // set while a decode step is recorded into its CUDA graph
-  bool fuse_qk = true;  // decode: QK norm + RoPE + KV append inside the attention kernel
-  std::vector<int> seq_len;
-  dp_graph *graph[2] = {nullptr, nullptr};
-  int graph_batch[2] = {0, 0};
-  cudaEvent_t ev0 = nullptr, ev1 = nullptr;
-  double last_ms = 0;
-  size_t weight_bytes = 0;
-  int allreduce_mode = 0;
-  bool final_norm_done = false;  // set by run_layers when the exchange kernel already applied the final RMSNorm
-};
 
 // ---- model-specific kernels ---------------------------------------------------
 
@@ -418,6 +374,26 @@ __global__ void __launch_bounds__(256) xchg_rmsnorm_kernel(const __grid_constant
 static size_t q4k_bytes(size_t n, size_t k) { return n * dp_cdiv(k, DP_QK_K) * DP_Q4K_BLOCK_BYTES; }
 static size_t align_up(size_t v, size_t a) { return dp_cdiv(v, a) * a; }
 
+// device state of the decode loop (positions, lengths, tokens, step counter), logits, argmax scratch and events
+dp_status dp_model_alloc_runner(dp_model *m) {
+  dp_ctx *ctx = m->ctx;
+  const size_t B = m->cfg.max_batch;
+  DP_TRY(dp_buf_acquire(ctx, 4096 + 1024 + 2048 + 16384 + B * 256 * 8, "decode_state", &m->state));
+  DP_TRY(dp_buf_acquire(ctx, B * m->vocab_l * 4, "logits", &m->logits_buf));
+  m->logits = (float *)m->logits_buf->dptr;
+  int *si = (int *)m->state->dptr;
+  m->d_pos = si; m->d_kvlen = si + 256; m->d_tok = si + 512; m->d_step = si + 768;
+  char *sp = (char *)m->state->dptr + 4096;
+  m->am_best = (float *)sp; sp += 1024;             // best logit per sequence
+  m->am_pair_i = (int *)sp; sp += 2048;             // (value, index) per sequence, this rank
+  m->am_gather = (float *)sp; sp += 16384;          // the pairs of up to 8 ranks
+  m->am_vals = (float *)sp; m->am_idx = (int *)(m->am_vals + B * 256);
+  m->d_ticket = (unsigned *)(ctx->dev_status + 16);  // zeroed with the context, then only ever incremented
+  if (cudaEventCreate(&m->ev0) != cudaSuccess || cudaEventCreate(&m->ev1) != cudaSuccess)
+    return dp_fail(ctx, DP_ERR_CUDA, "model: cudaEventCreate failed");
+  return dp_buf_fill(ctx, m->state, 0, 0, m->state->bytes);
+}
+
 extern "C" dp_status dp_model_create(dp_ctx *ctx, const dp_model_cfg *cfg, dp_model **out) {
   if (!ctx || !cfg || !out) return DP_ERR_INVALID;
   const dp_model_cfg &c = *cfg;
@@ -472,9 +448,8 @@ extern "C" dp_status dp_model_create(dp_ctx *ctx, const dp_model_cfg *cfg, dp_mo
   acquire((size_t)c.max_seq * D * 4, "rope_tables", &m->rope);
   const size_t T = m->T;
   const size_t n_h = align_up(T * H, 64), n_qkv = align_up(T * (m->qdim + 2 * m->kvdim), 64), n_q = align_up(T * m->qdim, 64);
-  const size_t n_gu = align_up(T * 2 * m->inter, 64), n_act = align_up(T * m->inter, 64), n_log = align_up((size_t)B * m->vocab_l, 64);
-  acquire((3 * n_h + n_qkv + 2 * n_q + n_gu + n_act + n_log + 2 * align_up(H, 64)) * 4, "activations", &m->act);
-  acquire(4096 + 1024 + 2048 + 16384 + (size_t)B * 256 * 8, "decode_state", &m->state);
+  const size_t n_gu = align_up(T * 2 * m->inter, 64), n_act = align_up(T * m->inter, 64);
+  acquire((3 * n_h + n_qkv + 2 * n_q + n_gu + n_act + 2 * align_up(H, 64)) * 4, "activations", &m->act);
   // split-K scratch sized for the longest context
   dpk_attn_params ap{};
   ap.batch = B; ap.seq_len = 1; ap.kv_len = c.max_seq; ap.num_heads = m->nh; ap.num_kv_heads = m->nkv; ap.head_dim = D;
@@ -496,17 +471,9 @@ extern "C" dp_status dp_model_create(dp_ctx *ctx, const dp_model_cfg *cfg, dp_mo
   m->final_norm = nb;
   float *a = (float *)m->act->dptr;
   m->h = a; a += n_h; m->n = a; a += n_h; m->partial = a; a += n_h; m->qkv = a; a += n_qkv; m->q = a; a += n_q;
-  m->att = a; a += n_q; m->gu = a; a += n_gu; m->actv = a; a += n_act; m->logits = a; a += n_log;
+  m->att = a; a += n_q; m->gu = a; a += n_gu; m->actv = a; a += n_act;
   m->hbuf[0] = m->h; m->hbuf[1] = a; a += align_up(H, 64); m->hbuf[2] = a; a += align_up(H, 64);
   m->h_last = m->h;
-  int *si = (int *)m->state->dptr;
-  m->d_pos = si; m->d_kvlen = si + 256; m->d_tok = si + 512; m->d_step = si + 768;
-  char *sp = (char *)m->state->dptr + 4096;
-  m->am_best = (float *)sp; sp += 1024;             // best logit per sequence
-  m->am_pair_i = (int *)sp; sp += 2048;             // (value, index) per sequence, this rank
-  m->am_gather = (float *)sp; sp += 16384;          // the pairs of up to 8 ranks
-  m->am_vals = (float *)sp; m->am_idx = (int *)(m->am_vals + (size_t)B * 256);
-  m->d_ticket = (unsigned *)(ctx->dev_status + 16);  // zeroed with the context, then only ever incremented
   // rope tables (host build, init-rope.js semantics)
   {
     std::vector<float> cs((size_t)c.max_seq * D / 2), sn((size_t)c.max_seq * D / 2);
@@ -515,9 +482,7 @@ extern "C" dp_status dp_model_create(dp_ctx *ctx, const dp_model_cfg *cfg, dp_mo
     st = dp_buf_upload(ctx, m->rope, cs.data(), 0, cs.size() * 4);
     if (st == DP_OK) st = dp_buf_upload(ctx, m->rope, sn.data(), cs.size() * 4, sn.size() * 4);
   }
-  if (st == DP_OK && (cudaEventCreate(&m->ev0) != cudaSuccess || cudaEventCreate(&m->ev1) != cudaSuccess))
-    st = dp_fail(ctx, DP_ERR_CUDA, "model: cudaEventCreate failed");
-  if (st == DP_OK) st = dp_buf_fill(ctx, m->state, 0, 0, m->state->bytes);
+  if (st == DP_OK) st = dp_model_alloc_runner(m);
   if (st != DP_OK) { dp_model_destroy(m); return st; }
   *out = m;
   return DP_OK;
@@ -528,9 +493,10 @@ extern "C" void dp_model_destroy(dp_model *m) {
   dp_ctx *ctx = m->ctx;
   cudaStreamSynchronize(ctx->stream);
   for (int i = 0; i < 2; i++) if (m->graph[i]) dp_graph_destroy(m->graph[i]);
+  dp_stack_destroy(m);
   auto rel = [&](dp_buf b) { if (b) dp_buf_release(ctx, b); };
   for (LayerW &L : m->layers) { rel(L.qkv); rel(L.o); rel(L.gateup); rel(L.down); }
-  rel(m->norms); rel(m->embed); rel(m->lm_head); rel(m->rope); rel(m->act); rel(m->state); rel(m->out_tokens); rel(m->attn_scratch); rel(m->actq);
+  rel(m->norms); rel(m->embed); rel(m->lm_head); rel(m->rope); rel(m->act); rel(m->state); rel(m->logits_buf); rel(m->out_tokens); rel(m->attn_scratch); rel(m->actq);
   for (dp_buf b : m->kc) rel(b);
   for (dp_buf b : m->vc) rel(b);
   if (m->pin_state) cudaFreeHost(m->pin_state);
@@ -545,6 +511,7 @@ extern "C" dp_status dp_model_load_q4k(dp_model *m, int layer, dp_weight_id whic
   if (!m) return DP_ERR_INVALID;
   dp_ctx *ctx = m->ctx;
   const dp_model_cfg &c = m->cfg;
+  DP_CHECK(ctx, !m->stack, "loadQ4K: a decoder described layer by layer takes dp_model_load_tensor");
   DP_CHECK(ctx, layer >= 0 && layer < c.n_layers, "loadQ4K: layer %d out of range", layer);
   DP_CHECK(ctx, host != nullptr, "loadQ4K: null host pointer");
   const int p = c.tp_size, r = c.tp_rank, H = c.hidden;
@@ -592,6 +559,7 @@ extern "C" dp_status dp_model_load_q4k(dp_model *m, int layer, dp_weight_id whic
 extern "C" dp_status dp_model_load_norm(dp_model *m, int layer, dp_weight_id which, const float *host, int n) {
   if (!m) return DP_ERR_INVALID;
   dp_ctx *ctx = m->ctx;
+  DP_CHECK(ctx, !m->stack, "loadNorm: a decoder described layer by layer takes dp_model_load_tensor");
   DP_CHECK(ctx, layer >= 0 && layer < m->cfg.n_layers && host, "loadNorm: bad layer or null pointer");
   LayerW &L = m->layers[layer];
   float *dst; int want;
@@ -608,12 +576,14 @@ extern "C" dp_status dp_model_load_norm(dp_model *m, int layer, dp_weight_id whi
 
 extern "C" dp_status dp_model_load_final_norm(dp_model *m, const float *host, int n) {
   if (!m || !host) return DP_ERR_INVALID;
+  DP_CHECK(m->ctx, !m->stack, "loadFinalNorm: a decoder described layer by layer takes dp_model_load_tensor");
   DP_CHECK(m->ctx, n == m->cfg.hidden, "loadFinalNorm: expected %d values, got %d", m->cfg.hidden, n);
   return dp_buf_upload(m->ctx, m->norms, host, (size_t)((char *)m->final_norm - (char *)m->norms->dptr), (size_t)n * 4);
 }
 
 extern "C" dp_status dp_model_load_embed(dp_model *m, const void *host, int row0, int rows) {
   if (!m || !host) return DP_ERR_INVALID;
+  DP_CHECK(m->ctx, !m->stack, "loadEmbed: a decoder described layer by layer takes dp_model_load_tensor");
   DP_CHECK(m->ctx, row0 >= 0 && rows >= 0 && row0 + rows <= m->cfg.vocab, "loadEmbed: rows [%d,%d) outside the vocabulary", row0, row0 + rows);
   return dp_buf_upload(m->ctx, m->embed, host, (size_t)row0 * m->cfg.hidden * 2, (size_t)rows * m->cfg.hidden * 2);
 }
@@ -621,6 +591,7 @@ extern "C" dp_status dp_model_load_embed(dp_model *m, const void *host, int row0
 // rows are GLOBAL vocabulary rows; only the part that falls in this rank's shard is kept
 extern "C" dp_status dp_model_load_lm_head(dp_model *m, const void *host, int row0, int rows) {
   if (!m || !host) return DP_ERR_INVALID;
+  DP_CHECK(m->ctx, !m->stack, "loadLmHead: a decoder described layer by layer takes dp_model_load_tensor");
   DP_CHECK(m->ctx, row0 >= 0 && rows >= 0 && row0 + rows <= m->cfg.vocab, "loadLmHead: rows [%d,%d) outside the vocabulary", row0, row0 + rows);
   int lo = row0 > m->vocab0 ? row0 : m->vocab0;
   int hi = row0 + rows < m->vocab0 + m->vocab_l ? row0 + rows : m->vocab0 + m->vocab_l;
@@ -642,6 +613,7 @@ extern "C" double dp_model_last_decode_ms(dp_model *m) { return m ? m->last_ms :
 extern "C" dp_status dp_model_set_allreduce_mode(dp_model *m, int mode) {
   if (!m) return DP_ERR_INVALID;
   if (mode != 0 && mode != 1) return dp_fail(m->ctx, DP_ERR_INVALID, "model: unknown allreduce mode %d", mode);
+  DP_CHECK(m->ctx, !m->stack, "model: a decoder described layer by layer runs on one GPU");
   if (mode == 1) {
     if (m->cfg.tp_size > 1 && !dp_tp_exchange_desc(m->ctx))
       return dp_fail(m->ctx, DP_ERR_STATE, "model: allreduce mode 1 needs the peer-memory exchange area (dp_tp_ipc_export / dp_tp_ipc_attach)");
@@ -857,6 +829,7 @@ static dp_status rows_linear_fused(dp_model *m, const uint8_t *W, const float *A
 }
 
 static dp_status run_layers(dp_model *m, int tokens, bool decode, int seq, int start_pos) {
+  if (m->stack) return dp_stack_run_layers(m, tokens, decode, seq, start_pos);
   dp_ctx *ctx = m->ctx;
   const dp_model_cfg &c = m->cfg;
   const int H = c.hidden, D = c.head_dim, p = c.tp_size;
@@ -1029,14 +1002,22 @@ static dp_status run_layers(dp_model *m, int tokens, bool decode, int seq, int s
   return DP_OK;
 }
 
-// final norm + LM head + greedy argmax for `rows` rows of hidden state starting at hrow
-static dp_status run_head(dp_model *m, const float *hrow, int rows) {
+// final norm + LM head for `rows` rows of hidden state starting at hrow -> m->logits
+static dp_status run_logits(dp_model *m, const float *hrow, int rows) {
+  if (m->stack) return dp_stack_logits(m, hrow, rows);
   dp_ctx *ctx = m->ctx;
   const dp_model_cfg &c = m->cfg;
   if (!(m->final_norm_done && rows == 1))
     DP_TRY(dpk_rmsnorm(ctx, hrow, m->final_norm, false, nullptr, false, nullptr, m->n, rows, c.hidden, c.eps, false, 1.0f));
   m->final_norm_done = false;
-  DP_TRY(dpk_gemv_f16w(ctx, (const __half *)m->lm_head->dptr, m->n, DP_F32, m->logits, DP_F32, rows, m->vocab_l, c.hidden, 1.0f));
+  return dpk_gemv_f16w(ctx, (const __half *)m->lm_head->dptr, m->n, DP_F32, m->logits, DP_F32, rows, m->vocab_l, c.hidden, 1.0f);
+}
+
+// ... and the greedy argmax of every row -> m->d_tok
+static dp_status run_head(dp_model *m, const float *hrow, int rows) {
+  dp_ctx *ctx = m->ctx;
+  const dp_model_cfg &c = m->cfg;
+  DP_TRY(run_logits(m, hrow, rows));
   if (rows == 1)
     DP_TRY(dpk_argmax(ctx, m->logits, m->vocab_l, -1, m->d_tok, 0, m->am_vals, m->am_idx, m->vocab0, m->am_best));
   else  // all rows in two launches
@@ -1057,40 +1038,80 @@ static dp_status run_head(dp_model *m, const float *hrow, int rows) {
   return DP_OK;
 }
 
-extern "C" dp_status dp_model_prefill(dp_model *m, int seq, const int32_t *tokens, int n, int32_t *next_token) {
-  if (!m) return DP_ERR_INVALID;
+// token ids on the device -> the rows the layers start from
+static dp_status embed_rows(dp_model *m, const int *ids, int rows, bool decode) {
+  if (m->stack) return dp_stack_embed(m, ids, rows, decode);
+  return dpk_gather_f16(m->ctx, ids, (const __half *)m->embed->dptr, m->h, rows, m->cfg.hidden);
+}
+
+// One portion of a sequence: `n` tokens that follow what the sequence holds already, in blocks of at most m->T rows.
+// want: ascending places among the n tokens whose logits are copied to `logits` [n_want][vocabulary share].
+// next_token (optional): the greedy token after the last one.
+static dp_status run_portion(dp_model *m, const char *op, int seq, const int32_t *tokens, int n, const int32_t *want, int n_want, float *logits,
+                             int32_t *next_token) {
   dp_ctx *ctx = m->ctx;
   const dp_model_cfg &c = m->cfg;
-  DP_CHECK(ctx, seq >= 0 && seq < c.max_batch, "prefill: sequence %d outside [0,%d)", seq, c.max_batch);
-  DP_CHECK(ctx, tokens && n > 0, "prefill: empty prompt");
-  DP_CHECK(ctx, m->seq_len[seq] + n <= c.max_seq, "prefill: %d + %d tokens exceed max_seq %d", m->seq_len[seq], n, c.max_seq);
-  for (int i = 0; i < n; i++) DP_CHECK(ctx, tokens[i] >= 0 && tokens[i] < c.vocab, "prefill: token id %d outside the vocabulary", tokens[i]);
+  DP_CHECK(ctx, seq >= 0 && seq < c.max_batch, "%s: sequence %d outside [0,%d)", op, seq, c.max_batch);
+  DP_CHECK(ctx, tokens && n > 0, "%s: empty prompt", op);
+  DP_CHECK(ctx, n <= c.max_seq - m->seq_len[seq], "%s: %d + %d tokens exceed max_seq %d", op, m->seq_len[seq], n, c.max_seq);
+  for (int i = 0; i < n; i++) DP_CHECK(ctx, tokens[i] >= 0 && tokens[i] < c.vocab, "%s: token id %d outside the vocabulary", op, tokens[i]);
+  for (int i = 0; i < n_want; i++)
+    DP_CHECK(ctx, want[i] >= 0 && want[i] < n && (i == 0 || want[i] > want[i - 1]), "%s: wanted place %d is not an ascending place among the %d tokens", op, want[i], n);
+  if (m->stack) DP_TRY(dp_stack_ready(m));
   dp_buf ids = nullptr;
   DP_TRY(dp_buf_acquire(ctx, (size_t)m->T * 4, "prefill_token_ids", &ids));
   dp_status st = DP_OK;
+  int w = 0;
   for (int off = 0; off < n && st == DP_OK; off += m->T) {
     const int cnt = n - off < m->T ? n - off : m->T;
     st = dp_buf_upload(ctx, ids, tokens + off, 0, (size_t)cnt * 4);
-    if (st == DP_OK) st = dpk_gather_f16(ctx, (const int *)ids->dptr, (const __half *)m->embed->dptr, m->h, cnt, c.hidden);
+    if (st == DP_OK) st = embed_rows(m, (const int *)ids->dptr, cnt, false);
     if (st == DP_OK) st = run_layers(m, cnt, false, seq, m->seq_len[seq]);
     if (st == DP_OK) {
       m->seq_len[seq] += cnt;
-      if (off + cnt >= n) st = run_head(m, m->h + (size_t)(cnt - 1) * c.hidden, 1);
+      for (; st == DP_OK && w < n_want && want[w] < off + cnt; w++) {
+        st = run_logits(m, m->h + (size_t)(want[w] - off) * c.hidden, 1);
+        if (st == DP_OK && cudaMemcpyAsync(logits + (size_t)w * m->vocab_l, m->logits, (size_t)m->vocab_l * 4, cudaMemcpyDeviceToHost, ctx->stream) != cudaSuccess)
+          st = dp_fail(ctx, DP_ERR_CUDA, "%s: copy of the logits failed", op);
+      }
+      if (next_token && st == DP_OK && off + cnt >= n) st = run_head(m, m->h + (size_t)(cnt - 1) * c.hidden, 1);
     }
   }
   dp_buf_release(ctx, ids);
   DP_TRY(st);
   int tok = 0;
-  DP_CUDA(ctx, cudaMemcpyAsync(&tok, m->d_tok, 4, cudaMemcpyDeviceToHost, ctx->stream));
+  if (next_token) DP_CUDA(ctx, cudaMemcpyAsync(&tok, m->d_tok, 4, cudaMemcpyDeviceToHost, ctx->stream));
   DP_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
   DP_TRY(dp_take_dev_status(ctx));  // a bounded device-side wait that gave up invalidates the result
   if (next_token) *next_token = tok;
   return DP_OK;
 }
 
+extern "C" dp_status dp_model_prefill(dp_model *m, int seq, const int32_t *tokens, int n, int32_t *next_token) {
+  if (!m) return DP_ERR_INVALID;
+  int32_t tok = 0;
+  DP_TRY(run_portion(m, "prefill", seq, tokens, n, nullptr, 0, nullptr, &tok));
+  if (next_token) *next_token = tok;
+  return DP_OK;
+}
+
+extern "C" dp_status dp_model_extend(dp_model *m, int seq, const int32_t *tokens, int n, const int32_t *want, int n_want, float *logits) {
+  if (!m) return DP_ERR_INVALID;
+  DP_CHECK(m->ctx, n_want == 0 || (n_want > 0 && want && logits), "extend: wanted places without a list or an output");
+  DP_CHECK(m->ctx, m->cfg.tp_size == 1 || n_want == 0, "extend: logits of a sharded vocabulary are not gathered");
+  return run_portion(m, "extend", seq, tokens, n, want, n_want, logits, nullptr);
+}
+
+extern "C" dp_status dp_model_release(dp_model *m, int seq) {
+  if (!m) return DP_ERR_INVALID;
+  DP_CHECK(m->ctx, seq >= 0 && seq < m->cfg.max_batch, "release: sequence %d outside [0,%d)", seq, m->cfg.max_batch);
+  m->seq_len[seq] = 0;  // a sequence's state is never read at or beyond its length, and position 0 starts from zeros
+  return DP_OK;
+}
+
 static dp_status record_decode_step(dp_model *m, int batch) {
   dp_ctx *ctx = m->ctx;
-  DP_TRY(dpk_gather_f16(ctx, m->d_tok, (const __half *)m->embed->dptr, m->h, batch, m->cfg.hidden));
+  DP_TRY(embed_rows(m, m->d_tok, batch, true));
   DP_TRY(run_layers(m, batch, true, 0, 0));
   DP_TRY(run_head(m, m->h, batch));
   DP_LAUNCH(ctx, advance_kernel, 1, 256, 0, m->d_pos, m->d_kvlen, m->d_tok, m->d_step, (int *)m->out_tokens->dptr, batch, m->d_ticket);
@@ -1107,6 +1128,7 @@ extern "C" dp_status dp_model_decode(dp_model *m, int batch, const int32_t *firs
     DP_CHECK(ctx, first_tokens[b] >= 0 && first_tokens[b] < c.vocab, "decode: token id %d outside the vocabulary", first_tokens[b]);
     DP_CHECK(ctx, m->seq_len[b] + steps <= c.max_seq, "decode: sequence %d would exceed max_seq %d", b, c.max_seq);
   }
+  if (m->stack) DP_TRY(dp_stack_ready(m));
   if (m->out_tokens_cap < steps * batch) {
     if (m->out_tokens) { dp_buf_release(ctx, m->out_tokens); m->out_tokens = nullptr; }
     for (int i = 0; i < 2; i++) if (m->graph[i]) { dp_graph_destroy(m->graph[i]); m->graph[i] = nullptr; }
@@ -1174,6 +1196,7 @@ extern "C" dp_status dp_model_bench_gemv(dp_model *m, int reps, double *ms_total
   dp_ctx *ctx = m->ctx;
   const dp_model_cfg &c = m->cfg;
   DP_CHECK(ctx, reps > 0, "bench_gemv: reps must be positive");
+  DP_CHECK(ctx, !m->stack, "bench_gemv: the model holds no Q4_K matrices");
   const int H = c.hidden;
   struct Shape { int N, K; };
   const Shape sh[4] = {{m->qdim + 2 * m->kvdim, H}, {H, m->qdim}, {2 * m->inter, H}, {H, m->inter}};

@@ -1,0 +1,316 @@
+// Residual streams (hyper-connections), grouped RMSNorm and the causal input convolution of a sublayer, for several
+// rows at once.  (A single decode row does all of this inside the GEMV kernels, gemv_bf16.cu.)
+//
+// The boundary kernel joins everything between two sublayers: x_t <- sum_s mix[s][t] x_s + out[t] y of the one that
+// ended, u = sum_t in[t] x_t, RMSNorm of u per group of channels, and h + conv(h) of the next one.  A group's norm
+// needs the channels of that group only, so a CTA owns (a block of rows, one group): one warp per row computes h
+// into shared memory, rows before the block (the convolution's reach) are recomputed or come from the sequence's
+// history, then all threads convolve.  x is read and written once per sublayer; h never goes to memory except for
+// the last taps - 1 rows of a portion.
+#include "layers.h"
+#include "pdl.cuh"
+
+namespace {
+
+constexpr int SB_THREADS = 256, SB_WARPS = SB_THREADS / 32;
+
+template <int V> struct FV { float v[V]; };
+template <int V> __device__ __forceinline__ FV<V> ldv(const float *p) {
+  FV<V> r;
+  if constexpr (V == 4) { const float4 a = *reinterpret_cast<const float4 *>(p); r.v[0] = a.x; r.v[1] = a.y; r.v[2] = a.z; r.v[3] = a.w; }
+  else r.v[0] = *p;
+  return r;
+}
+template <int V> __device__ __forceinline__ void stv(float *p, const FV<V> &r) {
+  if constexpr (V == 4) *reinterpret_cast<float4 *>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+  else *p = r.v[0];
+}
+template <int V> __device__ __forceinline__ void stv(__nv_bfloat16 *p, const FV<V> &r) {
+  if constexpr (V == 4) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(r.v[0], r.v[1]), b = __floats2bfloat162_rn(r.v[2], r.v[3]);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+  } else *p = __float2bfloat16_rn(r.v[0]);
+}
+template <int V> __device__ __forceinline__ FV<V> ldw(const __nv_bfloat16 *p) {
+  FV<V> r;
+#pragma unroll
+  for (int i = 0; i < V; i++) r.v[i] = __bfloat162float(p[i]);
+  return r;
+}
+
+struct BoundaryArgs {
+  const float *x, *y;
+  float *x_out;
+  SublayerOut end;
+  SublayerIn next;
+  int streams, width, rows, dst_stride, block_rows;
+  RowMap map;
+};
+
+template <int SM, int V, typename OutT>
+__global__ void __launch_bounds__(SB_THREADS) stream_boundary_kernel(const BoundaryArgs a, OutT *__restrict__ dst) {
+  pdl_launch();
+  pdl_wait();
+  extern __shared__ float sb_h[];  // [halo + block_rows][gs]
+  __shared__ float s_mix[SM * SM], s_out[SM], s_in[SM];
+  const int S = a.streams, H = a.width, gs = H / a.next.groups, taps = a.next.taps;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const bool per_seq = a.map.pos != nullptr;
+  const int halo = (per_seq || taps < 2) ? 0 : taps - 1;
+  const int row0 = blockIdx.x * a.block_rows, c0 = blockIdx.y * gs;
+  const int nrows = min(a.block_rows, a.rows - row0);
+  for (int i = tid; i < SM; i += SB_THREADS) {
+    s_in[i] = i < S ? a.next.in[i] : 0.0f;
+    s_out[i] = (i < S && a.y) ? a.end.out[i] : 0.0f;
+  }
+  for (int i = tid; i < SM * SM; i += SB_THREADS) {
+    const int s = i / SM, t = i % SM;
+    s_mix[i] = (s < S && t < S && a.y) ? a.end.mix[s * S + t] : 0.0f;
+  }
+  __syncthreads();
+
+  // ---- h of the block's rows and of the rows the convolution reaches back to: one warp per row ----
+  for (int j = warp; j < halo + nrows; j += SB_WARPS) {
+    const int row = row0 + j - halo;
+    float *h = sb_h + (size_t)j * gs;
+    if (row < 0) {  // before this portion: the sequence's history, zeros before its start
+      const int p = a.map.start_pos + row;
+      const float *src = a.next.hist + (size_t)a.map.seq * a.next.hist_seq + (size_t)(p >= 0 ? p % taps : 0) * H + c0;
+      for (int c = lane; c < gs; c += 32) h[c] = p >= 0 ? src[c] : 0.0f;
+      continue;
+    }
+    const float *xr = a.x + (size_t)row * S * H + c0;
+    float *xo = a.x_out + (size_t)row * S * H + c0;
+    const bool store = a.y && j >= halo;
+    float ss = 0.0f;
+    for (int c = lane * V; c < gs; c += 32 * V) {
+      FV<V> xs[SM], u;
+#pragma unroll
+      for (int i = 0; i < V; i++) u.v[i] = 0.0f;
+#pragma unroll
+      for (int s = 0; s < SM; s++)
+        if (s < S) xs[s] = ldv<V>(xr + (size_t)s * H + c);
+      if (a.y) {
+        const FV<V> yv = ldv<V>(a.y + (size_t)row * H + c0 + c);
+#pragma unroll
+        for (int t = 0; t < SM; t++) {
+          if (t < S) {
+            FV<V> n;
+#pragma unroll
+            for (int i = 0; i < V; i++) n.v[i] = s_out[t] * yv.v[i];
+#pragma unroll
+            for (int s = 0; s < SM; s++)
+              if (s < S)
+#pragma unroll
+                for (int i = 0; i < V; i++) n.v[i] = fmaf(s_mix[s * SM + t], xs[s].v[i], n.v[i]);
+            if (store) stv<V>(xo + (size_t)t * H + c, n);
+#pragma unroll
+            for (int i = 0; i < V; i++) u.v[i] = fmaf(s_in[t], n.v[i], u.v[i]);
+          }
+        }
+      } else {
+#pragma unroll
+        for (int s = 0; s < SM; s++)
+          if (s < S)
+#pragma unroll
+            for (int i = 0; i < V; i++) u.v[i] = fmaf(s_in[s], xs[s].v[i], u.v[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < V; i++) ss = fmaf(u.v[i], u.v[i], ss);
+      stv<V>(h + c, u);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float inv = 1.0f / sqrtf(ss / (float)gs + a.next.eps);
+    for (int c = lane * V; c < gs; c += 32 * V) {
+      FV<V> v = ldv<V>(h + c);
+      const FV<V> w = ldw<V>(a.next.norm_w + c0 + c);
+#pragma unroll
+      for (int i = 0; i < V; i++) v.v[i] = v.v[i] * inv * w.v[i];
+      stv<V>(h + c, v);
+    }
+  }
+  __syncthreads();
+
+  // ---- h + conv(h), the sublayer's input; the rows later tokens reach back to ----
+  const int cv = gs / V;
+  for (int idx = tid; idx < nrows * cv; idx += SB_THREADS) {
+    const int r = idx / cv, c = (idx - r * cv) * V, row = row0 + r;
+    const FV<V> h = ldv<V>(sb_h + (size_t)(halo + r) * gs + c);
+    FV<V> o = h;
+    if (taps > 0) {
+      const __nv_bfloat16 *w = a.next.conv_w + (size_t)(c0 + c) * taps;
+      const int pos = per_seq ? a.map.pos[row] : a.map.start_pos + row;
+      FV<V> acc;
+#pragma unroll
+      for (int i = 0; i < V; i++) acc.v[i] = 0.0f;
+      for (int k = taps - 1; k > 0; k--) {  // k positions back
+        FV<V> past;
+        if (per_seq) {
+#pragma unroll
+          for (int i = 0; i < V; i++) past.v[i] = 0.0f;
+          if (pos - k >= 0) past = ldv<V>(a.next.hist + (size_t)row * a.next.hist_seq + (size_t)((pos - k) % taps) * H + c0 + c);
+        } else {
+          past = ldv<V>(sb_h + (size_t)(halo + r - k) * gs + c);
+        }
+#pragma unroll
+        for (int i = 0; i < V; i++) acc.v[i] = fmaf(__bfloat162float(w[i * taps + taps - 1 - k]), past.v[i], acc.v[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < V; i++) o.v[i] = h.v[i] + fmaf(__bfloat162float(w[i * taps + taps - 1]), h.v[i], acc.v[i]);
+      if (taps > 1) {
+        if (per_seq) stv<V>(a.next.hist + (size_t)row * a.next.hist_seq + (size_t)(pos % taps) * H + c0 + c, h);
+        else if (row >= a.rows - (taps - 1)) stv<V>(a.next.stage + (size_t)(pos % taps) * H + c0 + c, h);
+      }
+    }
+    stv<V>(dst + (size_t)row * a.dst_stride + c0 + c, o);
+  }
+}
+
+template <int SM, int V>
+dp_status launch_boundary(dp_ctx *ctx, const BoundaryArgs &a, void *dst, bool bf16, dim3 grid, size_t smem) {
+  static dp_per_device_once attr;
+  if (attr.pending(ctx->device)) {
+    const int cap = (int)ctx->smem_optin - 4096;  // beside the kernel's static shared memory
+    DP_CUDA(ctx, cudaFuncSetAttribute((stream_boundary_kernel<SM, V, float>), cudaFuncAttributeMaxDynamicSharedMemorySize, cap));
+    DP_CUDA(ctx, cudaFuncSetAttribute((stream_boundary_kernel<SM, V, __nv_bfloat16>), cudaFuncAttributeMaxDynamicSharedMemorySize, cap));
+    attr.done(ctx->device);
+  }
+  if (bf16) DP_LAUNCH(ctx, (stream_boundary_kernel<SM, V, __nv_bfloat16>), grid, SB_THREADS, smem, a, (__nv_bfloat16 *)dst);
+  else DP_LAUNCH(ctx, (stream_boundary_kernel<SM, V, float>), grid, SB_THREADS, smem, a, (float *)dst);
+  return DP_OK;
+}
+
+__global__ void __launch_bounds__(256) stream_sum_kernel(const float *__restrict__ x, const float *__restrict__ y, const SublayerOut end, int S, int H,
+                                                         float *__restrict__ h, int rows) {
+  pdl_launch();
+  pdl_wait();
+  __shared__ float s_w[DP_MAX_STREAMS], s_o;
+  // sum_t (sum_s mix[s][t] x_s + out[t] y) = sum_s (sum_t mix[s][t]) x_s + (sum_t out[t]) y
+  if (threadIdx.x < (unsigned)S) {
+    float w = 0.0f;
+    for (int t = 0; t < S; t++) w += end.mix[threadIdx.x * S + t];
+    s_w[threadIdx.x] = w;
+  }
+  if (threadIdx.x == 32) {
+    float o = 0.0f;
+    for (int t = 0; t < S; t++) o += end.out[t];
+    s_o = o;
+  }
+  __syncthreads();
+  const size_t total = (size_t)rows * H;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = i / H, c = i - r * H;
+    float v = s_o * y[i];
+    for (int s = 0; s < S; s++) v = fmaf(s_w[s], x[(r * S + s) * H + c], v);
+    h[i] = v;
+  }
+}
+
+__global__ void __launch_bounds__(256) stream_embed_kernel(const int *__restrict__ ids, const __nv_bfloat16 *__restrict__ table, int table_stride, float scale,
+                                                           int S, int H, float *__restrict__ x, const float *__restrict__ in, float *__restrict__ u, int rows) {
+  pdl_launch();
+  pdl_wait();
+  float w = 0.0f;
+  if (u) for (int s = 0; s < S; s++) w += in[s];
+  const size_t total = (size_t)rows * H;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = i / H, c = i - r * H;
+    const float v = __bfloat162float(table[(size_t)ids[r] * table_stride + c]) * scale;
+    for (int s = 0; s < S; s++) x[(r * S + s) * H + c] = v;
+    if (u) u[i] = w * v;
+  }
+}
+
+template <typename OutT>
+__global__ void __launch_bounds__(256) group_norm_kernel(const float *__restrict__ x, int x_stride, const __nv_bfloat16 *__restrict__ w, int gs, float eps,
+                                                         OutT *__restrict__ dst, int dst_stride) {
+  pdl_launch();
+  pdl_wait();
+  __shared__ float sh[8];
+  const int c0 = blockIdx.y * gs, tid = threadIdx.x;
+  const float *xr = x + (size_t)blockIdx.x * x_stride + c0;
+  float ss = 0.0f;
+  for (int c = tid; c < gs; c += 256) ss = fmaf(xr[c], xr[c], ss);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if ((tid & 31) == 0) sh[tid >> 5] = ss;
+  __syncthreads();
+  float t = 0.0f;
+#pragma unroll
+  for (int i = 0; i < 8; i++) t += sh[i];
+  const float inv = 1.0f / sqrtf(t / (float)gs + eps);
+  OutT *d = dst + (size_t)blockIdx.x * dst_stride + c0;
+  for (int c = tid; c < gs; c += 256) {
+    const FV<1> v = {{xr[c] * inv * __bfloat162float(w[c0 + c])}};
+    stv<1>(d + c, v);
+  }
+}
+
+__global__ void __launch_bounds__(256) hist_commit_kernel(const HistEntry *__restrict__ entries, int rows, int start_pos, int seq) {
+  const HistEntry e = entries[blockIdx.y];
+  const int n = min(rows, e.taps - 1);
+  for (int c = blockIdx.x * 256 + threadIdx.x; c < e.channels; c += gridDim.x * 256)
+    for (int k = 0; k < n; k++) {
+      const size_t off = (size_t)((start_pos + rows - 1 - k) % e.taps) * e.channels + c;
+      e.hist[(size_t)seq * e.hist_seq + off] = e.stage[off];
+    }
+}
+
+unsigned flat_grid(dp_ctx *ctx, size_t n) {
+  size_t g = (n + 255) / 256;
+  const size_t cap = (size_t)ctx->sm_count * 16;
+  return (unsigned)(g < cap ? (g ? g : 1) : cap);
+}
+
+}  // namespace
+
+dp_status dpk_stream_boundary(dp_ctx *ctx, const float *x, float *x_out, const float *y, const SublayerOut &end, const SublayerIn &next, int streams, int width,
+                              void *dst, bool dst_bf16, int dst_stride, int rows, const RowMap &map) {
+  const int gs = width / next.groups;
+  const int halo = (map.pos || next.taps < 2) ? 0 : next.taps - 1;
+  const size_t row_bytes = (size_t)gs * 4;
+  // rows per CTA: as many as fit where two CTAs still share an SM, fewer when the launch would not fill the GPU
+  size_t cap = ((size_t)ctx->smem_optin - 4096) / row_bytes;
+  size_t want = (size_t)98304 / row_bytes;
+  if (want > 16) want = 16;  // two rounds of the CTA's eight warps, the reached-back rows included
+  if (want < 1 + (size_t)halo) want = 1 + (size_t)halo;
+  if (want > cap) return dp_fail(ctx, DP_ERR_UNSUPPORTED, "streams: %d channels per norm group and %d taps exceed shared memory", gs, next.taps);
+  int R = (int)want - halo;
+  if (map.pos) R = 1;
+  while (R > 4 && (long)((rows + R - 1) / R) * next.groups < 2l * ctx->sm_count) R = (R + 1) / 2;
+  BoundaryArgs a;
+  a.x = x; a.y = y; a.x_out = x_out; a.end = end; a.next = next;
+  a.streams = streams; a.width = width; a.rows = rows; a.dst_stride = dst_stride; a.block_rows = R; a.map = map;
+  const dim3 grid((rows + R - 1) / R, next.groups);
+  const size_t smem = (size_t)(R + halo) * row_bytes;
+  const bool vec = gs % 4 == 0 && dst_stride % 4 == 0;
+  if (streams <= 4) return vec ? launch_boundary<4, 4>(ctx, a, dst, dst_bf16, grid, smem) : launch_boundary<4, 1>(ctx, a, dst, dst_bf16, grid, smem);
+  return vec ? launch_boundary<DP_MAX_STREAMS, 4>(ctx, a, dst, dst_bf16, grid, smem) : launch_boundary<DP_MAX_STREAMS, 1>(ctx, a, dst, dst_bf16, grid, smem);
+}
+
+dp_status dpk_stream_sum(dp_ctx *ctx, const float *x, const float *y, const SublayerOut &end, int streams, int width, float *h, int rows) {
+  DP_LAUNCH(ctx, stream_sum_kernel, flat_grid(ctx, (size_t)rows * width), 256, 0, x, y, end, streams, width, h, rows);
+  return DP_OK;
+}
+
+dp_status dpk_stream_embed(dp_ctx *ctx, const int *ids, const __nv_bfloat16 *table, int table_stride, float scale, int streams, int width, float *x,
+                           const float *in, float *u, int rows) {
+  DP_LAUNCH(ctx, stream_embed_kernel, flat_grid(ctx, (size_t)rows * width), 256, 0, ids, table, table_stride, scale, streams, width, x, in, u, rows);
+  return DP_OK;
+}
+
+dp_status dpk_group_norm(dp_ctx *ctx, const float *x, int x_stride, const __nv_bfloat16 *w, int groups, float eps, int width, void *dst, bool dst_bf16,
+                         int dst_stride, int rows) {
+  const dim3 grid(rows, groups);
+  if (dst_bf16) DP_LAUNCH(ctx, group_norm_kernel<__nv_bfloat16>, grid, 256, 0, x, x_stride, w, width / groups, eps, (__nv_bfloat16 *)dst, dst_stride);
+  else DP_LAUNCH(ctx, group_norm_kernel<float>, grid, 256, 0, x, x_stride, w, width / groups, eps, (float *)dst, dst_stride);
+  return DP_OK;
+}
+
+dp_status dpk_hist_commit(dp_ctx *ctx, const HistEntry *entries, int n_entries, int max_channels, int rows, int start_pos, int seq) {
+  if (n_entries == 0) return DP_OK;
+  const dim3 grid((max_channels + 255) / 256, n_entries);
+  DP_LAUNCH(ctx, hist_commit_kernel, grid, 256, 0, entries, rows, start_pos, seq);
+  return DP_OK;
+}

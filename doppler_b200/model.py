@@ -1,4 +1,4 @@
-"""Decode / prefill runner for a dense Qwen3-shaped Q4_K model.
+"""Decode / prefill runner: the dense Qwen3-shaped Q4_K model and models described layer by layer.
 
 Host mirror of the scheduling slice of the reference text pipeline
 (``decodeStep`` src/inference/pipelines/text/generator-steps.js:588,
@@ -22,7 +22,79 @@ _Q4K_IDS = {"wq": L.W_Q, "wk": L.W_K, "wv": L.W_V, "wo": L.W_O, "wgate": L.W_GAT
 _NORM_IDS = {"in_norm": L.W_IN_NORM, "post_norm": L.W_POST_NORM, "q_norm": L.W_Q_NORM, "k_norm": L.W_K_NORM}
 
 
-class DecoderModel:
+class Runner:
+    """A model handle of the library and the calls every model answers.  Subclasses create the handle (``h``) and set
+    ``device``, ``cfg`` (with ``vocab``, ``hidden``, ``max_seq``), ``max_batch`` and ``tp_size``."""
+
+    h = None
+    tp_size = 1
+
+    # -- running ---------------------------------------------------------------------
+    def reset(self):
+        self.device.check(self.device.lib.dp_model_reset(self.h))
+
+    def prefill(self, tokens, seq: int = 0) -> int:
+        t = np.ascontiguousarray(tokens, np.int32)
+        nxt = C.c_int32()
+        self.device.check(self.device.lib.dp_model_prefill(self.h, seq, t.ctypes.data_as(C.c_void_p), t.size, C.byref(nxt)))
+        return int(nxt.value)
+
+    def decode(self, first_tokens, steps: int) -> np.ndarray:
+        """Greedy decode; returns int32 [steps, batch]."""
+        ft = np.ascontiguousarray(np.atleast_1d(first_tokens), np.int32)
+        out = np.empty((steps, ft.size), np.int32)
+        self.device.check(self.device.lib.dp_model_decode(self.h, ft.size, ft.ctypes.data_as(C.c_void_p), steps,
+                                                          out.ctypes.data_as(C.c_void_p)))
+        return out
+
+    @property
+    def last_decode_ms(self) -> float:
+        return float(self.device.lib.dp_model_last_decode_ms(self.h))
+
+    @property
+    def weight_bytes(self) -> int:
+        return int(self.device.lib.dp_model_weight_bytes(self.h))
+
+    def seq_len(self, seq: int = 0) -> int:
+        return int(self.device.lib.dp_model_seq_len(self.h, seq))
+
+    def read_logits(self, n: Optional[int] = None) -> np.ndarray:
+        n = n or self.cfg["vocab"] // self.tp_size
+        out = np.empty(n, np.float32)
+        self.device.check(self.device.lib.dp_model_read_logits(self.h, out.ctypes.data_as(C.c_void_p), n))
+        return out
+
+    def read_hidden(self, rows: int = 1) -> np.ndarray:
+        out = np.empty((rows, self.cfg["hidden"]), np.float32)
+        self.device.check(self.device.lib.dp_model_read_hidden(self.h, out.ctypes.data_as(C.c_void_p), out.size))
+        return out
+
+    def extend(self, tokens, want=(), seq: int = 0) -> np.ndarray:
+        """Run a portion of a sequence; returns the logits [len(want), vocab] at the wanted (ascending) places."""
+        t = np.ascontiguousarray(tokens, np.int32)
+        w = np.ascontiguousarray(want, np.int32)
+        out = np.empty((w.size, self.cfg["vocab"]), np.float32)
+        self.device.check(self.device.lib.dp_model_extend(self.h, seq, t.ctypes.data_as(C.c_void_p), t.size, w.ctypes.data_as(C.c_void_p), w.size,
+                                                          out.ctypes.data_as(C.c_void_p)))
+        return out
+
+    def release(self, seq: int = 0):
+        """Give back what a sequence holds; its slot starts again at position 0."""
+        self.device.check(self.device.lib.dp_model_release(self.h, seq))
+
+    @property
+    def state_bytes(self) -> int:
+        return int(self.device.lib.dp_model_state_bytes(self.h))
+
+    def destroy(self):
+        if self.h:
+            self.device.lib.dp_model_destroy(self.h)
+            self.h = None
+
+
+class DecoderModel(Runner):
+    """Dense Qwen3-shaped decoder with packed Q4_K matrices."""
+
     def __init__(self, device: Device, cfg: dict, max_seq: int, max_batch: int = 1, tp_rank: int = 0, tp_size: int = 1):
         self.device, self.cfg = device, dict(cfg)
         self.cfg["max_seq"] = max_seq
@@ -78,46 +150,6 @@ class DecoderModel:
                 self.load_lm_head(synthetic.make_lm_head(self.cfg, seed, lo, hi - lo), lo)
         self.load_final_norm(synthetic.make_final_norm(self.cfg, seed))
 
-    # -- running ---------------------------------------------------------------------
-    def reset(self):
-        self.device.check(self.device.lib.dp_model_reset(self.h))
-
-    def prefill(self, tokens, seq: int = 0) -> int:
-        t = np.ascontiguousarray(tokens, np.int32)
-        nxt = C.c_int32()
-        self.device.check(self.device.lib.dp_model_prefill(self.h, seq, t.ctypes.data_as(C.c_void_p), t.size, C.byref(nxt)))
-        return int(nxt.value)
-
-    def decode(self, first_tokens, steps: int) -> np.ndarray:
-        """Greedy decode; returns int32 [steps, batch]."""
-        ft = np.ascontiguousarray(np.atleast_1d(first_tokens), np.int32)
-        out = np.empty((steps, ft.size), np.int32)
-        self.device.check(self.device.lib.dp_model_decode(self.h, ft.size, ft.ctypes.data_as(C.c_void_p), steps,
-                                                          out.ctypes.data_as(C.c_void_p)))
-        return out
-
-    @property
-    def last_decode_ms(self) -> float:
-        return float(self.device.lib.dp_model_last_decode_ms(self.h))
-
-    @property
-    def weight_bytes(self) -> int:
-        return int(self.device.lib.dp_model_weight_bytes(self.h))
-
-    def seq_len(self, seq: int = 0) -> int:
-        return int(self.device.lib.dp_model_seq_len(self.h, seq))
-
-    def read_logits(self, n: Optional[int] = None) -> np.ndarray:
-        n = n or self.cfg["vocab"] // self.tp_size
-        out = np.empty(n, np.float32)
-        self.device.check(self.device.lib.dp_model_read_logits(self.h, out.ctypes.data_as(C.c_void_p), n))
-        return out
-
-    def read_hidden(self, rows: int = 1) -> np.ndarray:
-        out = np.empty((rows, self.cfg["hidden"]), np.float32)
-        self.device.check(self.device.lib.dp_model_read_hidden(self.h, out.ctypes.data_as(C.c_void_p), out.size))
-        return out
-
     def set_allreduce_mode(self, mode: int):
         """0: NCCL allreduce + residual add; 1: one-shot peer-memory exchange fused with the residual
         add and the next RMSNorm (single-token decode; needs tp.export_exchange + tp.attach_exchange)."""
@@ -129,7 +161,24 @@ class DecoderModel:
         self.device.check(self.device.lib.dp_model_bench_gemv(self.h, reps, C.byref(ms), C.byref(n), C.byref(b)))
         return {"ms": ms.value, "launches": int(n.value), "bytes": int(b.value)}
 
-    def destroy(self):
-        if self.h:
-            self.device.lib.dp_model_destroy(self.h)
-            self.h = None
+
+class StackModel(Runner):
+    """A decoder described layer by layer.  ``stack`` holds the fields of ``dp_stack_cfg`` that describe the model
+    (width, vocab, streams, norm_groups, input_taps, eps, embed_scale), ``layers`` one dictionary of ``dp_layer_cfg``
+    fields per layer.  ``dtype``: "bfloat16" (tensor cores, f16 K/V cache) or "float32" (every product in 32-bit)."""
+
+    def __init__(self, device: Device, stack: dict, layers: list, max_seq: int, max_batch: int = 1, dtype: str = "bfloat16", max_rows: int = 0):
+        self.device, self.max_batch, self.layers = device, max_batch, [dict(l) for l in layers]
+        self.cfg = dict(stack, hidden=stack["width"], n_layers=len(layers), max_seq=max_seq)
+        c = L.StackCfg(n_layers=len(layers), max_seq=max_seq, max_batch=max_batch, act_dtype={"bfloat16": L.BF16, "float32": L.F32}[dtype],
+                       max_rows=max_rows, **stack)
+        arr = (L.LayerCfg * len(layers))(*[L.LayerCfg(**l) for l in layers])
+        h = C.c_void_p()
+        device.check(device.lib.dp_model_create_stack(device.h, C.byref(c), arr, C.byref(h)))
+        self.h = h
+
+    def load_tensor(self, layer: int, tensor_id: int, bf16: np.ndarray):
+        """bf16 bits (uint16), vectors or matrices; layer -1 for the embedding and the final norm."""
+        a = np.ascontiguousarray(bf16, np.uint16)
+        rows, cols = (1, a.shape[0]) if a.ndim == 1 else a.shape
+        self.device.check(self.device.lib.dp_model_load_tensor(self.h, layer, tensor_id, a.ctypes.data_as(C.c_void_p), rows, cols))

@@ -46,7 +46,7 @@ typedef enum {
   DP_ERR_COMM = 7         /* NCCL / peer-memory failure */
 } dp_status;
 
-typedef enum { DP_F32 = 0, DP_F16 = 1, DP_Q4K = 2, DP_I32 = 3 } dp_dtype;
+typedef enum { DP_F32 = 0, DP_F16 = 1, DP_Q4K = 2, DP_I32 = 3, DP_BF16 = 4 } dp_dtype;
 
 typedef struct dp_ctx dp_ctx;
 typedef struct dp_buf_s *dp_buf; /* pooled device allocation (reference: GPUBuffer) */
@@ -350,6 +350,13 @@ dp_status dp_model_prefill(dp_model *m, int seq, const int32_t *tokens, int n, i
 /* `steps` greedy decode steps for `batch` sequences; out_tokens is [steps][batch] */
 dp_status dp_model_decode(dp_model *m, int batch, const int32_t *first_tokens, int steps,
                           int32_t *out_tokens);
+/* A portion of a sequence with logits: the n tokens continue what sequence `seq` holds, only they are run.
+ * want: n_want ascending places in [0,n); logits (host) receives [n_want][vocab] in that order.  Nothing is
+ * sampled.  The result does not depend on how a sequence was cut into portions, beyond rounding. */
+dp_status dp_model_extend(dp_model *m, int seq, const int32_t *tokens, int n, const int32_t *want, int n_want,
+                          float *logits);
+/* give back what sequence `seq` holds (its slot starts again at position 0) */
+dp_status dp_model_release(dp_model *m, int seq);
 /* timing of the last dp_model_decode (device time between events) and logits probe */
 double dp_model_last_decode_ms(dp_model *m);
 dp_status dp_model_read_logits(dp_model *m, float *host, int n);
@@ -365,6 +372,58 @@ dp_status dp_model_bench_gemv(dp_model *m, int reps, double *ms_total, uint64_t 
                               uint64_t *algorithmic_bytes);
 /* 0: NCCL allreduce; 1: one-shot peer-memory allreduce fused into the consumer kernels */
 dp_status dp_model_set_allreduce_mode(dp_model *m, int mode);
+
+/* ---- decoders described layer by layer ----------------------------------
+ * No counterpart in the reference's text pipeline (its layers are one dense shape).  A stack is an embedding, a list
+ * of layers and a tied head; each layer has a mixer (attention or a Mamba-2 recurrence) and optionally a dense
+ * feed-forward.  The handle is a dp_model: reset, prefill, extend, decode, release, read_logits, read_hidden and
+ * destroy are those above.  Every mechanism is a parameter:
+ *   streams      residual copies x_1..x_s.  A sublayer reads u = sum_s in[s] x_s and writes
+ *                x_t <- sum_s mix[s][t] x_s + out[t] y; 1 stream without loaded vectors is the plain residual sum.
+ *   norm_groups  RMSNorm of every one of that many equal consecutive parts of a row by itself.
+ *   input_taps   > 0: a sublayer reads h + causal depthwise convolution of h over time (weights [width, taps]).
+ *   chunk        > 0: a query sees the keys of its own chunk of positions only (chunks counted from position 0).
+ *   unit_rms_qk  q and k divided by their root mean square per head, no weight.
+ *   head_gate    head h's output times sigmoid((W_g x)_h).
+ *   ff           gated feed-forward: g = min(W_gate x, limit), u = clamp(W_up x, +-limit),
+ *                W_down (g * sigmoid(slope * g) * (u + shift)).
+ * Linear weights are bf16 [out, in].  act_dtype DP_BF16: matrix products of several rows on the tensor cores with
+ * bf16 activations, K and V cached as f16; DP_F32: every product in 32-bit, K and V cached as f32.  Residual
+ * streams, norms, scores, recurrent state and all vectors between kernels are f32 in both. */
+typedef enum { DP_MIXER_ATTENTION = 0, DP_MIXER_MAMBA2 = 1 } dp_mixer_kind;
+typedef struct {
+  int mixer; /* dp_mixer_kind */
+  int heads, vdim;
+  /* attention */
+  int kv_heads, dim, chunk, unit_rms_qk, head_gate;
+  float scale;
+  /* Mamba-2 */
+  int state, groups, conv_taps, norm_groups;
+  /* feed-forward; ff = 0: none */
+  int ff;
+  float ff_limit, ff_slope, ff_shift;
+} dp_layer_cfg;
+typedef struct {
+  int n_layers, width, vocab, max_seq, max_batch;
+  int streams, norm_groups, input_taps;
+  float eps, embed_scale;
+  int act_dtype; /* DP_BF16 or DP_F32 */
+  int max_rows;  /* rows of one block of a portion (0: chosen from max_seq) */
+} dp_stack_cfg;
+typedef enum {
+  DP_T_EMBED = 0, DP_T_FINAL_NORM,                           /* layer -1 */
+  DP_T_NORM1, DP_T_NORM2, DP_T_CONV1, DP_T_CONV2,            /* sublayer norms and input convolutions */
+  DP_T_HC1_IN, DP_T_HC1_OUT, DP_T_HC1_MIX, DP_T_HC2_IN, DP_T_HC2_OUT, DP_T_HC2_MIX,
+  DP_T_Q, DP_T_K, DP_T_V, DP_T_GATE_HEADS, DP_T_O,           /* attention; DP_T_O also Mamba-2 */
+  DP_T_SSM_IN, DP_T_SSM_CONV, DP_T_SSM_CONV_B, DP_T_SSM_DT_BIAS, DP_T_SSM_A_LOG, DP_T_SSM_D, DP_T_SSM_NORM,
+  DP_T_FF_GATE, DP_T_FF_UP, DP_T_FF_DOWN,
+  DP_T_COUNT
+} dp_tensor_id;
+dp_status dp_model_create_stack(dp_ctx *ctx, const dp_stack_cfg *cfg, const dp_layer_cfg *layers, dp_model **out);
+/* bf16 host data [rows, cols] (vectors: [1, n]); shapes are checked against the configuration */
+dp_status dp_model_load_tensor(dp_model *m, int layer, dp_tensor_id id, const void *host_bf16, int rows, int cols);
+/* bytes of K/V cache plus recurrent and convolution state, all sequences */
+size_t dp_model_state_bytes(dp_model *m);
 
 /* ---- tensor parallel group --------------------------------------------- */
 /* No counterpart in the reference (it has no collective backend; only the
