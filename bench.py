@@ -322,6 +322,113 @@ def kernels_record(dev, peak):
     }
 
 
+# Fenorax at the layer sizes of the dense workloads: per group of layers three Mamba-2 layers and one attention layer with
+# its feed-forward (random weights)
+STACK_SIZES = {
+    "9b": {"dense": "9b", "groups": 2, "stack": {"width": 4096, "vocab": 151936, "streams": 4, "norm_groups": 4, "input_taps": 4, "eps": 1e-6, "embed_scale": 1.0},
+           "mamba2": {"heads": 128, "vdim": 64, "state": 128, "groups": 8, "conv_taps": 4, "norm_groups": 8},
+           "attention": {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "chunk": 8192, "ff": 12288}},
+    "0.6b": {"dense": "qwen3-0.6b", "groups": 2,
+             "stack": {"width": 1024, "vocab": 151936, "streams": 4, "norm_groups": 2, "input_taps": 4, "eps": 1e-6, "embed_scale": 1.0},
+             "mamba2": {"heads": 32, "vdim": 64, "state": 128, "groups": 2, "conv_taps": 4, "norm_groups": 2},
+             "attention": {"heads": 16, "kv_heads": 8, "dim": 128, "vdim": 128, "chunk": 2048, "ff": 3072}},
+}
+
+
+def stack_model(dev, size, max_seq, seed=11):
+    """A Fenorax runner of one of STACK_SIZES; weights come from one pool of seeded gaussians, cut at random places."""
+    from doppler_b200 import _lib as L
+    from doppler_b200 import fenorax
+    from doppler_b200.model import StackModel
+    from doppler_b200.safetensors import bf16_bits
+
+    z = STACK_SIZES[size]
+    layers = []
+    for _ in range(z["groups"]):
+        layers += [dict(z["mamba2"], mixer=L.MIXER_MAMBA2) for _ in range(3)]
+        layers.append(dict(z["attention"], mixer=L.MIXER_ATTENTION, scale=z["attention"]["dim"] ** -0.5, unit_rms_qk=1, head_gate=1, ff_limit=7.0,
+                           ff_slope=fenorax.FF_SLOPE, ff_shift=fenorax.FF_SHIFT))
+    m = StackModel(dev, z["stack"], layers, max_seq)
+    rng = np.random.default_rng(seed)
+    pool = rng.standard_normal(1 << 22).astype(np.float32)
+    S, W = z["stack"]["streams"], z["stack"]["width"]
+
+    def mat(n, k):
+        bits = bf16_bits(pool / np.sqrt(k))
+        reps = -(-(n * k + bits.size) // bits.size)
+        return np.tile(bits, reps)[(o := int(rng.integers(bits.size))):o + n * k].reshape(n, k)
+
+    m.load_tensor(-1, L.T_EMBED, mat(z["stack"]["vocab"], W))
+    m.load_tensor(-1, L.T_FINAL_NORM, bf16_bits(np.ones(W)))
+    for i, l in enumerate(layers):
+        inner = l["heads"] * l["vdim"]
+        for q, ids in enumerate(((L.T_NORM1, L.T_CONV1, L.T_HC1_IN, L.T_HC1_OUT, L.T_HC1_MIX), (L.T_NORM2, L.T_CONV2, L.T_HC2_IN, L.T_HC2_OUT, L.T_HC2_MIX))):
+            if q and not l.get("ff"):
+                continue
+            m.load_tensor(i, ids[0], bf16_bits(np.ones(W)))
+            m.load_tensor(i, ids[1], bf16_bits(rng.standard_normal((W, z["stack"]["input_taps"])) * 0.1))
+            m.load_tensor(i, ids[2], bf16_bits(np.full(S, 1.0 / S)))
+            m.load_tensor(i, ids[3], bf16_bits(np.full(S, 0.5)))
+            m.load_tensor(i, ids[4], bf16_bits(np.eye(S) * 0.9 + 0.1 / S))
+        m.load_tensor(i, L.T_O, mat(W, inner))
+        if l["mixer"] == L.MIXER_MAMBA2:
+            ch = inner + 2 * l["groups"] * l["state"]
+            m.load_tensor(i, L.T_SSM_IN, mat(inner + ch + l["heads"], W))
+            m.load_tensor(i, L.T_SSM_CONV, bf16_bits(rng.standard_normal((ch, l["conv_taps"])) * 0.3))
+            for tid, n in ((L.T_SSM_CONV_B, ch), (L.T_SSM_DT_BIAS, l["heads"]), (L.T_SSM_A_LOG, l["heads"]), (L.T_SSM_D, l["heads"])):
+                m.load_tensor(i, tid, bf16_bits(rng.standard_normal(n) * 0.1))
+            m.load_tensor(i, L.T_SSM_NORM, bf16_bits(np.ones(inner)))
+        else:
+            for tid, n in ((L.T_Q, l["heads"] * l["dim"]), (L.T_K, l["kv_heads"] * l["dim"]), (L.T_V, l["kv_heads"] * l["vdim"]), (L.T_GATE_HEADS, l["heads"])):
+                m.load_tensor(i, tid, mat(n, W))
+            m.load_tensor(i, L.T_FF_GATE, mat(l["ff"], W)); m.load_tensor(i, L.T_FF_UP, mat(l["ff"], W)); m.load_tensor(i, L.T_FF_DOWN, mat(W, l["ff"]))
+    return m
+
+
+def stack_case(args, dev, synthetic, peak):
+    """Prefill and decode of the layer-by-layer decoder, beside the dense Q4_K decoder of the same width, heads, feed-forward,
+    vocabulary and number of layers.  --shape: prompt tokens."""
+    from doppler_b200.model import DecoderModel
+
+    n = int(args.shape) if args.shape else 1024
+    steps = args.steps
+    for size in ([args.size] if args.size else sorted(STACK_SIZES)):
+        z = STACK_SIZES[size]
+        for kind in ("fenorax", "dense_q4k"):
+            if kind == "fenorax":
+                m = stack_model(dev, size, n + 4 * steps + 64)
+            else:
+                m = DecoderModel(dev, dict(synthetic.MODEL_CONFIGS[z["dense"]], n_layers=4 * z["groups"]), n + 4 * steps + 64)
+                m.load_synthetic()
+            prompt = np.random.default_rng(5).integers(0, z["stack"]["vocab"], n).astype(np.int32)
+            tok = m.prefill(prompt)
+            sampler = ClockSampler(0)
+            pre = []
+            for _ in range(5):
+                m.reset(); dev.sync()
+                t0 = time.perf_counter()
+                tok = m.prefill(prompt)
+                pre.append((time.perf_counter() - t0) * 1e3)
+            tok = m.decode([tok], max(args.warmup, 3))[-1]
+            dec = []
+            for _ in range(3):
+                tok = m.decode(tok, steps)[-1]
+                dec.append(m.last_decode_ms / steps)
+            ms_p, ms_d = statistics.median(pre), statistics.median(dec)
+            line = {"case": "stack", "model": kind, "size": size, "layers": m.cfg["n_layers"], "width": z["stack"]["width"], "prompt_tokens": n,
+                    "prefill_ms": ms_p, "prefill_tokens_per_s": n / ms_p * 1e3, "decode_ms_per_step": ms_d, "decode_tokens_per_s": 1e3 / ms_d,
+                    "weight_bytes": m.weight_bytes, "decode_weight_GBps": m.weight_bytes / ms_d / 1e6,
+                    "decode_frac_of_measured_hbm": m.weight_bytes / ms_d / 1e6 / peak["hbm_gbs"], "peak_source": peak["source"], "clocks": sampler.stop(),
+                    "note": "prefill: host clock around the call, median of 5; decode: device time of graph launches, median of 3 regions; weights per step exceed L2"}
+            print(json.dumps(line), flush=True)
+            if args.kernel_trace:
+                barrier = dev.sync
+                kernel_trace(m, dev, tok, steps, f"{args.kernel_trace}.{size}.{kind}.decode", barrier, 1, 1)
+                prefill_trace(m, dev, prompt, f"{args.kernel_trace}.{size}.{kind}.prefill")
+            m.destroy()
+            dev.pool_trim()
+
+
 def kernel_case(args):
     from doppler_b200 import ops, synthetic
     dev = ops.Device(0)
@@ -357,6 +464,8 @@ def kernel_case(args):
         out_lines.append({"case": "prefill_9b", "prompt_tokens": n, "ms": dt * 1e3, "tokens_per_s": n / dt,
                           "q4k_gemm_TFLOPs_useful": layer_flops * cfg["n_layers"] / dt / 1e12})
         m.destroy()
+    elif args.case == "stack":
+        stack_case(args, dev, synthetic, peak)
     else:
         B, kv = tuple(int(v) for v in args.shape.split(",")) if args.shape else (32, 8192)
         out_lines.append(attention_case(dev, ops, synthetic, B, kv, max(args.steps // 2, 5), peak))
@@ -381,6 +490,22 @@ def kernel_trace(model, dev, tokens, steps, path, barrier, world, batch):
     barrier()
     if path is None:
         return
+    write_trace(prof, path, f"# decode step kernels, rank 0 of {world}, batch {batch}, {steps} steps traced (CUPTI activity records)", steps,
+                f"wall time of the traced region per step: {model.last_decode_ms * 1000.0 / steps:.1f} us")
+
+
+def prefill_trace(model, dev, prompt, path):
+    from torch.profiler import ProfilerActivity, profile
+
+    model.reset()
+    dev.sync()
+    with profile(activities=[ProfilerActivity.CUDA]) as prof:
+        model.prefill(prompt)
+        dev.sync()
+    write_trace(prof, path, f"# prefill kernels, {len(prompt)} tokens (CUPTI activity records)", 1, "")
+
+
+def write_trace(prof, path, title, steps, note):
     rows = []
     for e in prof.key_averages():
         t = float(getattr(e, "device_time_total", 0.0) or getattr(e, "cuda_time_total", 0.0) or 0.0)
@@ -389,8 +514,8 @@ def kernel_trace(model, dev, tokens, steps, path, barrier, world, batch):
     rows.sort(reverse=True)
     total = sum(r[0] for r in rows) or 1.0
     with open(path, "w") as f:
-        f.write(f"# decode step kernels, rank 0 of {world}, batch {batch}, {steps} steps traced (CUPTI activity records)\n")
-        f.write(f"# device time in kernels per step: {total / steps:.1f} us; wall time of the traced region per step: {model.last_decode_ms * 1000.0 / steps:.1f} us\n")
+        f.write(title + "\n")
+        f.write(f"# device time in kernels per step: {total / steps:.1f} us; {note}\n")
         f.write("share_pct\ttotal_us\tlaunches\tavg_us\tkernel\n")
         for t, c, k in rows:
             f.write(f"{100.0 * t / total:.1f}\t{t:.0f}\t{c}\t{t / max(c, 1):.2f}\t{k[:160]}\n")
@@ -407,13 +532,15 @@ def main():
     ap.add_argument("--workload", default="9b", choices=sorted(WORKLOADS))
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-kernels", action="store_true", help="skip the config 0/1/2 kernel record")
-    ap.add_argument("--case", default=None, choices=["gemv", "gemm", "attention", "prefill", "lm_head"],
+    ap.add_argument("--case", default=None, choices=["gemv", "gemm", "attention", "prefill", "lm_head", "stack"],
                     help="time ONE kernel of the path on a BASELINE configuration instead of the decoder "
-                         "(gemv: configs 0 and 9B shapes, gemm: config 1, attention: config 2); also the small "
+                         "(gemv: configs 0 and 9B shapes, gemm: config 1, attention: config 2; stack: prefill and decode of a "
+                         "Fenorax decoder beside the dense one); also the small "
                          "command the profiler captures use")
     ap.add_argument("--shape", default=None, help="--case gemv/gemm: N,K or M,N,K; --case attention: batch,kv_len")
     ap.add_argument("--variant", default="default", choices=["default", "f16_weights"], help="--case gemm: exact product or f16-rounded weights")
     ap.add_argument("--adtype", default="f16", choices=["f16", "f32"], help="--case gemm: activation (and output) dtype")
+    ap.add_argument("--size", default=None, choices=sorted(STACK_SIZES), help="--case stack: one layer size only")
     ap.add_argument("--copies", type=int, default=0, help="--case: distinct weight copies per pass (0 = enough to exceed L2)")
     ap.add_argument("--only-timed", action="store_true",
                     help="stop after the first device-resident timed region (used for profiler launch lists)")

@@ -12,8 +12,8 @@
 //   ATTN     merge of the split-K attention partials, times the per-head output gate
 //   STREAMS  x_t <- sum_s mix[s][t] x_s + out[t] y for the warp's rows, and u = sum_t in[t] x_t of the next sublayer
 //   GLU      gated activation of a gate row and its up row
-// Before griddepcontrol.wait a warp asks for its first rows' weights in L2 (cp.async.bulk.prefetch), so the weight
-// stream runs while the previous kernel drains and while the prologue works.
+// Before griddepcontrol.wait a warp asks for the start of its first rows in L2 (cp.async.bulk.prefetch) and the part of
+// the input convolution that lies in the past is summed up, so both run while the previous kernel drains.
 #include "layers.h"
 #include "pdl.cuh"
 
@@ -36,9 +36,43 @@ __device__ __forceinline__ void gb_w4(const __nv_bfloat16 *p, float (&w)[4]) {  
   w[2] = __uint_as_float(r.y << 16); w[3] = __uint_as_float(r.y & 0xffff0000u);
 }
 
+// The part of the input convolution that does not depend on this token: past[c] = sum over the history, and the two
+// per-channel factors packed as a bf16 pair (norm weight, the convolution's last tap).  The history was written by
+// earlier steps, so this runs before griddepcontrol.wait.
+__device__ __forceinline__ void gb_conv_past(const GemvBf16 &p, float *past, uint32_t *fac) {
+  const int taps = p.norm.taps, K = p.K, pos = *p.pos;
+  const uint16_t *nw = reinterpret_cast<const uint16_t *>(p.norm.norm_w), *cw = reinterpret_cast<const uint16_t *>(p.norm.conv_w);
+  if ((K & 3) == 0 && taps == 4) {
+    const float *h1 = p.norm.hist + (size_t)((pos + 3) & 3) * K, *h2 = p.norm.hist + (size_t)((pos + 2) & 3) * K, *h3 = p.norm.hist + (size_t)((pos + 1) & 3) * K;
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 2
+    for (int c = threadIdx.x * 4; c < K; c += GB_THREADS * 4) {
+      const float4 a1 = pos >= 1 ? gb_ld4(h1 + c) : zero, a2 = pos >= 2 ? gb_ld4(h2 + c) : zero, a3 = pos >= 3 ? gb_ld4(h3 + c) : zero;
+      const uint4 w01 = __ldg(reinterpret_cast<const uint4 *>(cw + (size_t)c * 4)), w23 = __ldg(reinterpret_cast<const uint4 *>(cw + (size_t)c * 4) + 1);
+      const uint2 n = __ldg(reinterpret_cast<const uint2 *>(nw + c));
+      const float q1[4] = {a1.x, a1.y, a1.z, a1.w}, q2[4] = {a2.x, a2.y, a2.z, a2.w}, q3[4] = {a3.x, a3.y, a3.z, a3.w};
+      const uint32_t lo[4] = {w01.x, w01.z, w23.x, w23.z}, hi[4] = {w01.y, w01.w, w23.y, w23.w};  // taps 0, 1 and taps 2, 3 of a channel
+      const uint32_t nn[4] = {n.x & 0xffffu, n.x >> 16, n.y & 0xffffu, n.y >> 16};
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        past[c + i] = fmaf(__uint_as_float(hi[i] << 16), q1[i], fmaf(__uint_as_float(lo[i] & 0xffff0000u), q2[i], __uint_as_float(lo[i] << 16) * q3[i]));
+        fac[c + i] = nn[i] | (hi[i] & 0xffff0000u);
+      }
+    }
+    return;
+  }
+  for (int c = threadIdx.x; c < K; c += GB_THREADS) {
+    float acc = 0.0f;
+    for (int k = taps - 1; k > 0; k--)
+      if (pos - k >= 0) acc = fmaf(__bfloat162float(p.norm.conv_w[(size_t)c * taps + taps - 1 - k]), p.norm.hist[(size_t)((pos - k) % taps) * K + c], acc);
+    past[c] = acc;
+    fac[c] = (uint32_t)nw[c] | (uint32_t)cw[(size_t)c * taps + taps - 1] << 16;
+  }
+}
+
 // x (in shared memory) = input convolution of the grouped RMSNorm of p.x.  Every warp owns whole groups or an equal
 // part of one, so the scale of its channels is one number.
-__device__ __forceinline__ void gb_prologue_norm(const GemvBf16 &p, float *sx, int plane, float *red) {
+__device__ __forceinline__ void gb_prologue_norm(const GemvBf16 &p, float *sx, int plane, float *red, const float *past, const uint32_t *fac) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int groups = p.norm.groups, gs = p.K / groups, taps = p.norm.taps;
   const int parts = groups >= GB_WARPS ? 1 : GB_WARPS / groups;
@@ -46,12 +80,15 @@ __device__ __forceinline__ void gb_prologue_norm(const GemvBf16 &p, float *sx, i
   const int unit = vec ? 4 : 1;
   const int part_len = ((gs / unit + parts - 1) / parts) * unit;
   const int tasks = groups * parts;
+  const bool keep = taps > 1 && blockIdx.x == 0;
+  float *slot = keep ? p.norm.hist + (size_t)(*p.pos % taps) * p.K : nullptr;
   for (int base = 0; base < tasks; base += GB_WARPS) {
     const int task = base + warp;
     const int g = task / parts, c_lo = g * gs + (task - g * parts) * part_len, c_hi = min(c_lo + part_len, (g + 1) * gs);
     float ss = 0.0f;
     if (task < tasks) {
       if (vec) {
+#pragma unroll 4
         for (int c = c_lo + lane * 4; c < c_hi; c += 128) {
           const float4 v = gb_ld4(p.x + c);
           *reinterpret_cast<float4 *>(sx + gb_slot(c, plane)) = v;
@@ -73,77 +110,76 @@ __device__ __forceinline__ void gb_prologue_norm(const GemvBf16 &p, float *sx, i
       float total = 0.0f;
       for (int i = 0; i < parts; i++) total += red[(warp / parts) * parts + i];
       const float inv = 1.0f / sqrtf(total / (float)gs + p.norm.eps);
-      const int pos = taps > 0 ? *p.pos : 0;
-      const bool keep = taps > 1 && blockIdx.x == 0;
-      if (vec && taps <= 4) {
-        for (int c = c_lo + lane * 4; c < c_hi; c += 128) {
-          float4 v = *reinterpret_cast<float4 *>(sx + gb_slot(c, plane));
-          float w[4];
+      for (int c = c_lo + lane * unit; c < c_hi; c += 32 * unit) {
+        float v[4], w[4];
+        if (vec) {
+          const float4 q = *reinterpret_cast<float4 *>(sx + gb_slot(c, plane));
+          v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+        } else v[0] = sx[gb_slot(c, plane)];
+        if (taps > 0) {
+#pragma unroll
+          for (int i = 0; i < 4; i++)
+            if (i < unit) {
+              const uint32_t f = fac[c + i];
+              const float h = v[i] * inv * __uint_as_float(f << 16);
+              if (keep) slot[c + i] = h;
+              v[i] = h + fmaf(__uint_as_float(f & 0xffff0000u), h, past[c + i]);
+            }
+        } else if (vec) {
           gb_w4(p.norm.norm_w + c, w);
-          float h[4] = {v.x * inv * w[0], v.y * inv * w[1], v.z * inv * w[2], v.w * inv * w[3]};
-          float o[4] = {h[0], h[1], h[2], h[3]};
-          if (taps > 0) {
-            float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            const __nv_bfloat16 *cw = p.norm.conv_w + (size_t)c * taps;
 #pragma unroll
-            for (int k = 3; k > 0; k--) {
-              if (k < taps) {
-                float4 past = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                if (pos - k >= 0) past = gb_ld4(p.norm.hist + (size_t)((pos - k) % taps) * p.K + c);
-                const int j = taps - 1 - k;
-                acc[0] = fmaf(__bfloat162float(cw[j]), past.x, acc[0]);
-                acc[1] = fmaf(__bfloat162float(cw[taps + j]), past.y, acc[1]);
-                acc[2] = fmaf(__bfloat162float(cw[2 * taps + j]), past.z, acc[2]);
-                acc[3] = fmaf(__bfloat162float(cw[3 * taps + j]), past.w, acc[3]);
-              }
-            }
-#pragma unroll
-            for (int i = 0; i < 4; i++) o[i] = h[i] + fmaf(__bfloat162float(cw[i * taps + taps - 1]), h[i], acc[i]);
-            if (keep) *reinterpret_cast<float4 *>(p.norm.hist + (size_t)(pos % taps) * p.K + c) = make_float4(h[0], h[1], h[2], h[3]);
-          }
-          *reinterpret_cast<float4 *>(sx + gb_slot(c, plane)) = make_float4(o[0], o[1], o[2], o[3]);
-        }
-      } else {
-        for (int c = c_lo + lane * unit; c < c_hi; c += 32 * unit)
-          for (int i = 0; i < unit; i++) {
-            const float h = sx[gb_slot(c + i, plane)] * inv * __bfloat162float(p.norm.norm_w[c + i]);
-            float o = h;
-            if (taps > 0) {
-              const __nv_bfloat16 *cw = p.norm.conv_w + (size_t)(c + i) * taps;
-              float acc = 0.0f;
-              for (int k = taps - 1; k > 0; k--)
-                if (pos - k >= 0) acc = fmaf(__bfloat162float(cw[taps - 1 - k]), p.norm.hist[(size_t)((pos - k) % taps) * p.K + c + i], acc);
-              o = h + fmaf(__bfloat162float(cw[taps - 1]), h, acc);
-              if (keep) p.norm.hist[(size_t)(pos % taps) * p.K + c + i] = h;
-            }
-            sx[gb_slot(c + i, plane)] = o;
-          }
+          for (int i = 0; i < 4; i++) v[i] = v[i] * inv * w[i];
+        } else v[0] = v[0] * inv * __bfloat162float(p.norm.norm_w[c]);
+        if (vec) *reinterpret_cast<float4 *>(sx + gb_slot(c, plane)) = make_float4(v[0], v[1], v[2], v[3]);
+        else sx[gb_slot(c, plane)] = v[0];
       }
     }
-    __syncthreads();  // red is reused
+    if (base + GB_WARPS < tasks) __syncthreads();  // red is reused
   }
 }
 
-// x = attention output of one row, merged from its split partials, times the head's gate
-__device__ __forceinline__ void gb_prologue_attn(const GemvBf16 &p, float *sx, int plane, float *red) {
-  (void)red;
-  const int tid = threadIdx.x, V = p.vdim, S = p.splits;
-  for (int e = tid; e < p.K; e += GB_THREADS) {
-    const int h = e / V, d = e - h * V;
-    const float *pp = p.x + (size_t)h * S * (V + 2);
-    float mm = -FLT_MAX;
-    for (int s = 0; s < S; s++) mm = fmaxf(mm, pp[s * (V + 2) + V]);
-    float ll = 0.0f, acc = 0.0f;
-#pragma unroll 4
-    for (int s = 0; s < S; s++) {
-      const float *ps = pp + s * (V + 2);
-      const float c = ps[V] == -FLT_MAX ? 0.0f : exp2f(ps[V] - mm);
-      ll = fmaf(ps[V + 1], c, ll);
-      acc = fmaf(ps[d], c, acc);
+// x = attention output of one row, merged from its split partials, times the head's gate.  wgt [head][split]: what a
+// split's partial counts for.
+__device__ __forceinline__ void gb_prologue_attn(const GemvBf16 &p, float *sx, int plane, float *wgt) {
+  const int tid = threadIdx.x, lane = tid & 31, V = p.vdim, S = p.splits, row = V + 2;
+  for (int h = tid >> 5; h < p.heads; h += GB_WARPS) {  // a warp per head, a lane per split (at most 32)
+    const float *pp = p.x + ((size_t)h * S + lane) * row + V;
+    const float m = lane < S ? pp[0] : -FLT_MAX, l = lane < S ? pp[1] : 0.0f;
+    const float g = p.gate ? p.gate[h] : 0.0f;
+    float mm = m;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, o));
+    const float c = m == -FLT_MAX ? 0.0f : exp2f(m - mm);
+    float ll = l * c;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ll += __shfl_xor_sync(0xffffffffu, ll, o);
+    float f = ll > 0.0f ? c / ll : 0.0f;
+    if (p.gate) f *= 1.0f / (1.0f + expf(-g));
+    if (lane < S) wgt[h * S + lane] = f;
+  }
+  __syncthreads();
+  if ((V & 1) == 0) {
+#pragma unroll 2
+    for (int e = 2 * tid; e < p.K; e += 2 * GB_THREADS) {
+      const int h = e / V;
+      const float *pp = p.x + (size_t)h * S * row + (e - h * V), *wh = wgt + h * S;
+      float a0 = 0.0f, a1 = 0.0f;
+#pragma unroll 8
+      for (int s = 0; s < S; s++) {
+        const float2 v = *reinterpret_cast<const float2 *>(pp + s * row);
+        a0 = fmaf(v.x, wh[s], a0);
+        a1 = fmaf(v.y, wh[s], a1);
+      }
+      *reinterpret_cast<float2 *>(sx + gb_slot(e, plane)) = make_float2(a0, a1);
     }
-    float v = ll > 0.0f ? acc / ll : 0.0f;
-    if (p.gate) v *= 1.0f / (1.0f + expf(-p.gate[h]));
-    sx[gb_slot(e, plane)] = v;
+  } else {
+    for (int e = tid; e < p.K; e += GB_THREADS) {
+      const int h = e / V;
+      const float *pp = p.x + (size_t)h * S * row + (e - h * V), *wh = wgt + h * S;
+      float acc = 0.0f;
+      for (int s = 0; s < S; s++) acc = fmaf(pp[s * row], wh[s], acc);
+      sx[gb_slot(e, plane)] = acc;
+    }
   }
 }
 
@@ -166,7 +202,6 @@ __device__ __forceinline__ uint4 gb_ldw(const uint4 *p) {
 
 template <int SRC, int DST>
 __global__ void __launch_bounds__(GB_THREADS, 2) gemv_bf16_kernel(const GemvBf16 p) {
-  pdl_launch();
   extern __shared__ __align__(16) float gb_sx[];
   __shared__ float red[GB_WARPS];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -177,19 +212,21 @@ __global__ void __launch_bounds__(GB_THREADS, 2) gemv_bf16_kernel(const GemvBf16
   const int pair0 = (int)blockIdx.x + (int)gridDim.x * warp, step = (int)gridDim.x * GB_WARPS;
   auto row_a = [&](int pr) { return DST == GEMV_DST_GLU ? ((pr >> 3) * 16 + (pr & 7)) : 2 * pr; };
   auto row_b = [&](int pr) { return DST == GEMV_DST_GLU ? row_a(pr) + 8 : (2 * pr + 1 < p.N ? 2 * pr + 1 : 2 * pr); };
-  {  // the weights are constant: ask for the first rows before the previous kernel has finished
-    const uint32_t row_bytes = (uint32_t)p.w_stride * 2u;
-    if (lane < 4) {
-      const int pr = pair0 + (lane >> 1) * step;
-      if (pr < pairs) gb_prefetch_l2(p.w + (size_t)((lane & 1) ? row_b(pr) : row_a(pr)) * p.w_stride, row_bytes);
-    }
+  float *extra = gb_sx + 2 * plane;  // behind the vector: what the prologue needs beside it
+  {  // the weights are constant: ask for the start of the first rows before the previous kernel has finished
+    const uint32_t row_bytes = min((uint32_t)p.w_stride * 2u, p.prefetch_bytes);
+    if (lane < 2 && pair0 < pairs && row_bytes) gb_prefetch_l2(p.w + (size_t)(lane ? row_b(pair0) : row_a(pair0)) * p.w_stride, row_bytes);
   }
-  pdl_wait();
   for (int k = p.K + tid; k < pieces * 8; k += GB_THREADS) gb_sx[gb_slot(k, plane)] = 0.0f;  // the padded tail
+  if constexpr (SRC == GEMV_SRC_NORM)
+    if (p.norm.taps > 0) gb_conv_past(p, extra, reinterpret_cast<uint32_t *>(extra) + p.K);
+  pdl_wait();
+  pdl_launch();  // not before the wait: the next kernel's early work then competes with this kernel's stream only
   if constexpr (SRC == GEMV_SRC_NORM) {
-    gb_prologue_norm(p, gb_sx, plane, red);
+    if (p.norm.taps > 0) __syncthreads();
+    gb_prologue_norm(p, gb_sx, plane, red, extra, reinterpret_cast<const uint32_t *>(extra) + p.K);
   } else if constexpr (SRC == GEMV_SRC_ATTN) {
-    gb_prologue_attn(p, gb_sx, plane, red);
+    gb_prologue_attn(p, gb_sx, plane, extra);
   } else {
     for (int k = tid; k < p.K; k += GB_THREADS) gb_sx[gb_slot(k, plane)] = p.x[k];
   }
@@ -255,7 +292,9 @@ __global__ void __launch_bounds__(GB_THREADS, 2) gemv_bf16_kernel(const GemvBf16
 
 template <int SRC, int DST>
 dp_status launch(dp_ctx *ctx, const GemvBf16 &p) {
-  const size_t smem = (size_t)(p.w_stride) * 4;
+  size_t smem = (size_t)p.w_stride * 4;
+  if (SRC == GEMV_SRC_NORM && p.norm.taps > 0) smem += (size_t)p.K * 8;
+  if (SRC == GEMV_SRC_ATTN) smem += (size_t)p.heads * p.splits * 4;
   if (smem > ctx->smem_optin - 1024)
     return dp_fail(ctx, DP_ERR_UNSUPPORTED, "gemv (bf16): a vector of %d values exceeds shared memory", p.K);
   static dp_per_device_once attr;

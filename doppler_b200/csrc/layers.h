@@ -74,6 +74,7 @@ struct GemvBf16 {
   float *streams_x = nullptr;
   const float *next_in = nullptr;
   float *next_u = nullptr;
+  uint32_t prefetch_bytes = 4096;  // per row, before the previous kernel has finished
 };
 dp_status dpk_gemv_bf16(dp_ctx *ctx, int src, int dst, const GemvBf16 &p);
 
@@ -116,8 +117,13 @@ struct SsmState {
 // proj [row][z | x | B | C | dt] of proj_stride floats -> out [row][heads * vdim]
 dp_status dpk_ssm_step(dp_ctx *ctx, const float *proj, int proj_stride, const SsmShape &sh, const SsmWeights &w, const SsmState &st, float *out, int rows,
                        const int *pos);
-// Consecutive tokens of one sequence.  xbc [rows][channels] and dt [rows][heads] are scratch.
-dp_status dpk_ssm_conv(dp_ctx *ctx, const float *proj, int proj_stride, const SsmShape &sh, const SsmWeights &w, const SsmState &st, float *xbc, float *dt,
-                       int rows, const RowMap &map);
+// Consecutive tokens of one sequence: the convolution (xbc [rows][channels], f32 or bf16) and step sizes (dt [rows][heads]),
+// then the recurrence, token by token in f32 (dpk_ssm_scan, any shape) or in chunks on the tensor cores with bf16 x, B
+// and C (dpk_ssm_chunk)
+dp_status dpk_ssm_conv(dp_ctx *ctx, const float *proj, int proj_stride, const SsmShape &sh, const SsmWeights &w, const SsmState &st, void *xbc, bool bf16,
+                       float *dt, int rows, const RowMap &map);
+bool dpk_ssm_chunk_ok(const SsmShape &sh, int rows);
+dp_status dpk_ssm_chunk(dp_ctx *ctx, const float *proj, int proj_stride, const __nv_bfloat16 *xbc, const float *dt, const SsmShape &sh, const SsmWeights &w,
+                        const SsmState &st, float *out, int rows, const RowMap &map);
 dp_status dpk_ssm_scan(dp_ctx *ctx, const float *proj, int proj_stride, const float *xbc, const float *dt, const SsmShape &sh, const SsmWeights &w,
                        const SsmState &st, float *out, int rows, const RowMap &map);

@@ -16,24 +16,14 @@ constexpr int SSM_COLS = 32, SSM_LANES = 8, SSM_THREADS = SSM_COLS * SSM_LANES;
 __device__ __forceinline__ float ssm_silu(float v) { return v / (1.0f + expf(-v)); }
 __device__ __forceinline__ float ssm_softplus(float v) { return fmaxf(v, 0.0f) + log1pf(expf(-fabsf(v))); }
 
-// convolution of channel ch of the token at `pos`, whose raw value is `cur`, over a sequence's history
-__device__ __forceinline__ float ssm_conv1(const SsmWeights &w, const float *hist, int taps, int CH, int ch, int pos, float cur) {
-  const float *cw = w.conv + (size_t)ch * taps;
-  float acc = w.conv_b[ch];
-  for (int k = taps - 1; k > 0; k--)
-    if (pos - k >= 0) acc = fmaf(cw[taps - 1 - k], hist[(size_t)((pos - k) % taps) * CH + ch], acc);
-  return ssm_silu(fmaf(cw[taps - 1], cur, acc));
-}
-
 // ---- one token per row, rows are sequences: grid (heads, column tiles, rows) ----
+// What earlier steps left (state, convolution histories, positions) is read before griddepcontrol.wait; after it only
+// this token's projections are.
 template <int NV>
 __global__ void __launch_bounds__(SSM_THREADS) ssm_step_kernel(const float *__restrict__ proj, int proj_stride, const SsmShape sh, const SsmWeights w,
                                                                const SsmState st, float *__restrict__ out, const int *__restrict__ pos_arr) {
-  pdl_launch();
-  pdl_wait();
-  constexpr int NP = NV * 32;
-  __shared__ __align__(16) float sB[NP], sC[NP], sx[SSM_COLS];
-  __shared__ float s_dt;
+  constexpr int NP = NV * 32, CHANNELS = 2 * NP + SSM_COLS, PER = (CHANNELS + SSM_THREADS - 1) / SSM_THREADS;
+  __shared__ __align__(16) float sv[CHANNELS];  // B, C, x
   const int tid = threadIdx.x, h = blockIdx.x, p0 = blockIdx.y * SSM_COLS, row = blockIdx.z;
   const int P = sh.vdim, N = sh.state, G = sh.groups, inner = sh.heads * P, CH = inner + 2 * G * N, taps = sh.taps;
   const int per = sh.heads / G, g = h / per;
@@ -43,40 +33,59 @@ __global__ void __launch_bounds__(SSM_THREADS) ssm_step_kernel(const float *__re
   float *hist = st.hist + (size_t)row * st.hist_seq;
   float *slot = hist + (size_t)(pos % taps) * CH;
   const int cols = min(SSM_COLS, P - p0);
-  const bool keep_bc = taps > 1 && blockIdx.y == 0 && h == g * per;  // one head of the group appends its B and C
-  // the state's first pieces are asked for while the convolution works
+  const bool keep_bc = blockIdx.y == 0 && h == g * per;  // one head of the group appends its B and C
   const int col = tid / SSM_LANES, sub = tid % SSM_LANES;
   float4 *S = reinterpret_cast<float4 *>(st.s + (size_t)row * st.s_seq + ((size_t)h * P + p0 + col) * NP) + sub;
   float4 v[NV];
 #pragma unroll
   for (int i = 0; i < NV; i++) v[i] = (col < cols && pos > 0) ? S[8 * i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-  for (int i = tid; i < 2 * NP + cols; i += SSM_THREADS) {
+  // this thread's channels of the convolution: what the history and the bias contribute
+  float acc[PER], last[PER];
+  int chan[PER];
+#pragma unroll
+  for (int j = 0; j < PER; j++) {
+    const int i = tid + j * SSM_THREADS;
+    int ch = -1;
     if (i < 2 * NP) {
-      const bool is_c = i >= NP;
-      const int n = is_c ? i - NP : i;
-      float val = 0.0f;
-      if (n < N) {
-        const int ch = inner + (is_c ? G * N : 0) + g * N + n;
-        const float cur = raw[ch];
-        val = ssm_conv1(w, hist, taps, CH, ch, pos, cur);
-        if (keep_bc) slot[ch] = cur;
-      }
-      (is_c ? sC : sB)[n] = val;
-    } else {
-      const int c = i - 2 * NP, ch = h * P + p0 + c;
-      const float cur = raw[ch];
-      sx[c] = ssm_conv1(w, hist, taps, CH, ch, pos, cur);
-      if (taps > 1) slot[ch] = cur;
+      const int n = i < NP ? i : i - NP;
+      if (n < N) ch = inner + (i < NP ? g : G + g) * N + n;
+    } else if (i < 2 * NP + cols) ch = h * P + p0 + i - 2 * NP;
+    chan[j] = ch;
+    acc[j] = last[j] = 0.0f;
+    if (ch >= 0) {
+      const float *cw = w.conv + (size_t)ch * taps;
+      acc[j] = w.conv_b[ch];
+      last[j] = cw[taps - 1];
+      for (int k = taps - 1; k > 0; k--)
+        if (pos - k >= 0) acc[j] = fmaf(cw[taps - 1 - k], hist[(size_t)((pos - k) % taps) * CH + ch], acc[j]);
     }
   }
-  if (tid == 0) s_dt = ssm_softplus(pr[inner + CH + h] + w.dt_bias[h]);
+  const float a = -expf(w.a_log[h]), dt_bias = w.dt_bias[h], dh = w.d[h];
+  pdl_wait();
+  pdl_launch();
+  const float dt_raw = pr[inner + CH + h];
+  const int e = h * P + p0 + col;
+  const float z = sub == 0 && col < cols ? pr[e] : 0.0f;
+#pragma unroll
+  for (int j = 0; j < PER; j++) {
+    const int i = tid + j * SSM_THREADS;
+    if (i < CHANNELS) {
+      float val = 0.0f;
+      if (chan[j] >= 0) {
+        const float cur = raw[chan[j]];
+        val = ssm_silu(fmaf(last[j], cur, acc[j]));
+        if (taps > 1 && (i >= 2 * NP || keep_bc)) slot[chan[j]] = cur;
+      }
+      sv[i] = val;
+    }
+  }
+  const float dt = ssm_softplus(dt_raw + dt_bias), decay = expf(a * dt);
   __syncthreads();
-  const float dt = s_dt, decay = expf(-expf(w.a_log[h]) * dt);
-  const float x = col < cols ? sx[col] : 0.0f, xdt = dt * x;
+  const float x = sv[2 * NP + col], xdt = dt * x;
   float y = 0.0f;
 #pragma unroll
   for (int i = 0; i < NV; i++) {
-    const float4 b = *reinterpret_cast<const float4 *>(sB + sub * 4 + 32 * i), c = *reinterpret_cast<const float4 *>(sC + sub * 4 + 32 * i);
+    const float4 b = *reinterpret_cast<const float4 *>(sv + sub * 4 + 32 * i), c = *reinterpret_cast<const float4 *>(sv + NP + sub * 4 + 32 * i);
     v[i].x = fmaf(decay, v[i].x, xdt * b.x); v[i].y = fmaf(decay, v[i].y, xdt * b.y);
     v[i].z = fmaf(decay, v[i].z, xdt * b.z); v[i].w = fmaf(decay, v[i].w, xdt * b.w);
     y = fmaf(v[i].x, c.x, fmaf(v[i].y, c.y, fmaf(v[i].z, c.z, fmaf(v[i].w, c.w, y))));
@@ -84,26 +93,81 @@ __global__ void __launch_bounds__(SSM_THREADS) ssm_step_kernel(const float *__re
   }
 #pragma unroll
   for (int o = 4; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-  if (sub == 0 && col < cols) {
-    const int e = h * P + p0 + col;
-    out[(size_t)row * inner + e] = fmaf(w.d[h], x, y) * ssm_silu(pr[e]);
-  }
+  if (sub == 0 && col < cols) out[(size_t)row * inner + e] = fmaf(dh, x, y) * ssm_silu(z);
 }
 
 // ---- several tokens of one sequence: convolution and step sizes ----
 constexpr int CONV_ROWS = 16;
-template <int TAPS>  // 0: any
-__global__ void __launch_bounds__(128) ssm_conv_kernel(const float *__restrict__ proj, int proj_stride, const SsmShape sh, const SsmWeights w, const SsmState st,
-                                                       float *__restrict__ xbc, float *__restrict__ dt, int rows, int start_pos, int seq) {
+__device__ __forceinline__ void conv_store(float *p, float v) { *p = v; }
+__device__ __forceinline__ void conv_store(__nv_bfloat16 *p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ void conv_store4(float *p, const float (&v)[4]) { *reinterpret_cast<float4 *>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void conv_store4(__nv_bfloat16 *p, const float (&v)[4]) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+  *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+}
+
+// an activation that is stored as bf16 needs no exact division
+template <typename OutT> __device__ __forceinline__ float conv_silu(float v) {
+  if constexpr (sizeof(OutT) == 2) return __fdividef(v, 1.0f + __expf(-v));
+  else return ssm_silu(v);
+}
+
+// step size of one (row, head)
+__device__ __forceinline__ void conv_dt(const float *proj, int proj_stride, const SsmShape &sh, const SsmWeights &w, int col0, int h, float *dt, int r0, int r1) {
+  for (int r = r0; r < r1; r++) dt[(size_t)r * sh.heads + h] = ssm_softplus(proj[(size_t)r * proj_stride + col0 + h] + w.dt_bias[h]);
+}
+
+// four taps, four neighbouring channels per thread (channel counts and row strides that are multiples of four)
+template <typename OutT>
+__global__ void __launch_bounds__(128) ssm_conv4_kernel(const float *__restrict__ proj, int proj_stride, const SsmShape sh, const SsmWeights w, const SsmState st,
+                                                        OutT *__restrict__ xbc, float *__restrict__ dt, int rows, int start_pos, int seq) {
   pdl_launch();
   pdl_wait();
-  const int inner = sh.heads * sh.vdim, CH = inner + 2 * sh.groups * sh.state, taps = TAPS ? TAPS : sh.taps;
+  const int inner = sh.heads * sh.vdim, CH = inner + 2 * sh.groups * sh.state;
+  const int idx = blockIdx.x * 128 + threadIdx.x, ch = idx * 4;
+  const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, rows);
+  if (ch >= CH) {
+    const int h = idx - CH / 4;
+    if (h < sh.heads) conv_dt(proj, proj_stride, sh, w, inner + CH, h, dt, r0, r1);
+    return;
+  }
+  const float *col = proj + inner + ch;
+  const float *hist = st.hist + (size_t)seq * st.hist_seq;
+  auto raw = [&](int r) -> float4 {
+    if (r >= 0) return *reinterpret_cast<const float4 *>(col + (size_t)r * proj_stride);
+    const int p = start_pos + r;
+    return p >= 0 ? *reinterpret_cast<const float4 *>(hist + (size_t)(p & 3) * CH + ch) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  };
+  float4 wv[4];  // the four taps of each channel
+#pragma unroll
+  for (int i = 0; i < 4; i++) wv[i] = *reinterpret_cast<const float4 *>(w.conv + (size_t)(ch + i) * 4);
+  const float4 bias = *reinterpret_cast<const float4 *>(w.conv_b + ch);
+  float4 a = raw(r0 - 3), b = raw(r0 - 2), c = raw(r0 - 1);
+#pragma unroll 8
+  for (int r = r0; r < r1; r++) {
+    const float4 d = *reinterpret_cast<const float4 *>(col + (size_t)r * proj_stride);
+    float o[4];
+    o[0] = conv_silu<OutT>(fmaf(wv[0].w, d.x, fmaf(wv[0].z, c.x, fmaf(wv[0].y, b.x, fmaf(wv[0].x, a.x, bias.x)))));
+    o[1] = conv_silu<OutT>(fmaf(wv[1].w, d.y, fmaf(wv[1].z, c.y, fmaf(wv[1].y, b.y, fmaf(wv[1].x, a.y, bias.y)))));
+    o[2] = conv_silu<OutT>(fmaf(wv[2].w, d.z, fmaf(wv[2].z, c.z, fmaf(wv[2].y, b.z, fmaf(wv[2].x, a.z, bias.z)))));
+    o[3] = conv_silu<OutT>(fmaf(wv[3].w, d.w, fmaf(wv[3].z, c.w, fmaf(wv[3].y, b.w, fmaf(wv[3].x, a.w, bias.w)))));
+    conv_store4(xbc + (size_t)r * CH + ch, o);
+    a = b; b = c; c = d;
+    if (r >= rows - 3) *reinterpret_cast<float4 *>(st.stage + (size_t)((start_pos + r) & 3) * CH + ch) = d;
+  }
+}
+
+// any number of taps and channels
+template <typename OutT>
+__global__ void __launch_bounds__(128) ssm_conv_kernel(const float *__restrict__ proj, int proj_stride, const SsmShape sh, const SsmWeights w, const SsmState st,
+                                                       OutT *__restrict__ xbc, float *__restrict__ dt, int rows, int start_pos, int seq) {
+  pdl_launch();
+  pdl_wait();
+  const int inner = sh.heads * sh.vdim, CH = inner + 2 * sh.groups * sh.state, taps = sh.taps;
   const int ch = blockIdx.x * 128 + threadIdx.x;
   const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, rows);
-  if (ch >= CH + sh.heads) return;
   if (ch >= CH) {
-    const int h = ch - CH;
-    for (int r = r0; r < r1; r++) dt[(size_t)r * sh.heads + h] = ssm_softplus(proj[(size_t)r * proj_stride + inner + ch] + w.dt_bias[h]);
+    if (ch < CH + sh.heads) conv_dt(proj, proj_stride, sh, w, inner + CH, ch - CH, dt, r0, r1);
     return;
   }
   const float *col = proj + inner + ch;
@@ -114,32 +178,12 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const float *__restrict__
     return p >= 0 ? hist[(size_t)(p % taps) * CH + ch] : 0.0f;
   };
   const float *cw = w.conv + (size_t)ch * taps;
-  const float bias = w.conv_b[ch];
-  if constexpr (TAPS > 0) {
-    float win[TAPS], wv[TAPS];
-#pragma unroll
-    for (int j = 0; j < TAPS; j++) wv[j] = cw[j];
-#pragma unroll
-    for (int j = 0; j < TAPS - 1; j++) win[j + 1] = raw(r0 - (TAPS - 1) + j);
-#pragma unroll 4
-    for (int r = r0; r < r1; r++) {
-#pragma unroll
-      for (int j = 0; j < TAPS - 1; j++) win[j] = win[j + 1];
-      win[TAPS - 1] = col[(size_t)r * proj_stride];
-      float acc = bias;
-#pragma unroll
-      for (int j = 0; j < TAPS; j++) acc = fmaf(wv[j], win[j], acc);
-      xbc[(size_t)r * CH + ch] = ssm_silu(acc);
-    }
-  } else {
-    for (int r = r0; r < r1; r++) {
-      float acc = bias;
-      for (int j = 0; j < taps; j++) acc = fmaf(cw[j], raw(r - (taps - 1) + j), acc);
-      xbc[(size_t)r * CH + ch] = ssm_silu(acc);
-    }
+  for (int r = r0; r < r1; r++) {
+    float acc = w.conv_b[ch];
+    for (int j = 0; j < taps; j++) acc = fmaf(cw[j], raw(r - (taps - 1) + j), acc);
+    conv_store(xbc + (size_t)r * CH + ch, conv_silu<OutT>(acc));
+    if (r >= rows - (taps - 1)) st.stage[(size_t)((start_pos + r) % taps) * CH + ch] = raw(r);
   }
-  if (taps > 1)
-    for (int r = max(r0, rows - (taps - 1)); r < r1; r++) st.stage[(size_t)((start_pos + r) % taps) * CH + ch] = col[(size_t)r * proj_stride];
 }
 
 // ---- several tokens of one sequence, token by token: grid (heads, column tiles) ----
@@ -260,12 +304,16 @@ dp_status dpk_ssm_step(dp_ctx *ctx, const float *proj, int proj_stride, const Ss
   return DP_OK;
 }
 
-dp_status dpk_ssm_conv(dp_ctx *ctx, const float *proj, int proj_stride, const SsmShape &sh, const SsmWeights &w, const SsmState &st, float *xbc, float *dt,
-                       int rows, const RowMap &map) {
-  const int cols = sh.heads * sh.vdim + 2 * sh.groups * sh.state + sh.heads;
-  const dim3 grid((cols + 127) / 128, (rows + CONV_ROWS - 1) / CONV_ROWS);
-  if (sh.taps == 4) DP_LAUNCH(ctx, ssm_conv_kernel<4>, grid, 128, 0, proj, proj_stride, sh, w, st, xbc, dt, rows, map.start_pos, map.seq);
-  else DP_LAUNCH(ctx, ssm_conv_kernel<0>, grid, 128, 0, proj, proj_stride, sh, w, st, xbc, dt, rows, map.start_pos, map.seq);
+dp_status dpk_ssm_conv(dp_ctx *ctx, const float *proj, int proj_stride, const SsmShape &sh, const SsmWeights &w, const SsmState &st, void *xbc, bool bf16,
+                       float *dt, int rows, const RowMap &map) {
+  const int inner = sh.heads * sh.vdim, CH = inner + 2 * sh.groups * sh.state;
+  const bool four = sh.taps == 4 && CH % 4 == 0 && inner % 4 == 0 && proj_stride % 4 == 0;
+  const int threads = (four ? CH / 4 : CH) + sh.heads;
+  const dim3 grid((threads + 127) / 128, (rows + CONV_ROWS - 1) / CONV_ROWS);
+#define DP_CONV(K, T) DP_LAUNCH(ctx, K<T>, grid, 128, 0, proj, proj_stride, sh, w, st, (T *)xbc, dt, rows, map.start_pos, map.seq)
+  if (four) { if (bf16) DP_CONV(ssm_conv4_kernel, __nv_bfloat16); else DP_CONV(ssm_conv4_kernel, float); }
+  else { if (bf16) DP_CONV(ssm_conv_kernel, __nv_bfloat16); else DP_CONV(ssm_conv_kernel, float); }
+#undef DP_CONV
   return DP_OK;
 }
 

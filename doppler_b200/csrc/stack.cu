@@ -328,8 +328,12 @@ dp_status run_rows(dp_model *m, int rows, bool decode, int seq, int start_pos) {
       if (decode) {
         DP_TRY(dpk_ssm_step(ctx, s->proj, L.proj.N, L.ssm, ssm_weights(L), L.st, s->mix, rows, m->d_pos));
       } else {
-        DP_TRY(dpk_ssm_conv(ctx, s->proj, L.proj.N, L.ssm, ssm_weights(L), L.st, s->xbc, s->dt, rows, map));
-        DP_TRY(dpk_ssm_scan(ctx, s->proj, L.proj.N, s->xbc, s->dt, L.ssm, ssm_weights(L), L.st, s->mix, rows, map));
+        const bool chunks = !s->f32 && dpk_ssm_chunk_ok(L.ssm, rows);
+        DP_TRY(dpk_ssm_conv(ctx, s->proj, L.proj.N, L.ssm, ssm_weights(L), L.st, s->xbc, chunks, s->dt, rows, map));
+        if (chunks)
+          DP_TRY(dpk_ssm_chunk(ctx, s->proj, L.proj.N, (const __nv_bfloat16 *)s->xbc, s->dt, L.ssm, ssm_weights(L), L.st, s->mix, rows, map));
+        else
+          DP_TRY(dpk_ssm_scan(ctx, s->proj, L.proj.N, s->xbc, s->dt, L.ssm, ssm_weights(L), L.st, s->mix, rows, map));
       }
       DP_TRY(dpk_group_norm(ctx, s->mix, L.inner(), L.ssm_norm, L.c.norm_groups, s->cfg.eps, L.inner(), s->a, !s->f32, ks, rows));
     }

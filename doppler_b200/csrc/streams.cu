@@ -12,7 +12,7 @@
 
 namespace {
 
-constexpr int SB_THREADS = 256, SB_WARPS = SB_THREADS / 32;
+constexpr int SB_THREADS = 288, SB_WARPS = SB_THREADS / 32;
 
 template <int V> struct FV { float v[V]; };
 template <int V> __device__ __forceinline__ FV<V> ldv(const float *p) {
@@ -33,6 +33,12 @@ template <int V> __device__ __forceinline__ void stv(__nv_bfloat16 *p, const FV<
 }
 template <int V> __device__ __forceinline__ FV<V> ldw(const __nv_bfloat16 *p) {
   FV<V> r;
+  if constexpr (V == 4) {
+    const uint2 q = *reinterpret_cast<const uint2 *>(p);
+    r.v[0] = __uint_as_float(q.x << 16); r.v[1] = __uint_as_float(q.x & 0xffff0000u);
+    r.v[2] = __uint_as_float(q.y << 16); r.v[3] = __uint_as_float(q.y & 0xffff0000u);
+    return r;
+  }
 #pragma unroll
   for (int i = 0; i < V; i++) r.v[i] = __bfloat162float(p[i]);
   return r;
@@ -48,7 +54,7 @@ struct BoundaryArgs {
 };
 
 template <int SM, int V, typename OutT>
-__global__ void __launch_bounds__(SB_THREADS) stream_boundary_kernel(const BoundaryArgs a, OutT *__restrict__ dst) {
+__global__ void __launch_bounds__(SB_THREADS, 2) stream_boundary_kernel(const BoundaryArgs a, OutT *__restrict__ dst) {
   pdl_launch();
   pdl_wait();
   extern __shared__ float sb_h[];  // [halo + block_rows][gs]
@@ -69,6 +75,19 @@ __global__ void __launch_bounds__(SB_THREADS) stream_boundary_kernel(const Bound
   }
   __syncthreads();
 
+  // few streams: the mixing weights in registers
+  constexpr bool REG = SM <= 4;
+  float r_mix[REG ? SM * SM : 1], r_out[REG ? SM : 1], r_in[REG ? SM : 1];
+  if constexpr (REG) {
+#pragma unroll
+    for (int i = 0; i < SM * SM; i++) r_mix[i] = s_mix[i];
+#pragma unroll
+    for (int i = 0; i < SM; i++) { r_out[i] = s_out[i]; r_in[i] = s_in[i]; }
+  }
+  auto mix = [&](int s, int t) { if constexpr (REG) return r_mix[s * SM + t]; else return s_mix[s * SM + t]; };
+  auto wout = [&](int t) { if constexpr (REG) return r_out[t]; else return s_out[t]; };
+  auto win = [&](int t) { if constexpr (REG) return r_in[t]; else return s_in[t]; };
+
   // ---- h of the block's rows and of the rows the convolution reaches back to: one warp per row ----
   for (int j = warp; j < halo + nrows; j += SB_WARPS) {
     const int row = row0 + j - halo;
@@ -83,6 +102,7 @@ __global__ void __launch_bounds__(SB_THREADS) stream_boundary_kernel(const Bound
     float *xo = a.x_out + (size_t)row * S * H + c0;
     const bool store = a.y && j >= halo;
     float ss = 0.0f;
+#pragma unroll(SM <= 4 ? 2 : 1)
     for (int c = lane * V; c < gs; c += 32 * V) {
       FV<V> xs[SM], u;
 #pragma unroll
@@ -97,15 +117,15 @@ __global__ void __launch_bounds__(SB_THREADS) stream_boundary_kernel(const Bound
           if (t < S) {
             FV<V> n;
 #pragma unroll
-            for (int i = 0; i < V; i++) n.v[i] = s_out[t] * yv.v[i];
+            for (int i = 0; i < V; i++) n.v[i] = wout(t) * yv.v[i];
 #pragma unroll
             for (int s = 0; s < SM; s++)
               if (s < S)
 #pragma unroll
-                for (int i = 0; i < V; i++) n.v[i] = fmaf(s_mix[s * SM + t], xs[s].v[i], n.v[i]);
+                for (int i = 0; i < V; i++) n.v[i] = fmaf(mix(s, t), xs[s].v[i], n.v[i]);
             if (store) stv<V>(xo + (size_t)t * H + c, n);
 #pragma unroll
-            for (int i = 0; i < V; i++) u.v[i] = fmaf(s_in[t], n.v[i], u.v[i]);
+            for (int i = 0; i < V; i++) u.v[i] = fmaf(win(t), n.v[i], u.v[i]);
           }
         }
       } else {
@@ -113,7 +133,7 @@ __global__ void __launch_bounds__(SB_THREADS) stream_boundary_kernel(const Bound
         for (int s = 0; s < SM; s++)
           if (s < S)
 #pragma unroll
-            for (int i = 0; i < V; i++) u.v[i] = fmaf(s_in[s], xs[s].v[i], u.v[i]);
+            for (int i = 0; i < V; i++) u.v[i] = fmaf(win(s), xs[s].v[i], u.v[i]);
       }
 #pragma unroll
       for (int i = 0; i < V; i++) ss = fmaf(u.v[i], u.v[i], ss);
@@ -209,8 +229,8 @@ __global__ void __launch_bounds__(256) stream_sum_kernel(const float *__restrict
 
 __global__ void __launch_bounds__(256) stream_embed_kernel(const int *__restrict__ ids, const __nv_bfloat16 *__restrict__ table, int table_stride, float scale,
                                                            int S, int H, float *__restrict__ x, const float *__restrict__ in, float *__restrict__ u, int rows) {
-  pdl_launch();
   pdl_wait();
+  pdl_launch();
   float w = 0.0f;
   if (u) for (int s = 0; s < S; s++) w += in[s];
   const size_t total = (size_t)rows * H;
@@ -222,7 +242,45 @@ __global__ void __launch_bounds__(256) stream_embed_kernel(const int *__restrict
   }
 }
 
-template <typename OutT>
+// one warp per (row, part), the part in registers (parts of at most 128 * MAXV values, all sizes multiples of four)
+template <int MAXV, typename OutT>
+__global__ void __launch_bounds__(256) group_norm_warp_kernel(const float *__restrict__ x, int x_stride, const __nv_bfloat16 *__restrict__ w, int groups, int gs,
+                                                              float eps, OutT *__restrict__ dst, int dst_stride, int rows) {
+  pdl_launch();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, part = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (part >= rows * groups) return;
+  const int row = part / groups, c0 = (part - row * groups) * gs;
+  const float *xr = x + (size_t)row * x_stride + c0;
+  FV<4> v[MAXV];
+  float ss = 0.0f;
+#pragma unroll
+  for (int j = 0; j < MAXV; j++) {
+    const int c = (lane + 32 * j) * 4;
+    if (c < gs) v[j] = ldv<4>(xr + c);
+    else v[j] = FV<4>{};
+  }
+#pragma unroll
+  for (int j = 0; j < MAXV; j++)
+#pragma unroll
+    for (int i = 0; i < 4; i++) ss = fmaf(v[j].v[i], v[j].v[i], ss);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = 1.0f / sqrtf(ss / (float)gs + eps);
+  OutT *d = dst + (size_t)row * dst_stride + c0;
+#pragma unroll
+  for (int j = 0; j < MAXV; j++) {
+    const int c = (lane + 32 * j) * 4;
+    if (c < gs) {
+      const FV<4> wv = ldw<4>(w + c0 + c);
+#pragma unroll
+      for (int i = 0; i < 4; i++) v[j].v[i] = v[j].v[i] * inv * wv.v[i];
+      stv<4>(d + c, v[j]);
+    }
+  }
+}
+
+template <int V, typename OutT>
 __global__ void __launch_bounds__(256) group_norm_kernel(const float *__restrict__ x, int x_stride, const __nv_bfloat16 *__restrict__ w, int gs, float eps,
                                                          OutT *__restrict__ dst, int dst_stride) {
   pdl_launch();
@@ -230,8 +288,13 @@ __global__ void __launch_bounds__(256) group_norm_kernel(const float *__restrict
   __shared__ float sh[8];
   const int c0 = blockIdx.y * gs, tid = threadIdx.x;
   const float *xr = x + (size_t)blockIdx.x * x_stride + c0;
+  const FV<V> first = tid * V < gs ? ldv<V>(xr + tid * V) : FV<V>{};  // kept for the second pass
   float ss = 0.0f;
-  for (int c = tid; c < gs; c += 256) ss = fmaf(xr[c], xr[c], ss);
+  for (int c = tid * V; c < gs; c += 256 * V) {
+    const FV<V> v = c == tid * V ? first : ldv<V>(xr + c);
+#pragma unroll
+    for (int i = 0; i < V; i++) ss = fmaf(v.v[i], v.v[i], ss);
+  }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
   if ((tid & 31) == 0) sh[tid >> 5] = ss;
@@ -241,9 +304,12 @@ __global__ void __launch_bounds__(256) group_norm_kernel(const float *__restrict
   for (int i = 0; i < 8; i++) t += sh[i];
   const float inv = 1.0f / sqrtf(t / (float)gs + eps);
   OutT *d = dst + (size_t)blockIdx.x * dst_stride + c0;
-  for (int c = tid; c < gs; c += 256) {
-    const FV<1> v = {{xr[c] * inv * __bfloat162float(w[c0 + c])}};
-    stv<1>(d + c, v);
+  for (int c = tid * V; c < gs; c += 256 * V) {
+    FV<V> v = c == tid * V ? first : ldv<V>(xr + c);
+    const FV<V> wv = ldw<V>(w + c0 + c);
+#pragma unroll
+    for (int i = 0; i < V; i++) v.v[i] = v.v[i] * inv * wv.v[i];
+    stv<V>(d + c, v);
   }
 }
 
@@ -270,15 +336,20 @@ dp_status dpk_stream_boundary(dp_ctx *ctx, const float *x, float *x_out, const f
   const int gs = width / next.groups;
   const int halo = (map.pos || next.taps < 2) ? 0 : next.taps - 1;
   const size_t row_bytes = (size_t)gs * 4;
-  // rows per CTA: as many as fit where two CTAs still share an SM, fewer when the launch would not fill the GPU
-  size_t cap = ((size_t)ctx->smem_optin - 4096) / row_bytes;
-  size_t want = (size_t)98304 / row_bytes;
-  if (want > 16) want = 16;  // two rounds of the CTA's eight warps, the reached-back rows included
-  if (want < 1 + (size_t)halo) want = 1 + (size_t)halo;
-  if (want > cap) return dp_fail(ctx, DP_ERR_UNSUPPORTED, "streams: %d channels per norm group and %d taps exceed shared memory", gs, next.taps);
-  int R = (int)want - halo;
-  if (map.pos) R = 1;
-  while (R > 4 && (long)((rows + R - 1) / R) * next.groups < 2l * ctx->sm_count) R = (R + 1) / 2;
+  // Rows per CTA: the shape with the fewest rounds of the CTA's warps (reached-back rows included) on two CTAs per SM.
+  const int cap = (int)(((size_t)ctx->smem_optin - 4096) / row_bytes), want = (int)((size_t)102400 / row_bytes);
+  if (cap < 1 + halo) return dp_fail(ctx, DP_ERR_UNSUPPORTED, "streams: %d channels per norm group and %d taps exceed shared memory", gs, next.taps);
+  int most = (want < cap ? want : cap) - halo;
+  if (most < 1) most = 1;
+  if (most > 32) most = 32;
+  if (most > rows) most = rows;
+  int R = 1;
+  long best = -1;
+  for (int r = 1; r <= most; r++) {
+    const long blocks = (long)((rows + r - 1) / r) * next.groups, slots = 2l * ctx->sm_count;
+    const long cost = ((blocks + slots - 1) / slots) * ((r + halo + SB_WARPS - 1) / SB_WARPS);
+    if (best < 0 || cost < best) { best = cost; R = r; }
+  }
   BoundaryArgs a;
   a.x = x; a.y = y; a.x_out = x_out; a.end = end; a.next = next;
   a.streams = streams; a.width = width; a.rows = rows; a.dst_stride = dst_stride; a.block_rows = R; a.map = map;
@@ -303,8 +374,18 @@ dp_status dpk_stream_embed(dp_ctx *ctx, const int *ids, const __nv_bfloat16 *tab
 dp_status dpk_group_norm(dp_ctx *ctx, const float *x, int x_stride, const __nv_bfloat16 *w, int groups, float eps, int width, void *dst, bool dst_bf16,
                          int dst_stride, int rows) {
   const dim3 grid(rows, groups);
-  if (dst_bf16) DP_LAUNCH(ctx, group_norm_kernel<__nv_bfloat16>, grid, 256, 0, x, x_stride, w, width / groups, eps, (__nv_bfloat16 *)dst, dst_stride);
-  else DP_LAUNCH(ctx, group_norm_kernel<float>, grid, 256, 0, x, x_stride, w, width / groups, eps, (float *)dst, dst_stride);
+  const int gs = width / groups;
+  const bool vec = gs % 4 == 0 && x_stride % 4 == 0 && dst_stride % 4 == 0;
+  if (vec && gs <= 1024) {
+    const unsigned blocks = (unsigned)(((size_t)rows * groups + 7) / 8);
+    if (dst_bf16) DP_LAUNCH(ctx, (group_norm_warp_kernel<8, __nv_bfloat16>), blocks, 256, 0, x, x_stride, w, groups, gs, eps, (__nv_bfloat16 *)dst, dst_stride, rows);
+    else DP_LAUNCH(ctx, (group_norm_warp_kernel<8, float>), blocks, 256, 0, x, x_stride, w, groups, gs, eps, (float *)dst, dst_stride, rows);
+    return DP_OK;
+  }
+#define DP_NORM(V, T) DP_LAUNCH(ctx, (group_norm_kernel<V, T>), grid, 256, 0, x, x_stride, w, gs, eps, (T *)dst, dst_stride)
+  if (dst_bf16) { if (vec) DP_NORM(4, __nv_bfloat16); else DP_NORM(1, __nv_bfloat16); }
+  else { if (vec) DP_NORM(4, float); else DP_NORM(1, float); }
+#undef DP_NORM
   return DP_OK;
 }
 
