@@ -5,6 +5,7 @@ Usage: python -m doppler_b200.build [--force] [--verbose]
 from __future__ import annotations
 
 import concurrent.futures as cf
+import fcntl
 import os
 import shutil
 import subprocess
@@ -44,7 +45,22 @@ def _deps_mtime() -> float:
 
 
 def build(force: bool = False, verbose: bool = False) -> str:
+    """Compile what is missing or older than its sources; one process at a time, outputs appear whole."""
     os.makedirs(OBJ, exist_ok=True)
+    with open(os.path.join(OBJ, "lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build(force, verbose)
+
+
+def _compile(cmd: list[str], out: str) -> subprocess.CompletedProcess:
+    part = f"{out}.part{os.path.splitext(out)[1]}"
+    res = subprocess.run([part if c == out else c for c in cmd], capture_output=True, text=True)
+    if res.returncode == 0:
+        os.replace(part, out)
+    return res
+
+
+def _build(force: bool, verbose: bool) -> str:
     nvcc, dep_t = _nvcc(), _deps_mtime()
     jobs = []
     for src in sources():
@@ -56,7 +72,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
             jobs.append(cmd)
     if jobs:
         with cf.ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
-            for cmd, res in zip(jobs, ex.map(lambda c: subprocess.run(c, capture_output=True, text=True), jobs)):
+            for cmd, res in zip(jobs, ex.map(lambda c: _compile(c, c[-1]), jobs)):
                 if verbose and res.stderr:
                     print(res.stderr, file=sys.stderr)
                 if res.returncode != 0:
@@ -64,7 +80,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
     objs = [os.path.join(OBJ, os.path.basename(s)[:-3] + ".o") for s in sources()]
     if jobs or not os.path.exists(LIB):
         cmd = [nvcc, *_host_cxx(), "-shared", "-o", LIB, *objs, "-ldl", "-lpthread"]
-        res = subprocess.run(cmd, capture_output=True, text=True)
+        res = _compile(cmd, LIB)
         if res.returncode != 0:
             raise RuntimeError("link failed: %s\n%s" % (" ".join(cmd), res.stderr))
     return LIB

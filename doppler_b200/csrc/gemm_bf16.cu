@@ -36,6 +36,15 @@ __device__ __forceinline__ float glu_act(float g, float u, const GluArgs &a) {
   return g * (1.0f / (1.0f + expf(-a.slope * g))) * (u + a.shift);
 }
 
+// ... for a result that is stored as bf16
+__device__ __forceinline__ float glu_act_fast(float g, float u, const GluArgs &a) {
+  if (a.limit > 0.0f) {
+    g = fminf(g, a.limit);
+    u = fminf(fmaxf(u, -a.limit), a.limit);
+  }
+  return __fdividef(g, 1.0f + __expf(-a.slope * g)) * (u + a.shift);
+}
+
 constexpr int BT_THREADS = 256, BT_MAX_STAGES = 8;
 constexpr uint32_t BT_W_TILE = 128u * 128u;  // 128 weight rows x 64 bf16
 
@@ -144,13 +153,16 @@ __global__ void __launch_bounds__(BT_THREADS, 1) gemm_bf16_tc_kernel(const __gri
         tmem_ld16(taddr + (uint32_t)c0, r);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         if (a.glu.dst) {
-          const int j = (f >> 4) * 8 + (f & 7);
-          __nv_bfloat16 *dst = reinterpret_cast<__nv_bfloat16 *>(a.glu.dst) + j;
+          // a gate row and its up row are eight lanes apart: the gate's lane takes the even activation rows of the pair,
+          // the other lane the odd ones
+          const bool is_up = lane & 8;
+          __nv_bfloat16 *dst = reinterpret_cast<__nv_bfloat16 *>(a.glu.dst) + (f >> 4) * 8 + (f & 7);
 #pragma unroll
-          for (int i = 0; i < 16; i++) {
-            const float up = __shfl_down_sync(0xffffffffu, __uint_as_float(r[i]), 8);
-            if (!(lane & 8) && f < a.N && m0 + c0 + i < a.M)
-              dst[(size_t)(m0 + c0 + i) * a.glu.stride] = __float2bfloat16_rn(glu_act(__uint_as_float(r[i]), up, a.glu));
+          for (int i = 0; i < 16; i += 2) {
+            const float got = __shfl_xor_sync(0xffffffffu, __uint_as_float(is_up ? r[i] : r[i + 1]), 8);
+            const float gv = is_up ? got : __uint_as_float(r[i]), uv = is_up ? __uint_as_float(r[i + 1]) : got;
+            const int row = m0 + c0 + i + (is_up ? 1 : 0);
+            if (f < a.N && row < a.M) dst[(size_t)row * a.glu.stride] = __float2bfloat16_rn(glu_act_fast(gv, uv, a.glu));
           }
         } else if (f < a.N) {
           float *dst = a.C + (size_t)(m0 + c0) * a.N + f;

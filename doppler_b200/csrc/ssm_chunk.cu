@@ -8,8 +8,9 @@
 // f32 operand (the state, the weighted C.B products, the weighted x) enters its product as three bf16 terms that add
 // up to its 24 bits, each multiplied exactly with the bf16 operand.
 //
-// One CTA = PB of a head's value columns, eight warps, chunks in sequence.  Per chunk, with mma.sync m16n8k16:
-//   G  [t, s] = C B^T                 each warp a (16 t, 32 s) block; weighted, split, to shared memory
+// One CTA = PB of a head's value columns, chunks in sequence.  Per chunk, with mma.sync m16n8k16:
+//   Xw [s, p] = exp(c_end - c_s) dt_s x_s  split, to shared memory
+//   G  [t, s] = C B^T                 each warp a block of it; weighted, split, to shared memory
 //   Y^T[p, t] = S^T C^T (state terms from shared memory), scaled by exp(c_t), then += X^T G'^T
 //   S^T[p, n] = exp(c_end) S^T + Xw^T B   in registers; its terms go to shared memory for the next chunk
 // with the warps dealt (16 p) x (64 / TW t) for Y and (16 p) x (N / TW n) for S.  The next chunk's rows are brought in
@@ -19,7 +20,7 @@
 
 namespace {
 
-constexpr int CQ = 64, CK_THREADS = 256, TERMS = 3;
+constexpr int CQ = 64, TERMS = 3;
 
 __device__ __forceinline__ uint32_t ck_smem(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void ck_cp16(uint32_t dst, const void *src, int bytes) {
@@ -65,25 +66,33 @@ __device__ __forceinline__ void ck_split(float x, float y, uint32_t (&t)[TERMS])
     y -= __uint_as_float(t[i] & 0xffff0000u);
   }
 }
+__device__ __forceinline__ float ck_exp2(float v) {  // relative error 2^-22
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+  return r;
+}
 __device__ __forceinline__ float ck_silu(float v) { return __fdividef(v, 1.0f + __expf(-v)); }  // the output gate, not the recurrence
 
 template <int N, int PB> struct CkLayout {
   static constexpr int NROW = N * 2 + 16, QROW = CQ * 2 + 16, PROW = PB * 2 + 16;  // bytes per shared row
   static constexpr int B = 0, C = B + CQ * NROW, X = C + CQ * NROW, DT = X + CQ * PROW, STAGE = DT + CQ * 4;
-  static constexpr int M = 2 * STAGE;                 // weighted C.B terms [TERMS][t][s]
+  static constexpr int WARPS = PB > 32 ? 16 : 8, THREADS = WARPS * 32;
+  static constexpr int STAGES = PB > 32 ? 2 : 1;      // one, where that lets two CTAs share an SM
+  static constexpr int M = STAGES * STAGE;                 // weighted C.B terms [TERMS][t][s]
   static constexpr int S = M + TERMS * CQ * QROW;     // state terms [TERMS][p][n]
-  static constexpr int CUM = S + TERMS * PB * NROW;   // c_t log2(e), then the weights of the state update
+  static constexpr int XW = S + TERMS * PB * NROW;    // weighted x terms [TERMS][s][p]
+  static constexpr int CUM = XW + TERMS * CQ * PROW;   // c_t log2(e), then the weights of the state update
   static constexpr int TOTAL = CUM + 2 * CQ * 4;
 };
 
 template <int N, int PB>
-__global__ void __launch_bounds__(CK_THREADS) ssm_chunk_kernel(const float *__restrict__ proj, int proj_stride, const __nv_bfloat16 *__restrict__ xbc,
+__global__ void __launch_bounds__((CkLayout<N, PB>::THREADS), PB > 32 ? 1 : 2) ssm_chunk_kernel(const float *__restrict__ proj, int proj_stride, const __nv_bfloat16 *__restrict__ xbc,
                                                                const float *__restrict__ dt, const SsmShape sh, const SsmWeights w, const SsmState st,
                                                                float *__restrict__ out, int rows, int start_pos, int seq) {
   pdl_launch();
   pdl_wait();
   using L = CkLayout<N, PB>;
-  constexpr int PBLK = PB / 16, TW = 8 / PBLK;         // p blocks, warps per p block
+  constexpr int PBLK = PB / 16, TW = L::WARPS / PBLK;  // p blocks, warps per p block
   constexpr int TT = CQ / TW / 8;                      // 8-token tiles of Y per warp
   constexpr int NTILES = N / 8, NT = NTILES >= TW ? NTILES / TW : 1;  // 8-wide state tiles per warp
   extern __shared__ __align__(128) unsigned char ck_raw[];
@@ -98,16 +107,25 @@ __global__ void __launch_bounds__(CK_THREADS) ssm_chunk_kernel(const float *__re
   float *s_cum = reinterpret_cast<float *>(ck_raw + L::CUM), *s_wt = s_cum + CQ;
 
   auto stage = [&](int chunk) {
-    const uint32_t base = sm + (uint32_t)(chunk & 1) * L::STAGE;
+    const uint32_t base = sm + (uint32_t)(chunk % L::STAGES) * L::STAGE;
     const int r0 = chunk * CQ;
-    constexpr int CB = N / 8, CX = PB / 8, PER = 2 * CB + CX;  // 16-byte pieces per token
-    for (int i = tid; i < CQ * PER; i += CK_THREADS) {
-      const int t = i / PER, e = i - t * PER;
+    constexpr int CB = N / 8, CX = PB / 8;  // 16-byte pieces per token
+    // B and C: a warp per token, a lane per piece
+    if (lane < 2 * CB) {
+      const bool is_c = lane >= CB;
+      const int e = is_c ? lane - CB : lane;
+      const __nv_bfloat16 *src = xbc + inner + ((is_c ? G : 0) + grp) * N + e * 8;
+      const uint32_t dst = base + (is_c ? L::C : L::B) + e * 16;
+#pragma unroll
+      for (int t = warp; t < CQ; t += L::WARPS) {
+        const bool ok = r0 + t < rows;
+        ck_cp16(dst + t * L::NROW, src + (size_t)(ok ? r0 + t : 0) * CH, ok ? 16 : 0);
+      }
+    }
+    if (tid < CQ * CX) {
+      const int t = tid / CX, e = tid % CX;
       const bool ok = r0 + t < rows;
-      const __nv_bfloat16 *row = xbc + (size_t)(ok ? r0 + t : 0) * CH;
-      if (e < CB) ck_cp16(base + L::B + t * L::NROW + e * 16, row + inner + grp * N + e * 8, ok ? 16 : 0);
-      else if (e < 2 * CB) ck_cp16(base + L::C + t * L::NROW + (e - CB) * 16, row + inner + (G + grp) * N + (e - CB) * 8, ok ? 16 : 0);
-      else ck_cp16(base + L::X + t * L::PROW + (e - 2 * CB) * 16, row + h * P + p0 + (e - 2 * CB) * 8, ok ? 16 : 0);
+      ck_cp16(base + L::X + t * L::PROW + e * 16, xbc + (size_t)(ok ? r0 + t : 0) * CH + h * P + p0 + e * 8, ok ? 16 : 0);
     }
     if (tid < CQ) {
       const bool ok = r0 + tid < rows;
@@ -149,9 +167,9 @@ __global__ void __launch_bounds__(CK_THREADS) ssm_chunk_kernel(const float *__re
   for (int chunk = 0; chunk < chunks; chunk++) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();  // this chunk's rows and the state terms are there; the other stage is free
-    if (chunk + 1 < chunks) stage(chunk + 1);
-    const uint32_t base = sm + (uint32_t)(chunk & 1) * L::STAGE;
-    const unsigned char *basep = ck_raw + (chunk & 1) * L::STAGE;
+    if (L::STAGES == 2 && chunk + 1 < chunks) stage(chunk + 1);
+    const uint32_t base = sm + (uint32_t)(chunk % L::STAGES) * L::STAGE;
+    const unsigned char *basep = ck_raw + (chunk % L::STAGES) * L::STAGE;
     const float *s_dt = reinterpret_cast<const float *>(basep + L::DT);
     const int r0 = chunk * CQ, n_tok = min(CQ, rows - r0);
 
@@ -179,22 +197,36 @@ __global__ void __launch_bounds__(CK_THREADS) ssm_chunk_kernel(const float *__re
       c_end = __shfl_sync(0xffffffffu, sum, 31);
       const float c1 = sum, c0 = sum - v1;
       s_cum[2 * lane] = c0; s_cum[2 * lane + 1] = c1;
-      s_wt[2 * lane] = exp2f(c_end - c0) * d0; s_wt[2 * lane + 1] = exp2f(c_end - c1) * d1;
+      s_wt[2 * lane] = ck_exp2(c_end - c0) * d0; s_wt[2 * lane + 1] = ck_exp2(c_end - c1) * d1;
       __syncwarp();
+    }
+
+    // ---- Xw[s, p] ----
+    static_assert(CQ * PB / 8 <= L::THREADS && (CQ * PB / 2) % L::THREADS == 0, "one 16-byte piece of x per thread at most, whole passes over its pairs");
+#pragma unroll
+    for (int i = 0; i < CQ * PB / 2 / L::THREADS; i++) {
+      const int idx = tid + i * L::THREADS, s = idx / (PB / 2), pp = idx % (PB / 2);
+      const uint32_t x = *reinterpret_cast<const uint32_t *>(basep + L::X + s * L::PROW + pp * 4);
+      const float wt = s_wt[s];
+      uint32_t t[TERMS];
+      ck_split(__uint_as_float(x << 16) * wt, __uint_as_float(x & 0xffff0000u) * wt, t);
+#pragma unroll
+      for (int j = 0; j < TERMS; j++) *reinterpret_cast<uint32_t *>(ck_raw + L::XW + (j * CQ + s) * L::PROW + pp * 4) = t[j];
     }
 
     // ---- G[t, s] = C_t . B_s, weighted by exp(c_t - c_s) dt_s below the diagonal ----
     {
-      const int tb = warp >> 1, s_lo = (warp & 1) * 32;
-      const int s_tiles = tb * 16 + 15 >= s_lo ? min(4, (tb * 16 + 15 - s_lo) / 8 + 1) : 0;  // 8-wide tiles that are not wholly masked
-      float acc[4][4] = {};
+      constexpr int SW = L::WARPS / 4, SC = CQ / SW, ST = SC / 8;  // warps across s, columns and 8-wide tiles of each
+      const int tb = warp / SW, s_lo = (warp % SW) * SC;
+      const int s_tiles = tb * 16 + 15 >= s_lo ? min(ST, (tb * 16 + 15 - s_lo) / 8 + 1) : 0;  // tiles that are not wholly masked
+      float acc[ST][4] = {};
       if (s_tiles > 0) {
 #pragma unroll
         for (int k = 0; k < N / 16; k++) {
           uint32_t a[4];
           ck_ldm(a, base + L::C + (tb * 16 + (lane & 15)) * L::NROW + (k * 16 + (lane >> 4) * 8) * 2);
 #pragma unroll
-          for (int jj = 0; jj < 2; jj++) {
+          for (int jj = 0; jj < ST / 2; jj++) {
             if (2 * jj < s_tiles) {
               uint32_t b[4];
               ck_ldm(b, base + L::B + (s_lo + jj * 16 + (lane & 7) + 8 * (lane >> 4)) * L::NROW + (k * 16 + ((lane >> 3) & 1) * 8) * 2);
@@ -204,19 +236,30 @@ __global__ void __launch_bounds__(CK_THREADS) ssm_chunk_kernel(const float *__re
           }
         }
       }
+      const float ct0 = s_cum[tb * 16 + g], ct1 = s_cum[tb * 16 + g + 8];
 #pragma unroll
-      for (int j = 0; j < 4; j++)
+      for (int j = 0; j < ST; j++) {
+        const int s = s_lo + j * 8 + 2 * t4;
+        if (j < s_tiles) {
+          const float2 cs = *reinterpret_cast<const float2 *>(s_cum + s), ds = *reinterpret_cast<const float2 *>(s_dt + s);
 #pragma unroll
-        for (int half = 0; half < 2; half++) {
-          const int t = tb * 16 + g + 8 * half, s = s_lo + j * 8 + 2 * t4;
-          const float ct = s_cum[t];
-          const float m0 = s <= t ? acc[j][2 * half] * exp2f(ct - s_cum[s]) * s_dt[s] : 0.0f;
-          const float m1 = s + 1 <= t ? acc[j][2 * half + 1] * exp2f(ct - s_cum[s + 1]) * s_dt[s + 1] : 0.0f;
-          uint32_t terms[TERMS];
-          ck_split(m0, m1, terms);
+          for (int half = 0; half < 2; half++) {
+            const int t = tb * 16 + g + 8 * half;
+            const float ct = half ? ct1 : ct0;
+            const float m0 = s <= t ? acc[j][2 * half] * ck_exp2(ct - cs.x) * ds.x : 0.0f;
+            const float m1 = s + 1 <= t ? acc[j][2 * half + 1] * ck_exp2(ct - cs.y) * ds.y : 0.0f;
+            uint32_t terms[TERMS];
+            ck_split(m0, m1, terms);
 #pragma unroll
-          for (int i = 0; i < TERMS; i++) *reinterpret_cast<uint32_t *>(ck_raw + L::M + (i * CQ + t) * L::QROW + s * 2) = terms[i];
+            for (int i = 0; i < TERMS; i++) *reinterpret_cast<uint32_t *>(ck_raw + L::M + (i * CQ + t) * L::QROW + s * 2) = terms[i];
+          }
+        } else {
+#pragma unroll
+          for (int half = 0; half < 2; half++)
+#pragma unroll
+            for (int i = 0; i < TERMS; i++) *reinterpret_cast<uint32_t *>(ck_raw + L::M + (i * CQ + tb * 16 + g + 8 * half) * L::QROW + s * 2) = 0u;
         }
+      }
     }
 
     // ---- Y^T[p, t] = exp(c_t) S^T C_t ----
@@ -240,22 +283,23 @@ __global__ void __launch_bounds__(CK_THREADS) ssm_chunk_kernel(const float *__re
 #pragma unroll
       for (int j = 0; j < TT; j++) {
         const int t = (tw * TT + j) * 8 + 2 * t4;
-        const float e0 = exp2f(s_cum[t]), e1 = exp2f(s_cum[t + 1]);
+        const float e0 = ck_exp2(s_cum[t]), e1 = ck_exp2(s_cum[t + 1]);
         y[j][0] *= e0; y[j][1] *= e1; y[j][2] *= e0; y[j][3] *= e1;
       }
     }
     __syncthreads();  // the weighted products are there, and nobody reads the state terms any more
 
-    // ---- Y^T += X^T G'^T and S^T = exp(c_end) S^T + Xw^T B, the x fragments shared ----
-    const float decay = exp2f(c_end);
+    // ---- Y^T += X^T G'^T and S^T = exp(c_end) S^T + Xw^T B ----
+    const float decay = ck_exp2(c_end);
 #pragma unroll
     for (int j = 0; j < NT; j++) { acc_s[j][0] *= decay; acc_s[j][1] *= decay; acc_s[j][2] *= decay; acc_s[j][3] *= decay; }
     const int t_last = (tw * TT + TT) * 8 - 1;  // last token of this warp's Y tile
 #pragma unroll
     for (int k = 0; k < CQ / 16; k++) {
-      uint32_t x[4];
-      ck_ldmt(x, base + L::X + (k * 16 + (lane & 7) + 8 * (lane >> 4)) * L::PROW + (pblk * 16 + ((lane >> 3) & 1) * 8) * 2);
+      const uint32_t x_off = (k * 16 + (lane & 7) + 8 * (lane >> 4)) * L::PROW + (pblk * 16 + ((lane >> 3) & 1) * 8) * 2;
       if (k * 16 <= t_last) {
+        uint32_t x[4];
+        ck_ldmt(x, base + L::X + x_off);
 #pragma unroll
         for (int i = TERMS - 1; i >= 0; i--) {
           uint32_t b[TT][2];
@@ -266,15 +310,8 @@ __global__ void __launch_bounds__(CK_THREADS) ssm_chunk_kernel(const float *__re
       }
       if (has_state) {
         uint32_t xw[TERMS][4];
-        const float2 w0 = *reinterpret_cast<const float2 *>(s_wt + k * 16 + 2 * t4), w1 = *reinterpret_cast<const float2 *>(s_wt + k * 16 + 8 + 2 * t4);
 #pragma unroll
-        for (int e = 0; e < 4; e++) {
-          const float2 wv = e < 2 ? w0 : w1;
-          uint32_t t[TERMS];
-          ck_split(__uint_as_float(x[e] << 16) * wv.x, __uint_as_float(x[e] & 0xffff0000u) * wv.y, t);
-#pragma unroll
-          for (int i = 0; i < TERMS; i++) xw[i][e] = t[i];
-        }
+        for (int i = 0; i < TERMS; i++) ck_ldmt(xw[i], sm + L::XW + i * CQ * L::PROW + x_off);
         if constexpr (NT >= 2) {
           uint32_t b[NT / 2][4];
 #pragma unroll
@@ -304,6 +341,10 @@ __global__ void __launch_bounds__(CK_THREADS) ssm_chunk_kernel(const float *__re
           out[(size_t)(r0 + t) * inner + h * P + p0 + p] = fmaf(dh, x, y[j][e]) * ck_silu(z[j][e]);
         }
       }
+    if (L::STAGES == 1 && chunk + 1 < chunks) {
+      __syncthreads();  // nobody reads this chunk's rows any more
+      stage(chunk + 1);
+    }
   }
   if (has_state)
 #pragma unroll
@@ -322,7 +363,7 @@ dp_status launch(dp_ctx *ctx, const float *proj, int proj_stride, const __nv_bfl
     DP_CUDA(ctx, cudaFuncSetAttribute((ssm_chunk_kernel<N, PB>), cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     attr.done(ctx->device);
   }
-  DP_LAUNCH(ctx, (ssm_chunk_kernel<N, PB>), dim3(sh.heads, sh.vdim / PB), CK_THREADS, smem, proj, proj_stride, xbc, dt, sh, w, st, out, rows, map.start_pos, map.seq);
+  DP_LAUNCH(ctx, (ssm_chunk_kernel<N, PB>), dim3(sh.heads, sh.vdim / PB), (CkLayout<N, PB>::THREADS), smem, proj, proj_stride, xbc, dt, sh, w, st, out, rows, map.start_pos, map.seq);
   return DP_OK;
 }
 

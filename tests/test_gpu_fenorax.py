@@ -284,6 +284,21 @@ def test_large_sizes_bf16(dev, name):
     m.destroy()
 
 
+@pytest.mark.parametrize("heads,kv_heads,dim", [(8, 2, 128), (6, 2, 64), (12, 1, 64)])
+def test_split_keys_bf16(dev, heads, kv_heads, dim):
+    """A chunk so long that decoding splits its keys over several CTAs, before and after the chunk's edge."""
+    cfg = config([attention(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=0.25, chunk=640)], width=128)
+    n = 660
+    w, t, logits, _ = oracle(f"split {heads} {dim}", cfg, n)
+    m = build(dev, cfg, w, 1300, dtype="bfloat16")
+    got = [m.extend(t[:620], range(600, 620))]
+    for i in range(620, n):
+        m.decode([t[i]], 1)
+        got.append(m.read_logits()[None])
+    check(np.concatenate(got), logits[600:], BF16_TOL / 2)
+    m.destroy()
+
+
 def test_recurrence_in_chunks_is_32_bit(dev):
     """Inputs that bf16 holds exactly (one-hot projections of small integers, a convolution that passes its input through a
     saturated silu) leave only the recurrence's own arithmetic: chunks, token by token and the f32 mode agree closely."""
