@@ -21,6 +21,8 @@ roofline  the dominant kernels (the Q4_K decode GEMVs as the decode graph launch
 kernels   the other BASELINE configurations, a few ms each through the C ABI: config 0 GEMV (us),
           config 1 GEMM (TFLOP/s, fraction of the measured bf16 burst and sustained peaks),
           config 2 decode attention (GB/s, fraction of measured HBM).  N = 1 only.
+--case stack (not part of the default line): prefill and decode of a Fenorax decoder at the same layer sizes, random
+          weights, beside the dense decoder.
 tokens_crc  CRC-32 of the tokens of the warm-up and the first timed region; every rank must hold
           the same tokens (checked), and the N = 1 and N = 8 lines can be compared.
 cpu_baseline / --impl reference

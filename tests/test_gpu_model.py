@@ -124,3 +124,41 @@ def test_batched_decode_is_independent_sequences(dev):
             assert int(out[s, i]) == cur, f"sequence {i} step {s}: {int(out[s, i])} vs oracle {cur} (margin {margin:.3e})"
         assert m.seq_len(i) == lens[i] + steps
     m.destroy()
+
+
+def test_portions_return_the_same_logits(dev):
+    """dp_model_extend: a prompt in portions, logits at wanted places, against whole prompts."""
+    cfg = dict(synthetic.MODEL_CONFIGS["tiny"])
+    m = DecoderModel(dev, cfg, max_seq=96)
+    m.load_all(gaussian_model_weights(cfg, 7))
+    prompt = synthetic.make_prompt(cfg, 40, seed=7)
+    assert m.extend(prompt[:9]).shape == (0, cfg["vocab"])
+    rows = m.extend(prompt[9:], [0, 12, 30])
+    for place, row in zip((9, 21, 39), rows):
+        m.reset()
+        m.prefill(prompt[:place + 1])
+        assert_close(row, m.read_logits(), f"logits at {place}")
+    m.destroy()
+
+
+def test_artifact_through_the_registry_and_scheduler(dev, tmp_path):
+    """An RDRR folder opened by the model registry and run by the scheduler gives the runner's own greedy tokens."""
+    from doppler_b200.rdrr import write_artifact
+    from doppler_b200.registry import load_model
+    from doppler_b200.scheduler import Scheduler
+
+    cfg = dict(synthetic.MODEL_CONFIGS["tiny"])
+    w = gaussian_model_weights(cfg, 11)
+    w["layers"] = [{k: v.astype(np.float16).astype(np.float32) if k.endswith("norm") else v for k, v in l.items()} for l in w["layers"]]
+    w["final_norm"] = w["final_norm"].astype(np.float16).astype(np.float32)
+    write_artifact(str(tmp_path), dict(cfg, max_seq_len=256), w)
+    prompts = [synthetic.make_prompt(cfg, n, seed=11, seq=n).tolist() for n in (12, 5)]
+    m = load_model(dev, str(tmp_path), 96, max_batch=2)
+    got = Scheduler(m).generate(prompts, 20, block=6)
+    m.destroy()
+    m = DecoderModel(dev, cfg, max_seq=96, max_batch=2)
+    m.load_all(w)
+    firsts = [m.prefill(p, seq=i) for i, p in enumerate(prompts)]
+    out = m.decode(firsts, 19)
+    m.destroy()
+    assert got == [[f, *out[:, i].tolist()] for i, f in enumerate(firsts)]
