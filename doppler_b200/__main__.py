@@ -50,11 +50,11 @@ def info(argv) -> int:
     ap = argparse.ArgumentParser(prog="doppler_b200 info")
     ap.add_argument("--model", required=True)
     args = ap.parse_args(argv)
-    from . import fenorax, registry
+    from . import registry
 
     d = registry.describe(args.model)
-    if d["kind"] == fenorax.ARCHITECTURE:
-        stack, layers = fenorax.stack_config(d["config"])
+    if d["kind"] in registry.ARCHITECTURES:
+        stack, layers = registry.ARCHITECTURES[d["kind"]].describe(args.model, d["config"])
         print(json.dumps({"kind": d["kind"], "stack": stack, "layers": layers}))
     else:
         print(json.dumps(d))

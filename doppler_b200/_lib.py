@@ -22,9 +22,11 @@ DTYPE_BYTES = {"f32": 4, "f16": 2, "i32": 4, "bf16": 2}
 W_Q, W_K, W_V, W_O, W_GATE, W_UP, W_DOWN, W_IN_NORM, W_POST_NORM, W_Q_NORM, W_K_NORM = range(11)
 
 # decoders described layer by layer: mixers and tensor ids
-MIXER_ATTENTION, MIXER_MAMBA2 = 0, 1
+MIXER_ATTENTION, MIXER_MAMBA2, MIXER_LIGHTNING, MIXER_DELTA, MIXER_LATENT = range(5)
 (T_EMBED, T_FINAL_NORM, T_NORM1, T_NORM2, T_CONV1, T_CONV2, T_HC1_IN, T_HC1_OUT, T_HC1_MIX, T_HC2_IN, T_HC2_OUT, T_HC2_MIX, T_Q, T_K, T_V, T_GATE_HEADS,
- T_O, T_SSM_IN, T_SSM_CONV, T_SSM_CONV_B, T_SSM_DT_BIAS, T_SSM_A_LOG, T_SSM_D, T_SSM_NORM, T_FF_GATE, T_FF_UP, T_FF_DOWN) = range(27)
+ T_O, T_SSM_IN, T_SSM_CONV, T_SSM_CONV_B, T_SSM_DT_BIAS, T_SSM_A_LOG, T_SSM_D, T_SSM_NORM, T_FF_GATE, T_FF_UP, T_FF_DOWN, T_NORM1B, T_NORM2B, T_GATE,
+ T_MIX_NORM, T_CONV_Q, T_CONV_K, T_CONV_V, T_BETA, T_A1, T_A2, T_G1, T_G2, T_A_LOG, T_DT_BIAS, T_DQ, T_DQ_NORM, T_UQ, T_DKV, T_DKV_NORM, T_UK,
+ T_UV) = range(48)
 
 
 class DopplerError(RuntimeError):
@@ -86,12 +88,15 @@ class ModelCfg(C.Structure):
 class LayerCfg(C.Structure):
     _fields_ = ([(n, C.c_int) for n in ("mixer", "heads", "vdim", "kv_heads", "dim", "chunk", "unit_rms_qk", "head_gate")] + [("scale", C.c_float)]
                 + [(n, C.c_int) for n in ("state", "groups", "conv_taps", "norm_groups", "ff")]
-                + [(n, C.c_float) for n in ("ff_limit", "ff_slope", "ff_shift")])
+                + [(n, C.c_float) for n in ("ff_limit", "ff_slope", "ff_shift")]
+                + [(n, C.c_int) for n in ("share", "decay_rank", "gate_rank", "q_rank", "kv_rank", "rot_dim")]
+                + [("rot_base", C.c_double), ("decay", C.POINTER(C.c_double))])
 
 
 class StackCfg(C.Structure):
     _fields_ = ([(n, C.c_int) for n in ("n_layers", "width", "vocab", "max_seq", "max_batch", "streams", "norm_groups", "input_taps")]
-                + [("eps", C.c_float), ("embed_scale", C.c_float), ("act_dtype", C.c_int), ("max_rows", C.c_int)])
+                + [("eps", C.c_float), ("embed_scale", C.c_float), ("act_dtype", C.c_int), ("max_rows", C.c_int), ("post_norm", C.c_int),
+                   ("residual_mult", C.c_float)])
 
 
 _vp, _sz, _i, _f, _u32, _u64, _dbl = C.c_void_p, C.c_size_t, C.c_int, C.c_float, C.c_uint32, C.c_uint64, C.c_double

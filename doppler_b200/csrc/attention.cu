@@ -181,9 +181,9 @@ __global__ void __launch_bounds__(ATT_THREADS, LPK == 16 ? 2 : 1) attn_split_ker
   }
 }
 
-// Any query/key size and any value size up to 512, any GQA ratio, f16 or f32 caches: one CTA per (split, query
+// Any query/key size and any value size up to 32 * MAXE, any GQA ratio, f16 or f32 caches: one CTA per (split, query
 // head, row), lanes over dims.  Used for shapes outside the fast kernels.
-template <typename KT>
+template <typename KT, int MAXE>
 __global__ void __launch_bounds__(128) attn_split_generic_kernel(dpk_attn_params p, float *__restrict__ part, int splits) {
   pdl_launch();
   pdl_wait();
@@ -200,13 +200,12 @@ __global__ void __launch_bounds__(128) attn_split_generic_kernel(dpk_attn_params
   int k_end = k_begin + per_split;
   if (k_end > r.hi) k_end = r.hi;
   const float LOG2E = 1.4426950408889634f;
-  constexpr int MAXE = 16;  // dims per lane
-  float q[MAXE], o[MAXE];
+  float q[MAXE], o[MAXE];  // MAXE dims per lane
   const float *qp = p.q + ((size_t)z * p.num_heads + h) * D;
 #pragma unroll
   for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; q[i] = d < D ? qp[d] * p.scale : 0.0f; o[i] = 0.0f; }
   float m = -FLT_MAX, l = 0.0f;
-  const size_t k_stride = (size_t)p.num_kv_heads * D, v_stride = (size_t)p.num_kv_heads * V;
+  const size_t k_stride = (size_t)p.num_kv_heads * D, v_stride = p.v_row_stride ? (size_t)p.v_row_stride : (size_t)p.num_kv_heads * V;
   const KT *kb = reinterpret_cast<const KT *>(p.k) + (size_t)b * p.kv_batch_stride + (size_t)kvh * D;
   const KT *vb = reinterpret_cast<const KT *>(p.v) + (size_t)b * (p.v_batch_stride ? p.v_batch_stride : p.kv_batch_stride) + (size_t)kvh * V;
   for (int key = k_begin + warp; key < k_end; key += 4) {
@@ -229,7 +228,7 @@ __global__ void __launch_bounds__(128) attn_split_generic_kernel(dpk_attn_params
 #pragma unroll
     for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; if (d < V) o[i] = fmaf(pr, (float)vb[(size_t)key * v_stride + d], o[i]); }
   }
-  __shared__ float sm_o[4][512];
+  __shared__ float sm_o[4][32 * MAXE];
   __shared__ float sm_m[4], sm_l[4];
 #pragma unroll
   for (int i = 0; i < MAXE; i++) { const int d = lane + 32 * i; if (d < V) sm_o[warp][d] = o[i]; }
@@ -277,7 +276,7 @@ __global__ void attn_combine_kernel(dpk_attn_params p, const float *__restrict__
 }
 
 // caches the f16 kernels of one head size can read
-static bool f16_square(const dpk_attn_params &p) { return !p.kv_f32 && (p.v_dim == 0 || p.v_dim == p.head_dim); }
+static bool f16_square(const dpk_attn_params &p) { return !p.kv_f32 && !p.v_row_stride && (p.v_dim == 0 || p.v_dim == p.head_dim); }
 
 static bool fast_shape(const dpk_attn_params &p, int *gt) {
   if ((p.head_dim != 128 && p.head_dim != 64) || !f16_square(p)) return false;
@@ -396,9 +395,15 @@ static dp_status attention_impl(dp_ctx *ctx, const dpk_attn_params &p, float *sc
     }
   } else {
     dim3 grid(splits, p.num_heads, p.batch * p.seq_len);
-    if (p.head_dim > 512 || p.v_dim > 512) return dp_fail(ctx, DP_ERR_UNSUPPORTED, "attention: head sizes above 512");
-    if (p.kv_f32) DP_LAUNCH(ctx, attn_split_generic_kernel<float>, grid, 128, 0, p, scratch, splits);
-    else DP_LAUNCH(ctx, attn_split_generic_kernel<__half>, grid, 128, 0, p, scratch, splits);
+    const int most = p.head_dim > p.v_dim ? p.head_dim : p.v_dim;
+    if (most > 1024) return dp_fail(ctx, DP_ERR_UNSUPPORTED, "attention: head sizes above 1024");
+    if (most > 512) {
+      if (p.kv_f32) DP_LAUNCH(ctx, (attn_split_generic_kernel<float, 32>), grid, 128, 0, p, scratch, splits);
+      else DP_LAUNCH(ctx, (attn_split_generic_kernel<__half, 32>), grid, 128, 0, p, scratch, splits);
+    } else {
+      if (p.kv_f32) DP_LAUNCH(ctx, (attn_split_generic_kernel<float, 16>), grid, 128, 0, p, scratch, splits);
+      else DP_LAUNCH(ctx, (attn_split_generic_kernel<__half, 16>), grid, 128, 0, p, scratch, splits);
+    }
   }
   if (splits > 1 && combine) {
     const unsigned rows = (unsigned)((long)p.batch * p.seq_len * p.num_heads);

@@ -238,6 +238,7 @@ struct dpk_attn_params {
   int v_dim = 0;             // value size per head (0: head_dim); other sizes, and f32 caches, run on the generic kernel
   bool kv_f32 = false;       // k and v point at f32 caches
   size_t v_batch_stride = 0; // elements between the sequences of v (0: kv_batch_stride)
+  int v_row_stride = 0;      // elements between the values of two keys (0: num_kv_heads * v_dim): values that are part of the key rows
   // output gate: row r's head h times sigmoid(gate[r * gate_stride + h]); null: none (kernels that write `out` only)
   const float *gate = nullptr;
   int gate_stride = 0;

@@ -10,6 +10,9 @@
 // gemm_bf16w_f32_kernel (f32 activations): the 32-bit mode.  bf16 weights are exact in f32; every product and sum is
 // an f32 FMA on the CUDA cores.
 //
+// dpk_gemm_f16_tc: the same kernel with f16 operands and an f16 result.
+//
+// Optional decay: exp(-rate softplus(c + bias)) of every product is stored instead of the product.
 // Optional gated activation: weight rows in groups of sixteen (eight gate rows, then their eight up rows) and
 // g' sigmoid(slope g') (u' + shift) with g' = min(g, limit), u' = clamp(u, +-limit) stored in A's type.
 #include "layers.h"
@@ -45,17 +48,24 @@ __device__ __forceinline__ float glu_act_fast(float g, float u, const GluArgs &a
   return __fdividef(g, 1.0f + __expf(-a.slope * g)) * (u + a.shift);
 }
 
+__device__ __forceinline__ float decay_of(float c, float rate, float bias) {
+  const float z = c + bias;
+  return expf(-rate * (fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z)))));
+}
+
 constexpr int BT_THREADS = 256, BT_MAX_STAGES = 8;
 constexpr uint32_t BT_W_TILE = 128u * 128u;  // 128 weight rows x 64 bf16
 
 struct TcArgs {
   float *C;
-  int M, N, K, bn, stages, tiles_n, tiles_m, tmem_cols;
+  __half *C16;   // f16 operands and result (rows of c_stride elements)
+  int M, N, K, bn, stages, tiles_n, tiles_m, tmem_cols, c_stride;
   GluArgs glu;
+  DecayOut decay;
 };
 
-__device__ __forceinline__ uint32_t idesc_bf16(int M, int N) {  // D = f32, A = B = bf16, both K-major
-  return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(M >> 4) << 24);
+__device__ __forceinline__ uint32_t idesc_16(int M, int N, bool f16) {  // D = f32, A = B = bf16 or f16, both K-major
+  return (1u << 4) | (f16 ? 0u : (1u << 7) | (1u << 10)) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(M >> 4) << 24);
 }
 
 __global__ void __launch_bounds__(BT_THREADS, 1) gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_a,
@@ -115,7 +125,7 @@ __global__ void __launch_bounds__(BT_THREADS, 1) gemm_bf16_tc_kernel(const __gri
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      const uint32_t idesc = idesc_bf16(128, a.bn);
+      const uint32_t idesc = idesc_16(128, a.bn, a.C16 != nullptr);
       uint32_t it = 0, n = 0;
       bool ok = true;
       for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x, n++) {
@@ -164,7 +174,19 @@ __global__ void __launch_bounds__(BT_THREADS, 1) gemm_bf16_tc_kernel(const __gri
             const int row = m0 + c0 + i + (is_up ? 1 : 0);
             if (f < a.N && row < a.M) dst[(size_t)row * a.glu.stride] = __float2bfloat16_rn(glu_act_fast(gv, uv, a.glu));
           }
+        } else if (a.C16) {
+          if (f < a.N) {
+            __half *dst = a.C16 + (size_t)(m0 + c0) * a.c_stride + f;
+#pragma unroll
+            for (int i = 0; i < 16; i++)
+              if (m0 + c0 + i < a.M) dst[(size_t)i * a.c_stride] = __float2half_rn(__uint_as_float(r[i]));
+          }
         } else if (f < a.N) {
+          if (a.decay.rate) {
+            const float rate = a.decay.rate[f], bias = a.decay.bias[f];
+#pragma unroll 4
+            for (int i = 0; i < 16; i++) r[i] = __float_as_uint(decay_of(__uint_as_float(r[i]), rate, bias));
+          }
           float *dst = a.C + (size_t)(m0 + c0) * a.N + f;
 #pragma unroll
           for (int i = 0; i < 16; i++)
@@ -185,7 +207,7 @@ __global__ void __launch_bounds__(BT_THREADS, 1) gemm_bf16_tc_kernel(const __gri
 // ---- 32-bit mode ----
 constexpr int FM = 64, FN = 64, FK = 16;
 __global__ void __launch_bounds__(256) gemm_bf16w_f32_kernel(const __nv_bfloat16 *__restrict__ W, int w_stride, const float *__restrict__ A, int a_stride,
-                                                             float *__restrict__ C, int M, int N, int K, const GluArgs glu) {
+                                                             float *__restrict__ C, int M, int N, int K, const GluArgs glu, const DecayOut decay) {
   pdl_launch();
   pdl_wait();
   __shared__ float sa[FK][FM + 4], sw[FK][FN + 4];
@@ -217,7 +239,10 @@ __global__ void __launch_bounds__(256) gemm_bf16w_f32_kernel(const __nv_bfloat16
     for (int i = 0; i < 4; i++)
 #pragma unroll
       for (int j = 0; j < 4; j++)
-        if (m0 + ty * 4 + i < M && n0 + tx * 4 + j < N) C[(size_t)(m0 + ty * 4 + i) * N + n0 + tx * 4 + j] = acc[i][j];
+        if (m0 + ty * 4 + i < M && n0 + tx * 4 + j < N) {
+          const int n = n0 + tx * 4 + j;
+          C[(size_t)(m0 + ty * 4 + i) * N + n] = decay.rate ? decay_of(acc[i][j], decay.rate[n], decay.bias[n]) : acc[i][j];
+        }
     return;
   }
 #pragma unroll
@@ -252,20 +277,15 @@ int pick_rows(dp_ctx *ctx, int M, int tiles_n) {
   return best;
 }
 
-}  // namespace
-
-dp_status dpk_gemm_bf16_tc(dp_ctx *ctx, const __nv_bfloat16 *W, int w_stride, const __nv_bfloat16 *A, int a_stride, float *C, int M, int N, int K,
-                           const GluOut *glu) {
+// shape, strides and outputs are in `a`; the rest is chosen here
+dp_status launch_tc(dp_ctx *ctx, const void *W, int w_stride, const void *A, int a_stride, TcArgs a) {
+  const int M = a.M, N = a.N, K = a.K;
   DP_CHECK(ctx, w_stride % 8 == 0 && a_stride % 8 == 0 && K <= w_stride && K <= a_stride && M > 0 && N > 0 && K > 0, "gemm (bf16): bad shape or stride");
-  DP_CHECK(ctx, !glu || N % 16 == 0, "gemm (bf16): gate and up rows come in groups of sixteen");
   EncodeTiledFn encode = get_encode();
   if (!encode) return dp_fail(ctx, DP_ERR_CUDA, "gemm (bf16): cuTensorMapEncodeTiled is not available");
-  TcArgs a;
-  a.C = C; a.M = M; a.N = N; a.K = K;
   a.tiles_n = (N + 127) / 128;
   a.bn = pick_rows(ctx, M, a.tiles_n);
   a.tiles_m = (M + a.bn - 1) / a.bn;
-  a.glu = glu_args(glu);
   const uint32_t stage_bytes = BT_W_TILE + (uint32_t)a.bn * 128u;
   const size_t budget = ctx->smem_optin - 2048;
   int stages = (int)((budget - 1024) / stage_bytes);
@@ -273,15 +293,16 @@ dp_status dpk_gemm_bf16_tc(dp_ctx *ctx, const __nv_bfloat16 *W, int w_stride, co
   a.stages = stages;
   a.tmem_cols = 32;
   while (a.tmem_cols < 2 * a.bn) a.tmem_cols *= 2;
+  const CUtensorMapDataType type = a.C16 ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   CUtensorMap tw, ta;
   const cuuint32_t estr[2] = {1, 1};
   const cuuint64_t wd[2] = {(cuuint64_t)K, (cuuint64_t)N}, ad[2] = {(cuuint64_t)K, (cuuint64_t)M};
   const cuuint64_t ws[1] = {(cuuint64_t)w_stride * 2}, as[1] = {(cuuint64_t)a_stride * 2};
   const cuuint32_t wb[2] = {BK, 128}, ab[2] = {BK, (cuuint32_t)a.bn};
-  CUresult r = encode(&tw, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (void *)W, wd, ws, wb, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+  CUresult r = encode(&tw, type, 2, (void *)W, wd, ws, wb, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
                       CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r == CUDA_SUCCESS)
-    r = encode(&ta, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (void *)A, ad, as, ab, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+    r = encode(&ta, type, 2, (void *)A, ad, as, ab, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
                CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   if (r != CUDA_SUCCESS) return dp_fail(ctx, DP_ERR_CUDA, "gemm (bf16): cuTensorMapEncodeTiled failed (%d) for [%d,%d] x [%d,%d]", (int)r, M, K, N, K);
   static dp_per_device_once attr;
@@ -294,10 +315,29 @@ dp_status dpk_gemm_bf16_tc(dp_ctx *ctx, const __nv_bfloat16 *W, int w_stride, co
   return DP_OK;
 }
 
+}  // namespace
+
+dp_status dpk_gemm_bf16_tc(dp_ctx *ctx, const __nv_bfloat16 *W, int w_stride, const __nv_bfloat16 *A, int a_stride, float *C, int M, int N, int K,
+                           const GluOut *glu, const DecayOut *decay) {
+  DP_CHECK(ctx, !glu || N % 16 == 0, "gemm (bf16): gate and up rows come in groups of sixteen");
+  TcArgs a = {};
+  a.C = C; a.M = M; a.N = N; a.K = K;
+  a.glu = glu_args(glu);
+  if (decay) a.decay = *decay;
+  return launch_tc(ctx, W, w_stride, A, a_stride, a);
+}
+
+dp_status dpk_gemm_f16_tc(dp_ctx *ctx, const __half *W, int w_stride, const __half *A, int a_stride, __half *C, int c_stride, int M, int N, int K) {
+  TcArgs a = {};
+  a.C16 = C; a.c_stride = c_stride; a.M = M; a.N = N; a.K = K;
+  return launch_tc(ctx, W, w_stride, A, a_stride, a);
+}
+
 dp_status dpk_gemm_bf16w_f32(dp_ctx *ctx, const __nv_bfloat16 *W, int w_stride, const float *A, int a_stride, float *C, int M, int N, int K,
-                             const GluOut *glu) {
+                             const GluOut *glu, const DecayOut *decay) {
   DP_CHECK(ctx, M > 0 && N > 0 && K > 0, "gemm (bf16 weights, f32): bad shape");
   DP_CHECK(ctx, !glu || N % 16 == 0, "gemm (bf16): gate and up rows come in groups of sixteen");
-  DP_LAUNCH(ctx, gemm_bf16w_f32_kernel, dim3((N + FN - 1) / FN, (M + FM - 1) / FM), 256, 0, W, w_stride, A, a_stride, C, M, N, K, glu_args(glu));
+  DP_LAUNCH(ctx, gemm_bf16w_f32_kernel, dim3((N + FN - 1) / FN, (M + FM - 1) / FM), 256, 0, W, w_stride, A, a_stride, C, M, N, K, glu_args(glu),
+            decay ? *decay : DecayOut());
   return DP_OK;
 }

@@ -9,6 +9,9 @@
 //   NORM     grouped RMSNorm of a row, then (where the sublayer has one) the causal input convolution over the
 //            sequence's history; CTA 0 appends the row to the history.  The history is a ring of `taps` positions, so
 //            the slot written is none of the slots read.
+//   RESIDUAL x + out norm(y) of the sublayer that ended (y has a norm of its own, one stream), then NORM; CTA 0 stores the
+//            sum to another buffer than the one that is read
+//   GATED    NORM (its weight may serve every group), times the sigmoid of a gate per value
 //   ATTN     merge of the split-K attention partials, times the per-head output gate
 //   STREAMS  x_t <- sum_s mix[s][t] x_s + out[t] y for the warp's rows, and u = sum_t in[t] x_t of the next sublayer
 //   GLU      gated activation of a gate row and its up row
@@ -72,6 +75,7 @@ __device__ __forceinline__ void gb_conv_past(const GemvBf16 &p, float *past, uin
 
 // x (in shared memory) = input convolution of the grouped RMSNorm of p.x.  Every warp owns whole groups or an equal
 // part of one, so the scale of its channels is one number.
+template <int SRC>
 __device__ __forceinline__ void gb_prologue_norm(const GemvBf16 &p, float *sx, int plane, float *red, const float *past, const uint32_t *fac) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int groups = p.norm.groups, gs = p.K / groups, taps = p.norm.taps;
@@ -81,12 +85,64 @@ __device__ __forceinline__ void gb_prologue_norm(const GemvBf16 &p, float *sx, i
   const int part_len = ((gs / unit + parts - 1) / parts) * unit;
   const int tasks = groups * parts;
   const bool keep = taps > 1 && blockIdx.x == 0;
+  const bool gate4 = SRC == GEMV_SRC_GATED && ((uintptr_t)p.gate & 15) == 0;
   float *slot = keep ? p.norm.hist + (size_t)(*p.pos % taps) * p.K : nullptr;
   for (int base = 0; base < tasks; base += GB_WARPS) {
     const int task = base + warp;
     const int g = task / parts, c_lo = g * gs + (task - g * parts) * part_len, c_hi = min(c_lo + part_len, (g + 1) * gs);
     float ss = 0.0f;
-    if (task < tasks) {
+    if constexpr (SRC == GEMV_SRC_RESIDUAL) {
+      // the sum, into shared memory; res.groups equals groups
+      float sy = 0.0f;
+      if (task < tasks) {
+        if (vec) {
+#pragma unroll 4
+          for (int c = c_lo + lane * 4; c < c_hi; c += 128) {
+            const float4 v = gb_ld4(p.res_y + c);
+            *reinterpret_cast<float4 *>(sx + gb_slot(c, plane)) = v;
+            sy = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, sy))));
+          }
+        } else {
+          for (int c = c_lo + lane; c < c_hi; c += 32) {
+            const float v = p.res_y[c];
+            sx[gb_slot(c, plane)] = v;
+            sy = fmaf(v, v, sy);
+          }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) sy += __shfl_xor_sync(0xffffffffu, sy, o);
+      }
+      if (lane == 0) red[GB_WARPS + warp] = sy;
+      __syncthreads();
+      if (task < tasks) {
+        float total = 0.0f;
+        for (int i = 0; i < parts; i++) total += red[GB_WARPS + (warp / parts) * parts + i];
+        const float f = p.res.out[0] / sqrtf(total / (float)gs + p.res.eps);
+        const float mix = p.res.mix[0];
+        if (vec) {
+#pragma unroll 4
+          for (int c = c_lo + lane * 4; c < c_hi; c += 128) {
+            float4 *slot4 = reinterpret_cast<float4 *>(sx + gb_slot(c, plane));
+            const float4 y = *slot4, x = gb_ld4(p.x + c);
+            float w[4];
+            gb_w4(p.res.norm_w + c, w);
+            const float4 v = make_float4(fmaf(mix, x.x, f * y.x * w[0]), fmaf(mix, x.y, f * y.y * w[1]), fmaf(mix, x.z, f * y.z * w[2]), fmaf(mix, x.w, f * y.w * w[3]));
+            *slot4 = v;
+            if (blockIdx.x == 0) *reinterpret_cast<float4 *>(p.x_out + c) = v;
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+          }
+        } else {
+          for (int c = c_lo + lane; c < c_hi; c += 32) {
+            const float v = fmaf(mix, p.x[c], f * sx[gb_slot(c, plane)] * __bfloat162float(p.res.norm_w[c]));
+            sx[gb_slot(c, plane)] = v;
+            if (blockIdx.x == 0) p.x_out[c] = v;
+            ss = fmaf(v, v, ss);
+          }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      }
+    } else if (task < tasks) {
       if (vec) {
 #pragma unroll 4
         for (int c = c_lo + lane * 4; c < c_hi; c += 128) {
@@ -125,11 +181,25 @@ __device__ __forceinline__ void gb_prologue_norm(const GemvBf16 &p, float *sx, i
               if (keep) slot[c + i] = h;
               v[i] = h + fmaf(__uint_as_float(f & 0xffff0000u), h, past[c + i]);
             }
-        } else if (vec) {
-          gb_w4(p.norm.norm_w + c, w);
+        } else {
+          const __nv_bfloat16 *nw = p.norm.norm_w + (SRC == GEMV_SRC_GATED && p.norm_w_shared ? c - g * gs : c);
+          if (vec) {
+            gb_w4(nw, w);
 #pragma unroll
-          for (int i = 0; i < 4; i++) v[i] = v[i] * inv * w[i];
-        } else v[0] = v[0] * inv * __bfloat162float(p.norm.norm_w[c]);
+            for (int i = 0; i < 4; i++) v[i] = v[i] * inv * w[i];
+          } else v[0] = v[0] * inv * __bfloat162float(*nw);
+        }
+        if constexpr (SRC == GEMV_SRC_GATED) {
+          if (vec && gate4) {
+            const float4 q = gb_ld4(p.gate + c);
+            v[0] *= 1.0f / (1.0f + expf(-q.x)); v[1] *= 1.0f / (1.0f + expf(-q.y));
+            v[2] *= 1.0f / (1.0f + expf(-q.z)); v[3] *= 1.0f / (1.0f + expf(-q.w));
+          } else {
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+              if (i < unit) v[i] *= 1.0f / (1.0f + expf(-p.gate[c + i]));
+          }
+        }
         if (vec) *reinterpret_cast<float4 *>(sx + gb_slot(c, plane)) = make_float4(v[0], v[1], v[2], v[3]);
         else sx[gb_slot(c, plane)] = v[0];
       }
@@ -203,7 +273,7 @@ __device__ __forceinline__ uint4 gb_ldw(const uint4 *p) {
 template <int SRC, int DST>
 __global__ void __launch_bounds__(GB_THREADS, 2) gemv_bf16_kernel(const GemvBf16 p) {
   extern __shared__ __align__(16) float gb_sx[];
-  __shared__ float red[GB_WARPS];
+  __shared__ float red[2 * GB_WARPS];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int pieces = p.w_stride >> 3;      // 16-byte pieces per row
   const int plane = pieces * 4;            // floats per plane
@@ -218,13 +288,14 @@ __global__ void __launch_bounds__(GB_THREADS, 2) gemv_bf16_kernel(const GemvBf16
     if (lane < 2 && pair0 < pairs && row_bytes) gb_prefetch_l2(p.w + (size_t)(lane ? row_b(pair0) : row_a(pair0)) * p.w_stride, row_bytes);
   }
   for (int k = p.K + tid; k < pieces * 8; k += GB_THREADS) gb_sx[gb_slot(k, plane)] = 0.0f;  // the padded tail
-  if constexpr (SRC == GEMV_SRC_NORM)
+  constexpr bool NORMS = SRC == GEMV_SRC_NORM || SRC == GEMV_SRC_RESIDUAL || SRC == GEMV_SRC_GATED;
+  if constexpr (NORMS)
     if (p.norm.taps > 0) gb_conv_past(p, extra, reinterpret_cast<uint32_t *>(extra) + p.K);
   pdl_wait();
   pdl_launch();  // not before the wait: the next kernel's early work then competes with this kernel's stream only
-  if constexpr (SRC == GEMV_SRC_NORM) {
+  if constexpr (NORMS) {
     if (p.norm.taps > 0) __syncthreads();
-    gb_prologue_norm(p, gb_sx, plane, red, extra, reinterpret_cast<const uint32_t *>(extra) + p.K);
+    gb_prologue_norm<SRC>(p, gb_sx, plane, red, extra, reinterpret_cast<const uint32_t *>(extra) + p.K);
   } else if constexpr (SRC == GEMV_SRC_ATTN) {
     gb_prologue_attn(p, gb_sx, plane, extra);
   } else {
@@ -293,7 +364,7 @@ __global__ void __launch_bounds__(GB_THREADS, 2) gemv_bf16_kernel(const GemvBf16
 template <int SRC, int DST>
 dp_status launch(dp_ctx *ctx, const GemvBf16 &p) {
   size_t smem = (size_t)p.w_stride * 4;
-  if (SRC == GEMV_SRC_NORM && p.norm.taps > 0) smem += (size_t)p.K * 8;
+  if (SRC != GEMV_SRC_PLAIN && SRC != GEMV_SRC_ATTN && p.norm.taps > 0) smem += (size_t)p.K * 8;
   if (SRC == GEMV_SRC_ATTN) smem += (size_t)p.heads * p.splits * 4;
   if (smem > ctx->smem_optin - 1024)
     return dp_fail(ctx, DP_ERR_UNSUPPORTED, "gemv (bf16): a vector of %d values exceeds shared memory", p.K);
@@ -318,5 +389,9 @@ dp_status dpk_gemv_bf16(dp_ctx *ctx, int src, int dst, const GemvBf16 &p) {
   if (src == GEMV_SRC_NORM && dst == GEMV_DST_GLU) return launch<GEMV_SRC_NORM, GEMV_DST_GLU>(ctx, p);
   if (src == GEMV_SRC_NORM && dst == GEMV_DST_STREAMS) return launch<GEMV_SRC_NORM, GEMV_DST_STREAMS>(ctx, p);
   if (src == GEMV_SRC_ATTN && dst == GEMV_DST_STREAMS) return launch<GEMV_SRC_ATTN, GEMV_DST_STREAMS>(ctx, p);
+  if (src == GEMV_SRC_ATTN && dst == GEMV_DST_PLAIN) return launch<GEMV_SRC_ATTN, GEMV_DST_PLAIN>(ctx, p);
+  if (src == GEMV_SRC_RESIDUAL && dst == GEMV_DST_PLAIN) return launch<GEMV_SRC_RESIDUAL, GEMV_DST_PLAIN>(ctx, p);
+  if (src == GEMV_SRC_RESIDUAL && dst == GEMV_DST_GLU) return launch<GEMV_SRC_RESIDUAL, GEMV_DST_GLU>(ctx, p);
+  if (src == GEMV_SRC_GATED && dst == GEMV_DST_PLAIN) return launch<GEMV_SRC_GATED, GEMV_DST_PLAIN>(ctx, p);
   return dp_fail(ctx, DP_ERR_UNSUPPORTED, "gemv (bf16): no kernel for source %d and destination %d", src, dst);
 }

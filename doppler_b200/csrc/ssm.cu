@@ -3,6 +3,8 @@
 // with x, B and C through a causal depthwise convolution and silu first, dt = softplus(dt + bias), B and C shared by
 // the heads of a group.
 //
+// The same kernels run linear attention with a constant decay per head (see SsmShape): no convolution, step size 1.
+//
 // State layout: [head][vdim][state_stride], the state index fastest and padded with zeros to 32 * 2^k, so that eight
 // lanes cover a column of the state with 16-byte pieces (lane s holds n = 4 s + 32 i + {0..3}) and reduce y over the
 // state with three shuffles.  A sequence at position 0 starts from zeros whatever its slot held before.
@@ -54,18 +56,18 @@ __global__ void __launch_bounds__(SSM_THREADS) ssm_step_kernel(const float *__re
     acc[j] = last[j] = 0.0f;
     if (ch >= 0) {
       const float *cw = w.conv + (size_t)ch * taps;
-      acc[j] = w.conv_b[ch];
-      last[j] = cw[taps - 1];
+      if (w.conv) acc[j] = w.conv_b[ch];
+      last[j] = w.conv ? cw[taps - 1] : 1.0f;
       for (int k = taps - 1; k > 0; k--)
         if (pos - k >= 0) acc[j] = fmaf(cw[taps - 1 - k], hist[(size_t)((pos - k) % taps) * CH + ch], acc[j]);
     }
   }
-  const float a = -expf(w.a_log[h]), dt_bias = w.dt_bias[h], dh = w.d[h];
+  const float a = w.a[h], dt_bias = w.decay ? 0.0f : w.dt_bias[h], dh = w.d ? w.d[h] : 0.0f, fixed = w.decay ? w.decay[h] : 0.0f;
   pdl_wait();
   pdl_launch();
-  const float dt_raw = pr[inner + CH + h];
+  const float dt_raw = w.decay ? 0.0f : pr[inner + CH + h];
   const int e = h * P + p0 + col;
-  const float z = sub == 0 && col < cols ? pr[e] : 0.0f;
+  const float z = sub == 0 && col < cols && sh.gated ? pr[e] : 0.0f;
 #pragma unroll
   for (int j = 0; j < PER; j++) {
     const int i = tid + j * SSM_THREADS;
@@ -79,7 +81,7 @@ __global__ void __launch_bounds__(SSM_THREADS) ssm_step_kernel(const float *__re
       sv[i] = val;
     }
   }
-  const float dt = ssm_softplus(dt_raw + dt_bias), decay = expf(a * dt);
+  const float dt = w.decay ? 1.0f : ssm_softplus(dt_raw + dt_bias), decay = w.decay ? fixed : expf(a * dt);
   __syncthreads();
   const float x = sv[2 * NP + col], xdt = dt * x;
   float y = 0.0f;
@@ -93,7 +95,7 @@ __global__ void __launch_bounds__(SSM_THREADS) ssm_step_kernel(const float *__re
   }
 #pragma unroll
   for (int o = 4; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-  if (sub == 0 && col < cols) out[(size_t)row * inner + e] = fmaf(dh, x, y) * ssm_silu(z);
+  if (sub == 0 && col < cols) out[(size_t)row * inner + e] = sh.gated ? fmaf(dh, x, y) * ssm_silu(z) : fmaf(dh, x, y);
 }
 
 // ---- several tokens of one sequence: convolution and step sizes ----
@@ -117,8 +119,8 @@ __device__ __forceinline__ void conv_dt(const float *proj, int proj_stride, cons
   for (int r = r0; r < r1; r++) dt[(size_t)r * sh.heads + h] = ssm_softplus(proj[(size_t)r * proj_stride + col0 + h] + w.dt_bias[h]);
 }
 
-// four taps, four neighbouring channels per thread (channel counts and row strides that are multiples of four)
-template <typename OutT>
+// up to four taps, four neighbouring channels per thread (channel counts and row strides that are multiples of four)
+template <int TAPS, typename OutT>
 __global__ void __launch_bounds__(128) ssm_conv4_kernel(const float *__restrict__ proj, int proj_stride, const SsmShape sh, const SsmWeights w, const SsmState st,
                                                         OutT *__restrict__ xbc, float *__restrict__ dt, int rows, int start_pos, int seq) {
   pdl_launch();
@@ -128,7 +130,7 @@ __global__ void __launch_bounds__(128) ssm_conv4_kernel(const float *__restrict_
   const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, rows);
   if (ch >= CH) {
     const int h = idx - CH / 4;
-    if (h < sh.heads) conv_dt(proj, proj_stride, sh, w, inner + CH, h, dt, r0, r1);
+    if (h < sh.heads && w.dt_bias) conv_dt(proj, proj_stride, sh, w, inner + CH, h, dt, r0, r1);
     return;
   }
   const float *col = proj + inner + ch;
@@ -136,24 +138,38 @@ __global__ void __launch_bounds__(128) ssm_conv4_kernel(const float *__restrict_
   auto raw = [&](int r) -> float4 {
     if (r >= 0) return *reinterpret_cast<const float4 *>(col + (size_t)r * proj_stride);
     const int p = start_pos + r;
-    return p >= 0 ? *reinterpret_cast<const float4 *>(hist + (size_t)(p & 3) * CH + ch) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    return p >= 0 ? *reinterpret_cast<const float4 *>(hist + (size_t)(p % TAPS) * CH + ch) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
   };
-  float4 wv[4];  // the four taps of each channel
+  float wv[4][TAPS], bias[4];  // the taps of each channel
 #pragma unroll
-  for (int i = 0; i < 4; i++) wv[i] = *reinterpret_cast<const float4 *>(w.conv + (size_t)(ch + i) * 4);
-  const float4 bias = *reinterpret_cast<const float4 *>(w.conv_b + ch);
-  float4 a = raw(r0 - 3), b = raw(r0 - 2), c = raw(r0 - 1);
+  for (int i = 0; i < 4; i++) {
+    bias[i] = w.conv ? w.conv_b[ch + i] : 0.0f;
+    if constexpr (TAPS == 4) {
+      const float4 v = *reinterpret_cast<const float4 *>(w.conv + (size_t)(ch + i) * 4);
+      wv[i][0] = v.x; wv[i][1] = v.y; wv[i][2] = v.z; wv[i][3] = v.w;
+    } else {
+#pragma unroll
+      for (int k = 0; k < TAPS; k++) wv[i][k] = w.conv ? w.conv[(size_t)(ch + i) * TAPS + k] : 1.0f;
+    }
+  }
+  float4 win[TAPS];  // rows r - (TAPS - 1) .. r
+#pragma unroll
+  for (int k = 0; k + 1 < TAPS; k++) win[k + 1] = raw(r0 - (TAPS - 1) + k);
 #pragma unroll 8
   for (int r = r0; r < r1; r++) {
-    const float4 d = *reinterpret_cast<const float4 *>(col + (size_t)r * proj_stride);
-    float o[4];
-    o[0] = conv_silu<OutT>(fmaf(wv[0].w, d.x, fmaf(wv[0].z, c.x, fmaf(wv[0].y, b.x, fmaf(wv[0].x, a.x, bias.x)))));
-    o[1] = conv_silu<OutT>(fmaf(wv[1].w, d.y, fmaf(wv[1].z, c.y, fmaf(wv[1].y, b.y, fmaf(wv[1].x, a.y, bias.y)))));
-    o[2] = conv_silu<OutT>(fmaf(wv[2].w, d.z, fmaf(wv[2].z, c.z, fmaf(wv[2].y, b.z, fmaf(wv[2].x, a.z, bias.z)))));
-    o[3] = conv_silu<OutT>(fmaf(wv[3].w, d.w, fmaf(wv[3].z, c.w, fmaf(wv[3].y, b.w, fmaf(wv[3].x, a.w, bias.w)))));
+#pragma unroll
+    for (int k = 0; k + 1 < TAPS; k++) win[k] = win[k + 1];
+    win[TAPS - 1] = *reinterpret_cast<const float4 *>(col + (size_t)r * proj_stride);
+    float o[4] = {bias[0], bias[1], bias[2], bias[3]};
+#pragma unroll
+    for (int k = 0; k < TAPS; k++) {
+      o[0] = fmaf(wv[0][k], win[k].x, o[0]); o[1] = fmaf(wv[1][k], win[k].y, o[1]);
+      o[2] = fmaf(wv[2][k], win[k].z, o[2]); o[3] = fmaf(wv[3][k], win[k].w, o[3]);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++) o[i] = conv_silu<OutT>(o[i]);
     conv_store4(xbc + (size_t)r * CH + ch, o);
-    a = b; b = c; c = d;
-    if (r >= rows - 3) *reinterpret_cast<float4 *>(st.stage + (size_t)((start_pos + r) & 3) * CH + ch) = d;
+    if (TAPS > 1 && r >= rows - (TAPS - 1)) *reinterpret_cast<float4 *>(st.stage + (size_t)((start_pos + r) % TAPS) * CH + ch) = win[TAPS - 1];
   }
 }
 
@@ -167,7 +183,7 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const float *__restrict__
   const int ch = blockIdx.x * 128 + threadIdx.x;
   const int r0 = blockIdx.y * CONV_ROWS, r1 = min(r0 + CONV_ROWS, rows);
   if (ch >= CH) {
-    if (ch < CH + sh.heads) conv_dt(proj, proj_stride, sh, w, inner + CH, ch - CH, dt, r0, r1);
+    if (ch < CH + sh.heads && w.dt_bias) conv_dt(proj, proj_stride, sh, w, inner + CH, ch - CH, dt, r0, r1);
     return;
   }
   const float *col = proj + inner + ch;
@@ -179,8 +195,9 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const float *__restrict__
   };
   const float *cw = w.conv + (size_t)ch * taps;
   for (int r = r0; r < r1; r++) {
-    float acc = w.conv_b[ch];
-    for (int j = 0; j < taps; j++) acc = fmaf(cw[j], raw(r - (taps - 1) + j), acc);
+    float acc = w.conv ? w.conv_b[ch] : raw(r);
+    if (w.conv)
+      for (int j = 0; j < taps; j++) acc = fmaf(cw[j], raw(r - (taps - 1) + j), acc);
     conv_store(xbc + (size_t)r * CH + ch, conv_silu<OutT>(acc));
     if (r >= rows - (taps - 1)) st.stage[(size_t)((start_pos + r) % taps) * CH + ch] = raw(r);
   }
@@ -209,7 +226,7 @@ __global__ void __launch_bounds__(SSM_THREADS) ssm_scan_kernel(const float *__re
   auto stage = [&](int blk) {
     float *dst = scan_smem + (blk & 1) * SCAN_TB * TOK;
     const int r0 = blk * SCAN_TB, n = min(SCAN_TB, rows - r0);
-    const int per = 2 * N + cols + 1;
+    const int per = 2 * N + cols + (w.decay ? 0 : 1);
     for (int i = tid; i < n * per; i += SSM_THREADS) {
       const int t = i / per, e = i - t * per;
       const float *src = xbc + (size_t)(r0 + t) * CH;
@@ -225,7 +242,7 @@ __global__ void __launch_bounds__(SSM_THREADS) ssm_scan_kernel(const float *__re
   float4 *S = reinterpret_cast<float4 *>(st.s + (size_t)seq * st.s_seq + ((size_t)h * P + p0 + col) * NP) + sub;
 #pragma unroll
   for (int i = 0; i < NV; i++) v[i] = (col < cols && start_pos > 0) ? S[8 * i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-  const float a = -expf(w.a_log[h]), dh = w.d[h];
+  const float a = w.a[h], dh = w.d ? w.d[h] : 0.0f, fixed = w.decay ? w.decay[h] : 0.0f;
   const int blocks = (rows + SCAN_TB - 1) / SCAN_TB;
   stage(0);
   for (int blk = 0; blk < blocks; blk++) {
@@ -241,7 +258,7 @@ __global__ void __launch_bounds__(SSM_THREADS) ssm_scan_kernel(const float *__re
 #pragma unroll 2
     for (int t = 0; t < n; t++) {
       const float *d = src + t * TOK;
-      const float step = d[2 * NP + SSM_COLS], decay = expf(a * step), x = d[2 * NP + col], xdt = step * x;
+      const float step = w.decay ? 1.0f : d[2 * NP + SSM_COLS], decay = w.decay ? fixed : expf(a * step), x = d[2 * NP + col], xdt = step * x;
       float y = 0.0f;
 #pragma unroll
       for (int i = 0; i < NV; i++) {
@@ -259,13 +276,21 @@ __global__ void __launch_bounds__(SSM_THREADS) ssm_scan_kernel(const float *__re
       const int t = i / SSM_COLS, c = i - t * SSM_COLS;
       if (c < cols) {
         const int e = h * P + p0 + c;
-        out[(size_t)(r0 + t) * inner + e] = sy[i] * ssm_silu(proj[(size_t)(r0 + t) * proj_stride + e]);
+        out[(size_t)(r0 + t) * inner + e] = sh.gated ? sy[i] * ssm_silu(proj[(size_t)(r0 + t) * proj_stride + e]) : sy[i];
       }
     }
   }
   if (col < cols)
 #pragma unroll
     for (int i = 0; i < NV; i++) S[8 * i] = v[i];
+}
+
+template <typename KB, typename KF>
+dp_status launch_conv(dp_ctx *ctx, bool bf16, KB kb, KF kf, dim3 grid, const float *proj, int proj_stride, const SsmShape &sh, const SsmWeights &w,
+                      const SsmState &st, void *xbc, float *dt, int rows, const RowMap &map) {
+  if (bf16) DP_LAUNCH(ctx, kb, grid, 128, 0, proj, proj_stride, sh, w, st, (__nv_bfloat16 *)xbc, dt, rows, map.start_pos, map.seq);
+  else DP_LAUNCH(ctx, kf, grid, 128, 0, proj, proj_stride, sh, w, st, (float *)xbc, dt, rows, map.start_pos, map.seq);
+  return DP_OK;
 }
 
 template <int NV>
@@ -307,14 +332,18 @@ dp_status dpk_ssm_step(dp_ctx *ctx, const float *proj, int proj_stride, const Ss
 dp_status dpk_ssm_conv(dp_ctx *ctx, const float *proj, int proj_stride, const SsmShape &sh, const SsmWeights &w, const SsmState &st, void *xbc, bool bf16,
                        float *dt, int rows, const RowMap &map) {
   const int inner = sh.heads * sh.vdim, CH = inner + 2 * sh.groups * sh.state;
-  const bool four = sh.taps == 4 && CH % 4 == 0 && inner % 4 == 0 && proj_stride % 4 == 0;
+  const bool four = sh.taps <= 4 && CH % 4 == 0 && inner % 4 == 0 && proj_stride % 4 == 0;
   const int threads = (four ? CH / 4 : CH) + sh.heads;
   const dim3 grid((threads + 127) / 128, (rows + CONV_ROWS - 1) / CONV_ROWS);
-#define DP_CONV(K, T) DP_LAUNCH(ctx, K<T>, grid, 128, 0, proj, proj_stride, sh, w, st, (T *)xbc, dt, rows, map.start_pos, map.seq)
-  if (four) { if (bf16) DP_CONV(ssm_conv4_kernel, __nv_bfloat16); else DP_CONV(ssm_conv4_kernel, float); }
-  else { if (bf16) DP_CONV(ssm_conv_kernel, __nv_bfloat16); else DP_CONV(ssm_conv_kernel, float); }
+  if (!four) return launch_conv(ctx, bf16, ssm_conv_kernel<__nv_bfloat16>, ssm_conv_kernel<float>, grid, proj, proj_stride, sh, w, st, xbc, dt, rows, map);
+#define DP_CONV(T) launch_conv(ctx, bf16, ssm_conv4_kernel<T, __nv_bfloat16>, ssm_conv4_kernel<T, float>, grid, proj, proj_stride, sh, w, st, xbc, dt, rows, map)
+  switch (sh.taps) {
+    case 1: return DP_CONV(1);
+    case 2: return DP_CONV(2);
+    case 3: return DP_CONV(3);
+  }
+  return DP_CONV(4);
 #undef DP_CONV
-  return DP_OK;
 }
 
 dp_status dpk_ssm_scan(dp_ctx *ctx, const float *proj, int proj_stride, const float *xbc, const float *dt, const SsmShape &sh, const SsmWeights &w,

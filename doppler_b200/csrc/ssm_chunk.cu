@@ -1,6 +1,6 @@
 // Mamba-2 recurrence over a portion of a prompt in chunks of 64 tokens, on the tensor cores.
 //
-// With c_t the running sum of a dt within the chunk (a = -exp(a_log)) and S the state before it, the recurrence unrolls to
+// With c_t the running sum of a dt within the chunk (a = -exp(A_log), or ln(decay) with dt = 1) and S the state before it, the recurrence unrolls to
 //   y_t = exp(c_t) S^T C_t + sum_{s <= t} exp(c_t - c_s) dt_s (C_t . B_s) x_s
 //   S'  = exp(c_end) S + sum_s exp(c_end - c_s) dt_s B_s x_s^T
 // (the chunked form of Dao and Gu, "Transformers are SSMs", 2024).  x, B and C, the activations of the short
@@ -103,7 +103,7 @@ __global__ void __launch_bounds__((CkLayout<N, PB>::THREADS), PB > 32 ? 1 : 2) s
   const int grp = h / (sh.heads / G);
   const int pblk = warp / TW, tw = warp % TW;
   const int chunks = (rows + CQ - 1) / CQ;
-  const float a2 = -expf(w.a_log[h]) * 1.4426950408889634f, dh = w.d[h];
+  const float a2 = w.a[h] * 1.4426950408889634f, dh = w.d ? w.d[h] : 0.0f;
   float *s_cum = reinterpret_cast<float *>(ck_raw + L::CUM), *s_wt = s_cum + CQ;
 
   auto stage = [&](int chunk) {
@@ -129,7 +129,8 @@ __global__ void __launch_bounds__((CkLayout<N, PB>::THREADS), PB > 32 ? 1 : 2) s
     }
     if (tid < CQ) {
       const bool ok = r0 + tid < rows;
-      asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(base + L::DT + tid * 4), "l"(dt + (size_t)(ok ? r0 + tid : 0) * sh.heads + h),
+      if (w.decay) *reinterpret_cast<float *>(ck_raw + (base - sm) + L::DT + tid * 4) = ok ? 1.0f : 0.0f;
+      else asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(base + L::DT + tid * 4), "l"(dt + (size_t)(ok ? r0 + tid : 0) * sh.heads + h),
                    "r"(ok ? 4 : 0) : "memory");
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -180,7 +181,7 @@ __global__ void __launch_bounds__((CkLayout<N, PB>::THREADS), PB > 32 ? 1 : 2) s
 #pragma unroll
       for (int e = 0; e < 4; e++) {
         const int t = (tw * TT + j) * 8 + 2 * t4 + (e & 1), p = h * P + p0 + pblk * 16 + g + 8 * (e >> 1);
-        z[j][e] = t < n_tok ? proj[(size_t)(r0 + t) * proj_stride + p] : 0.0f;
+        z[j][e] = t < n_tok && sh.gated ? proj[(size_t)(r0 + t) * proj_stride + p] : 0.0f;
       }
 
     // ---- c_t: every warp computes all of them and stores the same values ----
@@ -338,7 +339,8 @@ __global__ void __launch_bounds__((CkLayout<N, PB>::THREADS), PB > 32 ? 1 : 2) s
         const int t = (tw * TT + j) * 8 + 2 * t4 + (e & 1), p = pblk * 16 + g + 8 * (e >> 1);
         if (t < n_tok) {
           const float x = __bfloat162float(*reinterpret_cast<const __nv_bfloat16 *>(basep + L::X + t * L::PROW + p * 2));
-          out[(size_t)(r0 + t) * inner + h * P + p0 + p] = fmaf(dh, x, y[j][e]) * ck_silu(z[j][e]);
+          const float v = fmaf(dh, x, y[j][e]);
+          out[(size_t)(r0 + t) * inner + h * P + p0 + p] = sh.gated ? v * ck_silu(z[j][e]) : v;
         }
       }
     if (L::STAGES == 1 && chunk + 1 < chunks) {

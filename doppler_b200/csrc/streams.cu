@@ -101,7 +101,18 @@ __global__ void __launch_bounds__(SB_THREADS, 2) stream_boundary_kernel(const Bo
     const float *xr = a.x + (size_t)row * S * H + c0;
     float *xo = a.x_out + (size_t)row * S * H + c0;
     const bool store = a.y && j >= halo;
-    float ss = 0.0f;
+    float ss = 0.0f, y_inv = 1.0f;
+    if (a.end.norm_w) {  // what the sublayer hands over passes a norm of its own
+      float sy = 0.0f;
+      for (int c = lane * V; c < gs; c += 32 * V) {
+        const FV<V> yv = ldv<V>(a.y + (size_t)row * H + c0 + c);
+#pragma unroll
+        for (int i = 0; i < V; i++) sy = fmaf(yv.v[i], yv.v[i], sy);
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) sy += __shfl_xor_sync(0xffffffffu, sy, o);
+      y_inv = 1.0f / sqrtf(sy / (float)gs + a.end.eps);
+    }
 #pragma unroll(SM <= 4 ? 2 : 1)
     for (int c = lane * V; c < gs; c += 32 * V) {
       FV<V> xs[SM], u;
@@ -111,7 +122,12 @@ __global__ void __launch_bounds__(SB_THREADS, 2) stream_boundary_kernel(const Bo
       for (int s = 0; s < SM; s++)
         if (s < S) xs[s] = ldv<V>(xr + (size_t)s * H + c);
       if (a.y) {
-        const FV<V> yv = ldv<V>(a.y + (size_t)row * H + c0 + c);
+        FV<V> yv = ldv<V>(a.y + (size_t)row * H + c0 + c);
+        if (a.end.norm_w) {
+          const FV<V> w = ldw<V>(a.end.norm_w + c0 + c);
+#pragma unroll
+          for (int i = 0; i < V; i++) yv.v[i] = yv.v[i] * y_inv * w.v[i];
+        }
 #pragma unroll
         for (int t = 0; t < SM; t++) {
           if (t < S) {
@@ -201,6 +217,125 @@ dp_status launch_boundary(dp_ctx *ctx, const BoundaryArgs &a, void *dst, bool bf
   return DP_OK;
 }
 
+// One stream, one norm group, no input convolution: a CTA per row, the row in registers (at most 4 * 256 * MAXV values).
+// x_out (optional) <- mix x + out norm(y); dst (optional) <- RMSNorm of that.
+template <int MAXV, typename OutT>
+__global__ void __launch_bounds__(256) stream_row_kernel(const float *__restrict__ x, float *__restrict__ x_out, const float *__restrict__ y, const SublayerOut end,
+                                                         const SublayerIn next, int H, OutT *__restrict__ dst, int dst_stride) {
+  pdl_launch();
+  pdl_wait();
+  __shared__ float sh[16];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const size_t base = (size_t)blockIdx.x * H;
+  auto block_sum = [&](float v, float *red) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    if (lane == 0) red[warp] = v;
+    __syncthreads();
+    float t = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 8; i++) t += red[i];
+    return t;
+  };
+  FV<4> v[MAXV], yv[MAXV];
+#pragma unroll
+  for (int j = 0; j < MAXV; j++) {
+    const int c = (tid + 256 * j) * 4;
+    v[j] = c < H ? ldv<4>(x + base + c) : FV<4>{};
+    yv[j] = y && c < H ? ldv<4>(y + base + c) : FV<4>{};
+  }
+  if (y) {
+    float y_inv = 1.0f;
+    if (end.norm_w) {
+      float sy = 0.0f;
+#pragma unroll
+      for (int j = 0; j < MAXV; j++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) sy = fmaf(yv[j].v[i], yv[j].v[i], sy);
+      y_inv = 1.0f / sqrtf(block_sum(sy, sh) / (float)H + end.eps);
+    }
+    const float mix = end.mix[0], out = end.out[0];
+#pragma unroll
+    for (int j = 0; j < MAXV; j++) {
+      const int c = (tid + 256 * j) * 4;
+      if (c < H) {
+        FV<4> w = {{1.0f, 1.0f, 1.0f, 1.0f}};
+        if (end.norm_w) w = ldw<4>(end.norm_w + c);
+#pragma unroll
+        for (int i = 0; i < 4; i++) v[j].v[i] = fmaf(mix, v[j].v[i], out * (yv[j].v[i] * y_inv * w.v[i]));
+        if (x_out) stv<4>(x_out + base + c, v[j]);
+      }
+    }
+  }
+  if (!dst) return;
+  float ss = 0.0f;
+  const float in = next.in[0];
+#pragma unroll
+  for (int j = 0; j < MAXV; j++)
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      v[j].v[i] *= in;
+      ss = fmaf(v[j].v[i], v[j].v[i], ss);
+    }
+  const float inv = 1.0f / sqrtf(block_sum(ss, sh + 8) / (float)H + next.eps);
+#pragma unroll
+  for (int j = 0; j < MAXV; j++) {
+    const int c = (tid + 256 * j) * 4;
+    if (c < H) {
+      const FV<4> w = ldw<4>(next.norm_w + c);
+#pragma unroll
+      for (int i = 0; i < 4; i++) v[j].v[i] = v[j].v[i] * inv * w.v[i];
+      stv<4>(dst + (size_t)blockIdx.x * dst_stride + c, v[j]);
+    }
+  }
+}
+
+template <typename OutT>
+dp_status launch_row(dp_ctx *ctx, const float *x, float *x_out, const float *y, const SublayerOut &end, const SublayerIn &next, int H, OutT *dst, int dst_stride,
+                     int rows) {
+  if (H <= 1024) DP_LAUNCH(ctx, (stream_row_kernel<1, OutT>), rows, 256, 0, x, x_out, y, end, next, H, dst, dst_stride);
+  else if (H <= 2048) DP_LAUNCH(ctx, (stream_row_kernel<2, OutT>), rows, 256, 0, x, x_out, y, end, next, H, dst, dst_stride);
+  else if (H <= 4096) DP_LAUNCH(ctx, (stream_row_kernel<4, OutT>), rows, 256, 0, x, x_out, y, end, next, H, dst, dst_stride);
+  else DP_LAUNCH(ctx, (stream_row_kernel<8, OutT>), rows, 256, 0, x, x_out, y, end, next, H, dst, dst_stride);
+  return DP_OK;
+}
+
+// the streams' sum of a row after y has been written into them, y through its grouped norm: one CTA per row
+__global__ void __launch_bounds__(256) stream_sum_norm_kernel(const float *__restrict__ x, const float *__restrict__ y, const SublayerOut end, int S, int H,
+                                                              float *__restrict__ h) {
+  pdl_launch();
+  pdl_wait();
+  __shared__ float red[8], s_inv;
+  const int tid = threadIdx.x, gs = H / end.groups;
+  const float *yr = y + (size_t)blockIdx.x * H;
+  float w_out = 0.0f;
+  for (int t = 0; t < S; t++) w_out += end.out[t];
+  for (int g = 0; g < end.groups; g++) {
+    float sy = 0.0f;
+    for (int c = tid; c < gs; c += 256) sy = fmaf(yr[g * gs + c], yr[g * gs + c], sy);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sy += __shfl_xor_sync(0xffffffffu, sy, o);
+    if ((tid & 31) == 0) red[tid >> 5] = sy;
+    __syncthreads();
+    if (tid == 0) {
+      float t = 0.0f;
+      for (int i = 0; i < 8; i++) t += red[i];
+      s_inv = 1.0f / sqrtf(t / (float)gs + end.eps);
+    }
+    __syncthreads();
+    for (int c = g * gs + tid; c < (g + 1) * gs; c += 256) {
+      float v = w_out * (yr[c] * s_inv * __bfloat162float(end.norm_w[c]));
+      for (int s = 0; s < S; s++) {
+        float m = 0.0f;
+        for (int t = 0; t < S; t++) m += end.mix[s * S + t];
+        v = fmaf(m, x[((size_t)blockIdx.x * S + s) * H + c], v);
+      }
+      h[(size_t)blockIdx.x * H + c] = v;
+    }
+    __syncthreads();
+  }
+}
+
 __global__ void __launch_bounds__(256) stream_sum_kernel(const float *__restrict__ x, const float *__restrict__ y, const SublayerOut end, int S, int H,
                                                          float *__restrict__ h, int rows) {
   pdl_launch();
@@ -242,12 +377,19 @@ __global__ void __launch_bounds__(256) stream_embed_kernel(const int *__restrict
   }
 }
 
+template <int V> __device__ __forceinline__ void gate_by(FV<V> &v, const float *gate) {
+  const FV<V> g = ldv<V>(gate);
+#pragma unroll
+  for (int i = 0; i < V; i++) v.v[i] *= 1.0f / (1.0f + expf(-g.v[i]));
+}
+
 // one warp per (row, part), the part in registers (parts of at most 128 * MAXV values, all sizes multiples of four)
 template <int MAXV, typename OutT>
-__global__ void __launch_bounds__(256) group_norm_warp_kernel(const float *__restrict__ x, int x_stride, const __nv_bfloat16 *__restrict__ w, int groups, int gs,
-                                                              float eps, OutT *__restrict__ dst, int dst_stride, int rows) {
+__global__ void __launch_bounds__(256) group_norm_warp_kernel(const float *__restrict__ x, int x_stride, const GroupNorm n, int gs, OutT *__restrict__ dst,
+                                                              int dst_stride, int rows) {
   pdl_launch();
   pdl_wait();
+  const int groups = n.groups;
   const int lane = threadIdx.x & 31, part = blockIdx.x * 8 + (threadIdx.x >> 5);
   if (part >= rows * groups) return;
   const int row = part / groups, c0 = (part - row * groups) * gs;
@@ -266,23 +408,25 @@ __global__ void __launch_bounds__(256) group_norm_warp_kernel(const float *__res
     for (int i = 0; i < 4; i++) ss = fmaf(v[j].v[i], v[j].v[i], ss);
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  const float inv = 1.0f / sqrtf(ss / (float)gs + eps);
+  const float inv = 1.0f / sqrtf(ss / (float)gs + n.eps);
   OutT *d = dst + (size_t)row * dst_stride + c0;
+  const __nv_bfloat16 *w = n.w + (n.w_shared ? 0 : c0);
 #pragma unroll
   for (int j = 0; j < MAXV; j++) {
     const int c = (lane + 32 * j) * 4;
     if (c < gs) {
-      const FV<4> wv = ldw<4>(w + c0 + c);
+      const FV<4> wv = ldw<4>(w + c);
 #pragma unroll
       for (int i = 0; i < 4; i++) v[j].v[i] = v[j].v[i] * inv * wv.v[i];
+      if (n.gate) gate_by(v[j], n.gate + (size_t)row * n.gate_stride + c0 + c);
       stv<4>(d + c, v[j]);
     }
   }
 }
 
 template <int V, typename OutT>
-__global__ void __launch_bounds__(256) group_norm_kernel(const float *__restrict__ x, int x_stride, const __nv_bfloat16 *__restrict__ w, int gs, float eps,
-                                                         OutT *__restrict__ dst, int dst_stride) {
+__global__ void __launch_bounds__(256) group_norm_kernel(const float *__restrict__ x, int x_stride, const GroupNorm n, int gs, OutT *__restrict__ dst,
+                                                         int dst_stride) {
   pdl_launch();
   pdl_wait();
   __shared__ float sh[8];
@@ -302,13 +446,15 @@ __global__ void __launch_bounds__(256) group_norm_kernel(const float *__restrict
   float t = 0.0f;
 #pragma unroll
   for (int i = 0; i < 8; i++) t += sh[i];
-  const float inv = 1.0f / sqrtf(t / (float)gs + eps);
+  const float inv = 1.0f / sqrtf(t / (float)gs + n.eps);
   OutT *d = dst + (size_t)blockIdx.x * dst_stride + c0;
+  const __nv_bfloat16 *w = n.w + (n.w_shared ? 0 : c0);
   for (int c = tid * V; c < gs; c += 256 * V) {
     FV<V> v = c == tid * V ? first : ldv<V>(xr + c);
-    const FV<V> wv = ldw<V>(w + c0 + c);
+    const FV<V> wv = ldw<V>(w + c);
 #pragma unroll
     for (int i = 0; i < V; i++) v.v[i] = v.v[i] * inv * wv.v[i];
+    if (n.gate) gate_by(v, n.gate + (size_t)blockIdx.x * n.gate_stride + c0 + c);
     stv<V>(d + c, v);
   }
 }
@@ -333,6 +479,9 @@ unsigned flat_grid(dp_ctx *ctx, size_t n) {
 
 dp_status dpk_stream_boundary(dp_ctx *ctx, const float *x, float *x_out, const float *y, const SublayerOut &end, const SublayerIn &next, int streams, int width,
                               void *dst, bool dst_bf16, int dst_stride, int rows, const RowMap &map) {
+  if (streams == 1 && next.groups == 1 && next.taps == 0 && end.groups == 1 && width % 4 == 0 && width <= 8192 && dst_stride % 4 == 0)
+    return dst_bf16 ? launch_row(ctx, x, x_out, y, end, next, width, (__nv_bfloat16 *)dst, dst_stride, rows)
+                    : launch_row(ctx, x, x_out, y, end, next, width, (float *)dst, dst_stride, rows);
   const int gs = width / next.groups;
   const int halo = (map.pos || next.taps < 2) ? 0 : next.taps - 1;
   const size_t row_bytes = (size_t)gs * 4;
@@ -361,6 +510,12 @@ dp_status dpk_stream_boundary(dp_ctx *ctx, const float *x, float *x_out, const f
 }
 
 dp_status dpk_stream_sum(dp_ctx *ctx, const float *x, const float *y, const SublayerOut &end, int streams, int width, float *h, int rows) {
+  if (end.norm_w && streams == 1 && end.groups == 1 && width % 4 == 0 && width <= 8192)
+    return launch_row(ctx, x, h, y, end, SublayerIn(), width, (float *)nullptr, 0, rows);
+  if (end.norm_w) {
+    DP_LAUNCH(ctx, stream_sum_norm_kernel, rows, 256, 0, x, y, end, streams, width, h);
+    return DP_OK;
+  }
   DP_LAUNCH(ctx, stream_sum_kernel, flat_grid(ctx, (size_t)rows * width), 256, 0, x, y, end, streams, width, h, rows);
   return DP_OK;
 }
@@ -371,18 +526,18 @@ dp_status dpk_stream_embed(dp_ctx *ctx, const int *ids, const __nv_bfloat16 *tab
   return DP_OK;
 }
 
-dp_status dpk_group_norm(dp_ctx *ctx, const float *x, int x_stride, const __nv_bfloat16 *w, int groups, float eps, int width, void *dst, bool dst_bf16,
-                         int dst_stride, int rows) {
-  const dim3 grid(rows, groups);
-  const int gs = width / groups;
-  const bool vec = gs % 4 == 0 && x_stride % 4 == 0 && dst_stride % 4 == 0;
+dp_status dpk_group_norm(dp_ctx *ctx, const float *x, int x_stride, const GroupNorm &n, int width, void *dst, bool dst_bf16, int dst_stride, int rows) {
+  const dim3 grid(rows, n.groups);
+  const int gs = width / n.groups;
+  const bool aligned = ((uintptr_t)x & 15) == 0 && (!n.gate || (((uintptr_t)n.gate & 15) == 0 && n.gate_stride % 4 == 0));
+  const bool vec = gs % 4 == 0 && x_stride % 4 == 0 && dst_stride % 4 == 0 && aligned;
   if (vec && gs <= 1024) {
-    const unsigned blocks = (unsigned)(((size_t)rows * groups + 7) / 8);
-    if (dst_bf16) DP_LAUNCH(ctx, (group_norm_warp_kernel<8, __nv_bfloat16>), blocks, 256, 0, x, x_stride, w, groups, gs, eps, (__nv_bfloat16 *)dst, dst_stride, rows);
-    else DP_LAUNCH(ctx, (group_norm_warp_kernel<8, float>), blocks, 256, 0, x, x_stride, w, groups, gs, eps, (float *)dst, dst_stride, rows);
+    const unsigned blocks = (unsigned)(((size_t)rows * n.groups + 7) / 8);
+    if (dst_bf16) DP_LAUNCH(ctx, (group_norm_warp_kernel<8, __nv_bfloat16>), blocks, 256, 0, x, x_stride, n, gs, (__nv_bfloat16 *)dst, dst_stride, rows);
+    else DP_LAUNCH(ctx, (group_norm_warp_kernel<8, float>), blocks, 256, 0, x, x_stride, n, gs, (float *)dst, dst_stride, rows);
     return DP_OK;
   }
-#define DP_NORM(V, T) DP_LAUNCH(ctx, (group_norm_kernel<V, T>), grid, 256, 0, x, x_stride, w, gs, eps, (T *)dst, dst_stride)
+#define DP_NORM(V, T) DP_LAUNCH(ctx, (group_norm_kernel<V, T>), grid, 256, 0, x, x_stride, n, gs, (T *)dst, dst_stride)
   if (dst_bf16) { if (vec) DP_NORM(4, __nv_bfloat16); else DP_NORM(1, __nv_bfloat16); }
   else { if (vec) DP_NORM(4, float); else DP_NORM(1, float); }
 #undef DP_NORM

@@ -7,47 +7,35 @@ rotation, the gated feed-forward uses sigmoid(1.702 g) and u + 1, the head is th
 """
 from __future__ import annotations
 
-import os
 from typing import List, Tuple
 
 from . import _lib as L
-from .safetensors import SafetensorsFile
+from . import stack as st
+from .stack import ConfigError
 
 ARCHITECTURE = "Fenorax"
-WEIGHTS_FILE = "model.safetensors"
 FF_SLOPE, FF_SHIFT = 1.702, 1.0
-
-
-class ConfigError(Exception):
-    pass
-
-
-def _need(d: dict, where: str, *keys):
-    missing = [k for k in keys if k not in d]
-    if missing:
-        raise ConfigError(f"{where}: missing {', '.join(missing)}")
-    return [d[k] for k in keys]
 
 
 def layer_config(entry: dict, index: int) -> dict:
     """One entry of config 'layers' -> the fields of dp_layer_cfg."""
     where = f"layer {index}"
-    kind, m = _need(entry, where, "type", "mixer")
-    heads, vdim = _need(m, where, "heads", "vdim")
+    kind, m = st.need(entry, where, "type", "mixer")
+    heads, vdim = st.need(m, where, "heads", "vdim")
     out = {"heads": heads, "vdim": vdim}
     if kind == "mamba2":
-        state, groups, conv, norm_groups = _need(m, where, "state", "groups", "conv", "norm_groups")
+        state, groups, conv, norm_groups = st.need(m, where, "state", "groups", "conv", "norm_groups")
         out.update(mixer=L.MIXER_MAMBA2, state=state, groups=groups, conv_taps=conv, norm_groups=norm_groups)
     elif kind == "attention":
-        kv_heads, dim, scale, mask = _need(m, where, "kv_heads", "dim", "scale", "mask")
-        out.update(mixer=L.MIXER_ATTENTION, kv_heads=kv_heads, dim=dim, scale=scale, chunk=_need(mask, where + " mask", "size")[0], unit_rms_qk=1, head_gate=1)
+        kv_heads, dim, scale, mask = st.need(m, where, "kv_heads", "dim", "scale", "mask")
+        out.update(mixer=L.MIXER_ATTENTION, kv_heads=kv_heads, dim=dim, scale=scale, chunk=st.need(mask, where + " mask", "size")[0], unit_rms_qk=1, head_gate=1)
     else:
         raise ConfigError(f"{where}: unknown type '{kind}'")
     mlp = entry.get("mlp")
     if mlp is not None:
         if mlp.get("kind") != "dense":
             raise ConfigError(f"{where}: unknown feed-forward '{mlp.get('kind')}'")
-        ff, limit = _need(mlp, where + " mlp", "ff", "limit")
+        ff, limit = st.need(mlp, where + " mlp", "ff", "limit")
         if not limit > 0:
             raise ConfigError(f"{where}: feed-forward limit {limit} must be positive")
         out.update(ff=ff, ff_limit=limit, ff_slope=FF_SLOPE, ff_shift=FF_SHIFT)
@@ -58,10 +46,10 @@ def stack_config(config: dict) -> Tuple[dict, List[dict]]:
     """config.json -> (stack fields, layer fields)."""
     if config.get("architecture") != ARCHITECTURE:
         raise ConfigError(f"architecture '{config.get('architecture')}' is not {ARCHITECTURE}")
-    width, vocab, streams, norm, canon, embedding, layers = _need(config, "config", "width", "vocab", "streams", "norm", "canon", "embedding", "layers")
-    eps, groups = _need(norm, "norm", "eps", "groups")
-    stack = {"width": width, "vocab": vocab, "streams": streams, "norm_groups": groups, "input_taps": _need(canon, "canon", "taps")[0], "eps": eps,
-             "embed_scale": _need(embedding, "embedding", "scale")[0]}
+    width, vocab, streams, norm, canon, embedding, layers = st.need(config, "config", "width", "vocab", "streams", "norm", "canon", "embedding", "layers")
+    eps, groups = st.need(norm, "norm", "eps", "groups")
+    stack = {"width": width, "vocab": vocab, "streams": streams, "norm_groups": groups, "input_taps": st.need(canon, "canon", "taps")[0], "eps": eps,
+             "embed_scale": st.need(embedding, "embedding", "scale")[0]}
     return stack, [layer_config(e, i) for i, e in enumerate(layers)]
 
 
@@ -89,28 +77,19 @@ def model_tensors(layers: List[dict]) -> List[Tuple[str, int, int]]:
 
 def load_weights(model, get):
     """Upload every tensor of the model; ``get(name)`` returns its bfloat16 bits."""
-    for name, layer, tid in model_tensors(model.layers):
-        model.load_tensor(layer, tid, get(name))
+    st.load_tensors(model, model_tensors(model.layers), get)
+
+
+def describe(path: str, config: dict) -> Tuple[dict, List[dict]]:
+    """The description of the model in a folder."""
+    return stack_config(config)
 
 
 def load(device, path: str, config: dict, max_seq: int, max_batch: int = 1, dtype: str = "bfloat16", max_rows: int = 0):
     """Open a model folder (config.json already read) and upload it."""
-    from .model import StackModel  # needs the CUDA library
-
-    stack, layers = stack_config(config)
-    weights = SafetensorsFile(os.path.join(path, WEIGHTS_FILE))
-
-    def get(name):
-        if name in weights and weights.dtype(name) != "BF16":
-            raise ConfigError(f"{name}: dtype {weights.dtype(name)}, expected BF16")
-        return weights.tensor(name)
-
-    model = StackModel(device, stack, layers, max_seq, max_batch, dtype, max_rows)
+    fields, layers = stack_config(config)
+    weights = st.open_weights(path)
     try:
-        load_weights(model, get)
-    except Exception:
-        model.destroy()
-        raise
+        return st.load(device, weights, fields, layers, model_tensors(layers), max_seq, max_batch, dtype, max_rows)
     finally:
         weights.close()
-    return model

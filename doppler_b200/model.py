@@ -164,15 +164,15 @@ class DecoderModel(Runner):
 
 class StackModel(Runner):
     """A decoder described layer by layer.  ``stack`` holds the fields of ``dp_stack_cfg`` that describe the model
-    (width, vocab, streams, norm_groups, input_taps, eps, embed_scale), ``layers`` one dictionary of ``dp_layer_cfg``
-    fields per layer.  ``dtype``: "bfloat16" (tensor cores, f16 K/V cache) or "float32" (every product in 32-bit)."""
+    (width, vocab, streams, norm_groups, input_taps, eps, embed_scale, post_norm, residual_mult), ``layers`` one dictionary
+    of ``dp_layer_cfg`` fields per layer (``decay`` a list).  ``dtype``: "bfloat16" (tensor cores, f16 K/V cache) or "float32" (every product in 32-bit)."""
 
     def __init__(self, device: Device, stack: dict, layers: list, max_seq: int, max_batch: int = 1, dtype: str = "bfloat16", max_rows: int = 0):
         self.device, self.max_batch, self.layers = device, max_batch, [dict(l) for l in layers]
         self.cfg = dict(stack, hidden=stack["width"], n_layers=len(layers), max_seq=max_seq)
         c = L.StackCfg(n_layers=len(layers), max_seq=max_seq, max_batch=max_batch, act_dtype={"bfloat16": L.BF16, "float32": L.F32}[dtype],
                        max_rows=max_rows, **stack)
-        arr = (L.LayerCfg * len(layers))(*[L.LayerCfg(**l) for l in layers])
+        arr = (L.LayerCfg * len(layers))(*[L.LayerCfg(**{k: (C.c_double * len(v))(*v) if k == "decay" else v for k, v in l.items()}) for l in layers])
         h = C.c_void_p()
         device.check(device.lib.dp_model_create_stack(device.h, C.byref(c), arr, C.byref(h)))
         self.h = h

@@ -7,9 +7,10 @@ from __future__ import annotations
 
 import json
 import os
-from typing import Callable, Dict
+from types import ModuleType
+from typing import Dict
 
-from . import fenorax
+from . import fenorax, virolorn
 
 DTYPES = ("bfloat16", "float32")
 
@@ -18,12 +19,9 @@ class UnknownModel(Exception):
     pass
 
 
-def _load_fenorax(device, path, config, max_seq, max_batch, dtype, max_rows):
-    return fenorax.load(device, path, config, max_seq, max_batch, dtype, max_rows)
-
-
-# architecture named by config.json -> loader(device, path, config, max_seq, max_batch, dtype, max_rows)
-ARCHITECTURES: Dict[str, Callable] = {fenorax.ARCHITECTURE: _load_fenorax}
+# architecture named by config.json -> the design's module: describe(path, config) and
+# load(device, path, config, max_seq, max_batch, dtype, max_rows)
+ARCHITECTURES: Dict[str, ModuleType] = {m.ARCHITECTURE: m for m in (fenorax, virolorn)}
 
 
 def describe(path: str) -> dict:
@@ -51,4 +49,4 @@ def load_model(device, path: str, max_seq: int, max_batch: int = 1, dtype: str =
         from .rdrr import load_decoder
 
         return load_decoder(device, path, max_seq, max_batch)
-    return ARCHITECTURES[d["kind"]](device, path, d["config"], max_seq, max_batch, dtype, max_rows)
+    return ARCHITECTURES[d["kind"]].load(device, path, d["config"], max_seq, max_batch, dtype, max_rows)

@@ -41,6 +41,10 @@ class SafetensorsFile:
     def dtype(self, name: str) -> str:
         return self.header[name]["dtype"]
 
+    def shape(self, name: str):
+        """A tensor's shape, None if there is none of that name."""
+        return tuple(self.header[name]["shape"]) if name in self.header else None
+
     def tensor(self, name: str) -> np.ndarray:
         if name not in self.header:
             raise SafetensorsError(f"{self.path}: no tensor '{name}'")

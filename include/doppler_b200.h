@@ -386,22 +386,41 @@ dp_status dp_model_set_allreduce_mode(dp_model *m, int mode);
  *   unit_rms_qk  q and k divided by their root mean square per head, no weight.
  *   head_gate    head h's output times sigmoid((W_g x)_h).
  *   ff           gated feed-forward: g = min(W_gate x, limit), u = clamp(W_up x, +-limit),
- *                W_down (g * sigmoid(slope * g) * (u + shift)).
+ *                W_down (g * sigmoid(slope * g) * (u + shift)); limit 0: no clamp.
+ *   post_norm    a sublayer's result y passes an RMSNorm of its own (norm1b, norm2b) before it is added (one stream).
+ *   residual_mult  factor of what a sublayer adds (one stream without loaded vectors).
+ *   share        n > 0: the layer has no tensors, it uses those of layer n - 1 (same description) with its own state.
+ * Mixers beside grouped-query attention and Mamba-2:
+ *   LIGHTNING    linear attention with one constant decay per head: q, k, v = silu of their projections,
+ *                S <- decay S + k v^T, o = S^T q; all heads normed together, times sigmoid(W_g x).
+ *   DELTA        gated delta rule with one decay per key channel: q, k, v through short convolutions and silu, q and k
+ *                made unit vectors (q also / sqrt(dim)), S <- g S; S <- S + k (beta (v - S^T k))^T; o = S^T q, with
+ *                g = exp(-exp(A_log) softplus(W_a2 W_a1 x + dt_bias)); heads normed one by one, times sigmoid(W_g2 W_g1 x).
+ *   LATENT       attention whose keys and values are linear in one low-rank vector per token, which is what the cache
+ *                holds, beside a rotated key part shared by the heads; queries come from a normed low-rank vector too.
  * Linear weights are bf16 [out, in].  act_dtype DP_BF16: matrix products of several rows on the tensor cores with
  * bf16 activations, K and V cached as f16; DP_F32: every product in 32-bit, K and V cached as f32.  Residual
  * streams, norms, scores, recurrent state and all vectors between kernels are f32 in both. */
-typedef enum { DP_MIXER_ATTENTION = 0, DP_MIXER_MAMBA2 = 1 } dp_mixer_kind;
+typedef enum { DP_MIXER_ATTENTION = 0, DP_MIXER_MAMBA2 = 1, DP_MIXER_LIGHTNING = 2, DP_MIXER_DELTA = 3, DP_MIXER_LATENT = 4 } dp_mixer_kind;
 typedef struct {
   int mixer; /* dp_mixer_kind */
   int heads, vdim;
   /* attention */
   int kv_heads, dim, chunk, unit_rms_qk, head_gate;
   float scale;
-  /* Mamba-2 */
+  /* Mamba-2 (conv_taps also the delta rule) */
   int state, groups, conv_taps, norm_groups;
   /* feed-forward; ff = 0: none */
   int ff;
   float ff_limit, ff_slope, ff_shift;
+  int share;
+  /* delta rule (with kv_heads, dim): sizes between the two matrices of the decay and of the output gate */
+  int decay_rank, gate_rank;
+  /* latent attention (with dim, vdim, scale, head_gate): low-rank sizes, rotated dimensions, their base */
+  int q_rank, kv_rank, rot_dim;
+  double rot_base;
+  /* lightning (with dim): one per head, copied */
+  const double *decay;
 } dp_layer_cfg;
 typedef struct {
   int n_layers, width, vocab, max_seq, max_batch;
@@ -409,6 +428,8 @@ typedef struct {
   float eps, embed_scale;
   int act_dtype; /* DP_BF16 or DP_F32 */
   int max_rows;  /* rows of one block of a portion (0: chosen from max_seq) */
+  int post_norm;
+  float residual_mult;  /* 0 counts as 1 */
 } dp_stack_cfg;
 typedef enum {
   DP_T_EMBED = 0, DP_T_FINAL_NORM,                           /* layer -1 */
@@ -417,6 +438,10 @@ typedef enum {
   DP_T_Q, DP_T_K, DP_T_V, DP_T_GATE_HEADS, DP_T_O,           /* attention; DP_T_O also Mamba-2 */
   DP_T_SSM_IN, DP_T_SSM_CONV, DP_T_SSM_CONV_B, DP_T_SSM_DT_BIAS, DP_T_SSM_A_LOG, DP_T_SSM_D, DP_T_SSM_NORM,
   DP_T_FF_GATE, DP_T_FF_UP, DP_T_FF_DOWN,
+  DP_T_NORM1B, DP_T_NORM2B,                                  /* norms behind the sublayers */
+  DP_T_GATE, DP_T_MIX_NORM,                                  /* lightning (W_g), norm of a mixer's heads (also delta) */
+  DP_T_CONV_Q, DP_T_CONV_K, DP_T_CONV_V, DP_T_BETA, DP_T_A1, DP_T_A2, DP_T_G1, DP_T_G2, DP_T_A_LOG, DP_T_DT_BIAS, /* delta */
+  DP_T_DQ, DP_T_DQ_NORM, DP_T_UQ, DP_T_DKV, DP_T_DKV_NORM, DP_T_UK, DP_T_UV,                  /* latent attention */
   DP_T_COUNT
 } dp_tensor_id;
 dp_status dp_model_create_stack(dp_ctx *ctx, const dp_stack_cfg *cfg, const dp_layer_cfg *layers, dp_model **out);
