@@ -21,7 +21,7 @@ roofline  the dominant kernels (the Q4_K decode GEMVs as the decode graph launch
 kernels   the other BASELINE configurations, a few ms each through the C ABI: config 0 GEMV (us),
           config 1 GEMM (TFLOP/s, fraction of the measured bf16 burst and sustained peaks),
           config 2 decode attention (GB/s, fraction of measured HBM).  N = 1 only.
---case stack (not part of the default line): prefill and decode of a Fenorax decoder at the same layer sizes, random
+--case stack (not part of the default line): prefill and decode of Virolorn and Fenorax decoders at the same layer sizes, random
           weights, beside the dense decoder.
 tokens_crc  CRC-32 of the tokens of the warm-up and the first timed region; every rank must hold
           the same tokens (checked), and the N = 1 and N = 8 lines can be compared.
@@ -337,6 +337,84 @@ STACK_SIZES = {
 }
 
 
+# Virolorn at the same widths: per group of layers a delta rule, lightning, a delta rule and latent attention, each with a
+# feed-forward chosen so that a decode step reads about as many weight bytes as Fenorax's
+def virolorn_config(size):
+    w, heads, ff, kv_rank, q_rank, rank = {"9b": (4096, 32, 6144, 512, 1536, 128), "0.6b": (1024, 8, 1536, 256, 768, 64)}[size]
+    mlp = {"kind": "dense", "ff": ff}
+    delta = {"type": "channel_delta", "mixer": {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4}, "mlp": mlp}
+    lightning = {"type": "lightning", "mixer": {"heads": heads, "dim": 128, "vdim": 128, "decay": [float(np.exp(-2.0 ** (-8.0 * (h + 1) / heads))) for h in range(heads)]},
+                 "mlp": mlp}
+    latent = {"type": "latent_attention", "mlp": mlp,
+              "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": kv_rank, "q_rank": q_rank, "scale": 192.0 ** -0.5,
+                        "rot": {"base": 1e6, "dims": 64}}}
+    cfg = {"architecture": "Virolorn", "width": w, "vocab": STACK_SIZES[size]["stack"]["vocab"], "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+           "layers": [delta, lightning, delta, latent] * STACK_SIZES[size]["groups"]}
+    return cfg, rank
+
+
+class RandomMatrices:
+    """Weights from one pool of seeded gaussians, cut at random places."""
+
+    def __init__(self, seed):
+        self.rng = np.random.default_rng(seed)
+        self.pool = self.rng.standard_normal(1 << 22).astype(np.float32)
+
+    def __call__(self, n, k):
+        from doppler_b200.safetensors import bf16_bits
+
+        bits = bf16_bits(self.pool / np.sqrt(k))
+        reps = -(-(n * k + bits.size) // bits.size)
+        return np.tile(bits, reps)[(o := int(self.rng.integers(bits.size))):o + n * k].reshape(n, k)
+
+
+def virolorn_model(dev, size, max_seq, seed=11):
+    """A Virolorn runner of one of the sizes, random weights."""
+    from doppler_b200 import virolorn
+    from doppler_b200.model import StackModel
+    from doppler_b200.safetensors import bf16_bits
+
+    cfg, rank = virolorn_config(size)
+    W, V = cfg["width"], cfg["vocab"]
+    mat = RandomMatrices(seed)
+
+    def shape(name):
+        if name == "embed":
+            return (V, W)
+        if name == "final.norm":
+            return (W,)
+        layer, part = name.split(".", 1)
+        e = cfg["layers"][int(layer[1:])]
+        m, ff = e["mixer"], e["mlp"]["ff"]
+        H, D, inner = m["heads"], m["dim"], m["heads"] * m["vdim"]
+        if part.startswith("norm"):
+            return (W,)
+        if part.startswith("mlp."):
+            return (W, ff) if part == "mlp.down" else (ff, W)
+        key = part[4:]
+        if key == "o":
+            return (W, inner)
+        if e["type"] == "lightning":
+            return {"q": (H * D, W), "k": (H * D, W), "v": (inner, W), "g": (inner, W), "norm": (inner,)}[key]
+        if e["type"] == "latent_attention":
+            R, K, Q = m["rot_dim"], m["kv_rank"], m["q_rank"]
+            return {"dq": (Q, W), "dq.norm": (Q,), "uq": (H * (D + R), Q), "dkv": (K + R, W), "dkv.norm": (K,), "uk": (H * D, K), "uv": (inner, K), "g": (H, W)}[key]
+        QK, taps = m["kv_heads"] * D, m["conv"]
+        return {"q": (QK, W), "k": (QK, W), "v": (inner, W), "q.conv": (QK, taps), "k.conv": (QK, taps), "v.conv": (inner, taps), "b": (H, W), "A_log": (H,),
+                "dt_bias": (H * D,), "a1": (rank, W), "a2": (H * D, rank), "g1": (rank, W), "g2": (inner, rank), "norm": (m["vdim"],)}[key]
+
+    def get(name):
+        s = shape(name)
+        if len(s) == 1:
+            return bf16_bits(np.full(s, -2.0 if name.endswith("dt_bias") else 0.0 if name.endswith("A_log") else 1.0))
+        return mat(*s)
+
+    fields, layers = virolorn.stack_config(cfg, shape)
+    m = StackModel(dev, fields, layers, max_seq)
+    virolorn.load_weights(m, get)
+    return m
+
+
 def stack_model(dev, size, max_seq, seed=11):
     """A Fenorax runner of one of STACK_SIZES; weights come from one pool of seeded gaussians, cut at random places."""
     from doppler_b200 import _lib as L
@@ -351,14 +429,9 @@ def stack_model(dev, size, max_seq, seed=11):
         layers.append(dict(z["attention"], mixer=L.MIXER_ATTENTION, scale=z["attention"]["dim"] ** -0.5, unit_rms_qk=1, head_gate=1, ff_limit=7.0,
                            ff_slope=fenorax.FF_SLOPE, ff_shift=fenorax.FF_SHIFT))
     m = StackModel(dev, z["stack"], layers, max_seq)
-    rng = np.random.default_rng(seed)
-    pool = rng.standard_normal(1 << 22).astype(np.float32)
+    mat = RandomMatrices(seed)
+    rng = mat.rng
     S, W = z["stack"]["streams"], z["stack"]["width"]
-
-    def mat(n, k):
-        bits = bf16_bits(pool / np.sqrt(k))
-        reps = -(-(n * k + bits.size) // bits.size)
-        return np.tile(bits, reps)[(o := int(rng.integers(bits.size))):o + n * k].reshape(n, k)
 
     m.load_tensor(-1, L.T_EMBED, mat(z["stack"]["vocab"], W))
     m.load_tensor(-1, L.T_FINAL_NORM, bf16_bits(np.ones(W)))
@@ -388,17 +461,17 @@ def stack_model(dev, size, max_seq, seed=11):
 
 
 def stack_case(args, dev, synthetic, peak):
-    """Prefill and decode of the layer-by-layer decoder, beside the dense Q4_K decoder of the same width, heads, feed-forward,
-    vocabulary and number of layers.  --shape: prompt tokens."""
+    """Prefill and decode of the layer-by-layer decoders, beside the dense Q4_K decoder of the same width, heads, feed-forward,
+    vocabulary and number of layers.  --shape: prompt tokens; --models: some of them only."""
     from doppler_b200.model import DecoderModel
 
     n = int(args.shape) if args.shape else 1024
     steps = args.steps
     for size in ([args.size] if args.size else sorted(STACK_SIZES)):
         z = STACK_SIZES[size]
-        for kind in ("fenorax", "dense_q4k"):
-            if kind == "fenorax":
-                m = stack_model(dev, size, n + 4 * steps + 64)
+        for kind in args.models.split(","):
+            if kind in ("fenorax", "virolorn"):
+                m = {"fenorax": stack_model, "virolorn": virolorn_model}[kind](dev, size, n + 4 * steps + 64)
             else:
                 m = DecoderModel(dev, dict(synthetic.MODEL_CONFIGS[z["dense"]], n_layers=4 * z["groups"]), n + 4 * steps + 64)
                 m.load_synthetic()
@@ -536,13 +609,14 @@ def main():
     ap.add_argument("--no-kernels", action="store_true", help="skip the config 0/1/2 kernel record")
     ap.add_argument("--case", default=None, choices=["gemv", "gemm", "attention", "prefill", "lm_head", "stack"],
                     help="time ONE kernel of the path on a BASELINE configuration instead of the decoder "
-                         "(gemv: configs 0 and 9B shapes, gemm: config 1, attention: config 2; stack: prefill and decode of a "
-                         "Fenorax decoder beside the dense one); also the small "
+                         "(gemv: configs 0 and 9B shapes, gemm: config 1, attention: config 2; stack: prefill and decode of the "
+                         "Virolorn and Fenorax decoders beside the dense one); also the small "
                          "command the profiler captures use")
     ap.add_argument("--shape", default=None, help="--case gemv/gemm: N,K or M,N,K; --case attention: batch,kv_len")
     ap.add_argument("--variant", default="default", choices=["default", "f16_weights"], help="--case gemm: exact product or f16-rounded weights")
     ap.add_argument("--adtype", default="f16", choices=["f16", "f32"], help="--case gemm: activation (and output) dtype")
     ap.add_argument("--size", default=None, choices=sorted(STACK_SIZES), help="--case stack: one layer size only")
+    ap.add_argument("--models", default="virolorn,fenorax,dense_q4k", help="--case stack: which models")
     ap.add_argument("--copies", type=int, default=0, help="--case: distinct weight copies per pass (0 = enough to exceed L2)")
     ap.add_argument("--only-timed", action="store_true",
                     help="stop after the first device-resident timed region (used for profiler launch lists)")

@@ -306,6 +306,11 @@ bool dpk_attention_uses_tc(dp_ctx *ctx, const dpk_attn_params &p) {
   return use_tc(ctx, p, &gt);
 }
 
+// one latent row per token shared by all heads (attention_latent.cu)
+bool dpk_attention_latent_eligible(dp_ctx *ctx, const dpk_attn_params &p);
+int dpk_attention_latent_splits(dp_ctx *ctx, const dpk_attn_params &p);
+dp_status dpk_attention_latent(dp_ctx *ctx, const dpk_attn_params &p, float *scratch, int splits);
+
 // the most keys one query row sees
 static long row_keys(const dpk_attn_params &p) { return p.chunk > 0 && p.chunk < p.kv_len ? p.chunk : p.kv_len; }
 
@@ -334,6 +339,11 @@ size_t dpk_attention_scratch_bytes(dp_ctx *ctx, const dpk_attn_params &p, int *s
     const int s = tc_splits(ctx, p, gt);
     *splits_out = s;
     return s == 1 ? 0 : (size_t)p.batch * p.seq_len * p.num_heads * s * (p.head_dim + 2) * sizeof(float);
+  }
+  if (dpk_attention_latent_eligible(ctx, p)) {
+    const int s = dpk_attention_latent_splits(ctx, p);
+    *splits_out = s;
+    return s == 1 ? 0 : (size_t)p.batch * p.seq_len * p.num_heads * s * (p.v_dim + 2) * sizeof(float);
   }
   const bool fast = fast_shape(p, &gt);
   const int G = p.num_heads / p.num_kv_heads;
@@ -380,8 +390,11 @@ static dp_status attention_impl(dp_ctx *ctx, const dpk_attn_params &p, float *sc
   int gt = 1;
   // several causal query rows: one CTA per tile of query positions shares each K / V tile (DP_ATTN_TC=0: off)
   static const int tc_mode = [] { const char *e = getenv("DP_ATTN_TC"); return e ? atoi(e) : 1; }();
-  if (tc_mode && combine && f16_square(p) && dpk_attention_prefill_eligible(p)) return dpk_attention_prefill(ctx, p);
-  if (use_tc(ctx, p, &gt)) {
+  if (tc_mode && combine && (p.k2 || f16_square(p)) && dpk_attention_prefill_eligible(p)) return dpk_attention_prefill(ctx, p);
+  if (p.k2) return dp_fail(ctx, DP_ERR_UNSUPPORTED, "attention: keys in two parts run on the prefill kernel only");
+  if (dpk_attention_latent_eligible(ctx, p)) {
+    DP_TRY(dpk_attention_latent(ctx, p, scratch, splits));
+  } else if (use_tc(ctx, p, &gt)) {
     DP_TRY(dpk_attention_tc_split(ctx, p, scratch, splits));
   } else if (fast_shape(p, &gt)) {
     if (p.head_dim == 128) {

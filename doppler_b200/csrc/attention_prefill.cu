@@ -1,4 +1,6 @@
-// Causal prefill attention over the f16 KV cache, query-tiled (head_dim 128, GQA groups of 1, 2, 4 or 8).
+// Causal prefill attention over f16 keys and values, query-tiled (GQA groups of 1, 2, 4 or 8).  Key and value sizes are
+// template parameters; smaller ones are padded with zeros on the way into shared memory.  A key may consist of two parts,
+// one per head and one that all heads share (the rotated part of latent attention), in different arrays.
 //
 // Replaces src/gpu/kernels/attention_streaming_f16kv.wgsl:96 (one thread per (query, head), two passes
 // over K) and, in this library, running every query row as its own CTA of the decode kernel, which
@@ -20,11 +22,13 @@
 
 #define APF_WARPS 8
 #define APF_THREADS (APF_WARPS * 32)
-#define APF_D 128
 #define APF_KT 32                       // keys per tile
-#define APF_ROWB (APF_D * 2 + 16)       // bytes per key row in shared memory
-#define APF_TILE (APF_KT * APF_ROWB)    // one K (or V) tile
-#define APF_STAGE (2 * APF_TILE)        // K tile then V tile
+
+template <int DK, int DV> struct ApfLayout {
+  static constexpr int KROW = DK * 2 + 16, VROW = DV * 2 + 16;  // bytes per row in shared memory
+  static constexpr int VTILE = APF_KT * KROW;                   // K tile, then V tile
+  static constexpr int STAGE = VTILE + APF_KT * VROW;
+};
 
 __device__ __forceinline__ void apf_cp_async16(uint32_t dst, const void *src, int src_bytes) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(src), "r"(src_bytes) : "memory");
@@ -46,9 +50,14 @@ __device__ __forceinline__ uint32_t apf_pack(float a, float b) {
 }
 
 // grid: (query tiles, KV heads, batch); G = num_heads / num_kv_heads in {1, 2, 4, 8}
+template <int DK, int DV>
 __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_attn_params p, int G) {
   pdl_launch();
   pdl_wait();
+  using L = ApfLayout<DK, DV>;
+  constexpr int KS = DK / 16, NV = DV / 8;
+  const int D = p.head_dim, V = p.v_dim ? p.v_dim : D;  // sizes of a query and of a value; keys: k_dim + k2_dim
+  const int kd = p.k2 ? p.k_dim : D, k_pieces = (kd + 7) / 8, k2_pieces = p.k2 ? (p.k2_dim + 7) / 8 : 0, v_pieces = (V + 7) / 8;
   extern __shared__ __align__(128) unsigned char apf_smem[];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g = lane >> 2, t = lane & 3;
@@ -74,42 +83,61 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
   const int tile0 = p.chunk > 0 ? (p.start_pos + qtile * QT) / p.chunk * p.chunk / APF_KT : 0;
   const int warp_lo = p.chunk > 0 ? (p.start_pos + q0) / p.chunk * p.chunk : 0;
 
-  const __half *kbase = p.k + (size_t)b * p.kv_batch_stride + (size_t)kvh * APF_D;
-  const __half *vbase = p.v + (size_t)b * p.kv_batch_stride + (size_t)kvh * APF_D;
-  const size_t key_stride = (size_t)p.num_kv_heads * APF_D;  // elements between consecutive keys
+  const __half *kbase = p.k + (size_t)b * p.kv_batch_stride + (size_t)kvh * k_pieces * 8;
+  const __half *vbase = p.v + (size_t)b * (p.v_batch_stride ? p.v_batch_stride : p.kv_batch_stride) + (size_t)kvh * v_pieces * 8;
+  const __half *k2base = p.k2 + (size_t)b * p.k2_batch_stride;
+  // elements between consecutive keys
+  const size_t key_stride = p.k_row_stride ? (size_t)p.k_row_stride : (size_t)p.num_kv_heads * D, val_stride = p.v_row_stride ? (size_t)p.v_row_stride : (size_t)p.num_kv_heads * V;
   const uint32_t smem0 = (uint32_t)__cvta_generic_to_shared(apf_smem);
 
   auto issue_tile = [&](int tile) {
     const int s = tile & 1;
     const int key0 = tile * APF_KT;
-    // 32 keys x 16 chunks of 16 bytes, for K and for V: two chunks of each per thread
+    const uint32_t dst = smem0 + (uint32_t)s * L::STAGE;
+    // 32 keys, 16-byte pieces; rows past the range and pieces past a part are zero filled
 #pragma unroll
-    for (int i = 0; i < 2; i++) {
-      const int c = tid + i * APF_THREADS;       // 0 .. 511
-      const int key = c >> 4, ch = c & 15;
-      const bool ok = key0 + key < cta_keys;
-      const size_t off = (size_t)(ok ? key0 + key : 0) * key_stride + (size_t)ch * 8;
-      const uint32_t dst = smem0 + (uint32_t)s * APF_STAGE + (uint32_t)key * APF_ROWB + (uint32_t)ch * 16;
-      apf_cp_async16(dst, kbase + off, ok ? 16 : 0);            // rows past the range are zero filled
-      apf_cp_async16(dst + APF_TILE, vbase + off, ok ? 16 : 0);
+    for (int i = 0; i < (APF_KT * DK / 8 + APF_THREADS - 1) / APF_THREADS; i++) {
+      const int c = tid + i * APF_THREADS, key = c / (DK / 8), ch = c % (DK / 8);
+      if (c < APF_KT * DK / 8) {
+        const bool in = key0 + key < cta_keys, first = ch < k_pieces, ok = in && ch < k_pieces + k2_pieces;
+        const size_t row = (size_t)(in ? key0 + key : 0);
+        const __half *src = first || !ok ? kbase + row * key_stride + (first ? ch * 8 : 0) : k2base + row * p.k2_row_stride + (ch - k_pieces) * 8;
+        apf_cp_async16(dst + (uint32_t)(key * L::KROW + ch * 16), src, ok ? 16 : 0);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < (APF_KT * DV / 8 + APF_THREADS - 1) / APF_THREADS; i++) {
+      const int c = tid + i * APF_THREADS, key = c / (DV / 8), ch = c % (DV / 8);
+      if (c < APF_KT * DV / 8) {
+        const bool in = key0 + key < cta_keys, ok = in && ch < v_pieces;
+        apf_cp_async16(dst + (uint32_t)(L::VTILE + key * L::VROW + ch * 16), vbase + (size_t)(in ? key0 + key : 0) * val_stride + (ok ? ch * 8 : 0), ok ? 16 : 0);
+      }
     }
     apf_commit();
   };
 
-  // ---- Q fragments (A operand, 16 rows x 128 dims): f16 hi and lo halves of scale * q ----
+  // ---- Q fragments (A operand, 16 rows x DK dims): f16 hi and lo halves of scale * q ----
   const float LOG2E = 1.4426950408889634f;
   const float qmul = p.scale * LOG2E;  // scores in log2 units: softmax with exp2
-  uint32_t qh[8][4], ql[8][4];
+  uint32_t qh[KS][4], ql[KS][4];
   {
     const bool okA = rowA < p.seq_len, okB = rowB < p.seq_len;
-    const float *qa = p.q + (((size_t)b * p.seq_len + (okA ? rowA : 0)) * p.num_heads + h) * APF_D;
-    const float *qb = p.q + (((size_t)b * p.seq_len + (okB ? rowB : 0)) * p.num_heads + h) * APF_D;
+    const float *qa = p.q + (((size_t)b * p.seq_len + (okA ? rowA : 0)) * p.num_heads + h) * D;
+    const float *qb = p.q + (((size_t)b * p.seq_len + (okB ? rowB : 0)) * p.num_heads + h) * D;
+    // a pair of dims where the keys have them: both parts of a key are padded to whole pieces, the query is not
+    auto pair = [&](const float *q, bool ok, int d) {
+      float2 v = make_float2(0.0f, 0.0f);
+      if (!ok) return v;
+      const int at = d < k_pieces * 8 ? d : kd + (d - k_pieces * 8), end = d < k_pieces * 8 ? kd : D;
+      if (at + 1 < end && (((D | at) & 1) == 0)) return *reinterpret_cast<const float2 *>(q + at);
+      if (at < end) v.x = q[at];
+      if (at + 1 < end) v.y = q[at + 1];
+      return v;
+    };
 #pragma unroll
-    for (int ks = 0; ks < 8; ks++) {
-      const float2 a0 = okA ? *reinterpret_cast<const float2 *>(qa + 16 * ks + 2 * t) : make_float2(0.f, 0.f);
-      const float2 a1 = okB ? *reinterpret_cast<const float2 *>(qb + 16 * ks + 2 * t) : make_float2(0.f, 0.f);
-      const float2 a2 = okA ? *reinterpret_cast<const float2 *>(qa + 16 * ks + 2 * t + 8) : make_float2(0.f, 0.f);
-      const float2 a3 = okB ? *reinterpret_cast<const float2 *>(qb + 16 * ks + 2 * t + 8) : make_float2(0.f, 0.f);
+    for (int ks = 0; ks < KS; ks++) {
+      const float2 a0 = pair(qa, okA, 16 * ks + 2 * t), a1 = pair(qb, okB, 16 * ks + 2 * t), a2 = pair(qa, okA, 16 * ks + 2 * t + 8),
+                   a3 = pair(qb, okB, 16 * ks + 2 * t + 8);
       const float x[8] = {a0.x * qmul, a0.y * qmul, a1.x * qmul, a1.y * qmul, a2.x * qmul, a2.y * qmul, a3.x * qmul, a3.y * qmul};
 #pragma unroll
       for (int j = 0; j < 4; j++) {
@@ -121,9 +149,9 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
     }
   }
 
-  float o[16][4];
+  float o[NV][4];
 #pragma unroll
-  for (int j = 0; j < 16; j++) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f; }
+  for (int j = 0; j < NV; j++) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.0f; }
   float mA = -INFINITY, mB = -INFINITY, lA = 0.0f, lB = 0.0f;  // running max (log2 units) and this lane's share of the running sum
 
   if (tile0 < n_tiles) issue_tile(tile0);
@@ -132,17 +160,17 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
     __syncthreads();
     const int key0 = tile * APF_KT;
     if (key0 < warp_keys && key0 + APF_KT > warp_lo) {  // (warp-uniform) other tiles are masked for all of this warp's rows
-      const unsigned char *sK = apf_smem + (tile & 1) * APF_STAGE;
-      const uint32_t sV = smem0 + (uint32_t)(tile & 1) * APF_STAGE + APF_TILE;
+      const unsigned char *sK = apf_smem + (tile & 1) * L::STAGE;
+      const uint32_t sV = smem0 + (uint32_t)(tile & 1) * L::STAGE + L::VTILE;
       // ---- S = (scale * Q) K^T for 16 rows x 32 keys ----
       float sc[4][4];
 #pragma unroll
       for (int nt = 0; nt < 4; nt++) { sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.0f; }
 #pragma unroll
-      for (int ks = 0; ks < 8; ks++) {
+      for (int ks = 0; ks < KS; ks++) {
 #pragma unroll
         for (int nt = 0; nt < 4; nt++) {
-          const unsigned char *kr = sK + (nt * 8 + g) * APF_ROWB + (16 * ks + 2 * t) * 2;
+          const unsigned char *kr = sK + (nt * 8 + g) * L::KROW + (16 * ks + 2 * t) * 2;
           const uint32_t b0 = *reinterpret_cast<const uint32_t *>(kr), b1 = *reinterpret_cast<const uint32_t *>(kr + 16);
           apf_mma(sc[nt], qh[ks], b0, b1);
           apf_mma(sc[nt], ql[ks], b0, b1);
@@ -178,7 +206,7 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
       lA = lA * cA + sA;
       lB = lB * cB + sB;
 #pragma unroll
-      for (int j = 0; j < 16; j++) { o[j][0] *= cA; o[j][1] *= cA; o[j][2] *= cB; o[j][3] *= cB; }
+      for (int j = 0; j < NV; j++) { o[j][0] *= cA; o[j][1] *= cA; o[j][2] *= cB; o[j][3] *= cB; }
       // ---- O += P V: P (16 x 32) as two A fragments, V fragments transposed out of shared memory ----
 #pragma unroll
       for (int kk = 0; kk < 2; kk++) {
@@ -191,9 +219,9 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
           pa[i] = *reinterpret_cast<const uint32_t *>(&hi);
           pl[i] = apf_pack(x0 - hf.x, x1 - hf.y);
         }
-        const uint32_t vrow = sV + (uint32_t)(16 * kk + (lane & 15)) * APF_ROWB;
+        const uint32_t vrow = sV + (uint32_t)(16 * kk + (lane & 15)) * L::VROW;
 #pragma unroll
-        for (int j = 0; j < 16; j++) {
+        for (int j = 0; j < NV; j++) {
           uint32_t b0, b1;
           apf_ldmatrix_x2_trans(b0, b1, vrow + (uint32_t)j * 16u);
           apf_mma(o[j], pa, b0, b1);
@@ -214,22 +242,38 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
     const size_t z = (size_t)b * p.seq_len + row;
     float inv = l > 0.0f ? 1.0f / l : 0.0f;
     if (p.gate) inv *= 1.0f / (1.0f + expf(-p.gate[z * p.gate_stride + h]));
-    if (p.out_bf16) {
-      __nv_bfloat16 *dst = p.out_bf16 + z * p.out_stride + (size_t)h * APF_D + 2 * t;
+    const bool whole = (V & 1) == 0;  // pairs do not straddle the end
+    auto put = [&](auto *dst, auto two, auto one) {
 #pragma unroll
-      for (int j = 0; j < 16; j++) *reinterpret_cast<__nv_bfloat162 *>(dst + 8 * j) = __floats2bfloat162_rn(o[j][2 * half] * inv, o[j][2 * half + 1] * inv);
-    } else {
-      float *dst = p.out + (z * p.num_heads + h) * APF_D + 2 * t;
-#pragma unroll
-      for (int j = 0; j < 16; j++) *reinterpret_cast<float2 *>(dst + 8 * j) = make_float2(o[j][2 * half] * inv, o[j][2 * half + 1] * inv);
-    }
+      for (int j = 0; j < NV; j++) {
+        const int d = 8 * j + 2 * t;
+        if (d >= V) break;
+        if (whole) two(dst + d, o[j][2 * half] * inv, o[j][2 * half + 1] * inv);
+        else {
+          one(dst + d, o[j][2 * half] * inv);
+          if (d + 1 < V) one(dst + d + 1, o[j][2 * half + 1] * inv);
+        }
+      }
+    };
+    if (p.out_bf16)
+      put(p.out_bf16 + z * p.out_stride + (size_t)h * V, [](__nv_bfloat16 *d, float x, float y) { *reinterpret_cast<__nv_bfloat162 *>(d) = __floats2bfloat162_rn(x, y); },
+          [](__nv_bfloat16 *d, float x) { *d = __float2bfloat16_rn(x); });
+    else
+      put(p.out + (z * p.num_heads + h) * V, [](float *d, float x, float y) { *reinterpret_cast<float2 *>(d) = make_float2(x, y); }, [](float *d, float x) { *d = x; });
   }
 }
 
-// Shapes this kernel takes: seq_len > 1, causal, head_dim 128, groups of 1 / 2 / 4 / 8 query heads per KV head,
-// no sliding window / softcap / kv_start, 16-byte aligned K and V rows.
+// Shapes this kernel takes: seq_len > 1, causal, groups of 1 / 2 / 4 / 8 query heads per KV head, no sliding window /
+// softcap / kv_start, 16-byte aligned K and V rows; head_dim 128, or keys in two parts of up to 192 values padded and
+// values of up to 128 (the heads' rows are then whole 16-byte pieces apart).
 bool dpk_attention_prefill_eligible(const dpk_attn_params &p) {
-  if (p.seq_len < 2 || !p.causal || p.head_dim != APF_D || p.fuse.qkv) return false;
+  if (p.seq_len < 2 || !p.causal || p.fuse.qkv || p.kv_f32) return false;
+  if (p.k2) {
+    if ((p.k_dim + 7) / 8 * 8 + (p.k2_dim + 7) / 8 * 8 > 192 || p.v_dim > 128 || p.v_dim <= 0) return false;
+    if (p.k_row_stride % 8 || p.v_row_stride % 8 || p.k2_row_stride % 8 || p.k2_batch_stride % 8 || p.v_batch_stride % 8 || ((uintptr_t)p.k2 & 15)) return false;
+  } else if (p.head_dim != 128 || p.v_row_stride || (p.v_dim && p.v_dim != p.head_dim)) {
+    return false;
+  }
   if (p.num_kv_heads <= 0 || p.num_heads % p.num_kv_heads) return false;
   const int G = p.num_heads / p.num_kv_heads;
   if (G != 1 && G != 2 && G != 4 && G != 8) return false;
@@ -239,16 +283,24 @@ bool dpk_attention_prefill_eligible(const dpk_attn_params &p) {
   return true;
 }
 
-dp_status dpk_attention_prefill(dp_ctx *ctx, const dpk_attn_params &p) {
-  const int G = p.num_heads / p.num_kv_heads;
+template <int DK, int DV>
+static dp_status launch_prefill(dp_ctx *ctx, const dpk_attn_params &p, int G) {
   const int QT = 16 * APF_WARPS / G;
-  const size_t smem = 2 * APF_STAGE;
+  const size_t smem = 2 * ApfLayout<DK, DV>::STAGE;
   static dp_per_device_once attr;
   if (attr.pending(ctx->device)) {
-    DP_CUDA(ctx, cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    DP_CUDA(ctx, cudaFuncSetAttribute((attn_prefill_tc_kernel<DK, DV>), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     attr.done(ctx->device);
   }
   dim3 grid((p.seq_len + QT - 1) / QT, p.num_kv_heads, p.batch);
-  DP_LAUNCH(ctx, attn_prefill_tc_kernel, grid, APF_THREADS, smem, p, G);
+  DP_LAUNCH(ctx, (attn_prefill_tc_kernel<DK, DV>), grid, APF_THREADS, smem, p, G);
   return DP_OK;
+}
+
+dp_status dpk_attention_prefill(dp_ctx *ctx, const dpk_attn_params &p) {
+  const int G = p.num_heads / p.num_kv_heads;
+  const int dk = p.k2 ? (p.k_dim + 7) / 8 * 8 + (p.k2_dim + 7) / 8 * 8 : p.head_dim, dv = p.v_dim ? p.v_dim : p.head_dim;
+  if (dk <= 64 && dv <= 64) return launch_prefill<64, 64>(ctx, p, G);
+  if (dk <= 128) return launch_prefill<128, 128>(ctx, p, G);
+  return launch_prefill<192, 128>(ctx, p, G);
 }

@@ -239,6 +239,11 @@ struct dpk_attn_params {
   bool kv_f32 = false;       // k and v point at f32 caches
   size_t v_batch_stride = 0; // elements between the sequences of v (0: kv_batch_stride)
   int v_row_stride = 0;      // elements between the values of two keys (0: num_kv_heads * v_dim): values that are part of the key rows
+  // keys in two parts (prefill kernel): k holds k_dim values per head, heads padded to 8 values; k2 holds k2_dim values that
+  // all heads share.  head_dim = k_dim + k2_dim is the query's size.
+  const __half *k2 = nullptr;
+  int k_dim = 0, k2_dim = 0, k_row_stride = 0, k2_row_stride = 0;
+  size_t k2_batch_stride = 0;
   // output gate: row r's head h times sigmoid(gate[r * gate_stride + h]); null: none (kernels that write `out` only)
   const float *gate = nullptr;
   int gate_stride = 0;

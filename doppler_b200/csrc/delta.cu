@@ -3,13 +3,21 @@
 // q, k (of kv_heads heads) and v through a causal depthwise convolution and silu, q and k then unit vectors per head (q also
 // divided by sqrt(dim)), beta = sigmoid(b), g = exp(-exp(A_log) softplus(W_a2 a1 + dt_bias)).
 //
-// State layout as in ssm.cu: [head][vdim][state_stride], the key channel fastest and padded with zeros to 32 * 2^k; eight
-// lanes cover a column with 16-byte pieces (lane s holds channels 4 s + 32 i + {0..3}) and reduce over the channels with
-// three shuffles.  A sequence at position 0 starts from zeros whatever its slot held before.
+// State layout as in ssm.cu: [head][vdim][state_stride], the key channel fastest and padded with zeros to 32 * 2^k.  A
+// sequence at position 0 starts from zeros whatever its slot held before.  State arithmetic is packed two channels at a
+// time (fma.rn.f32x2).
 //
-// With S already decayed the read-out needs no second pass over the new state: o = S^T q + (k . q) u, so both sums over the
-// channels run on the same values and only the one with k is on the path from token to token.  State arithmetic is
-// packed two channels at a time (fma.rn.f32x2).
+// A decode step has eight lanes cover a column (lane s holds channels 4 s + 32 i + {0..3}).  With S already decayed the
+// read-out needs no second pass over the new state: o = S^T q + (k . q) u.
+//
+// A portion takes four tokens at a time.  With S the state before them and P(s, t) the product of the decays of tokens
+// s + 1 .. t per channel (products only, nothing is ever divided by a decay):
+//   u_t = beta_t (v_t - S^T (P(-1, t) k_t) - sum_{s < t} (k_t . P(s, t) k_s) u_s)
+//   o_t = S^T (P(-1, t) q_t) + sum_{s <= t} (q_t . P(s, t) k_s) u_s
+//   S'  = P(-1, 3) S + sum_s (P(s, 3) k_s) u_s^T
+// so the sums over the channels of four tokens are reduced across lanes together and the chain from token to token is a
+// handful of scalars.  What does not depend on the state (the vectors in brackets and the scalars) is prepared for all
+// heads and blocks at once.
 #include "layers.h"
 #include "pdl.cuh"
 
@@ -248,9 +256,25 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(const float *__r
   }
 }
 
-// ---- several tokens of one sequence: everything but the recurrence.  A warp owns 16 rows of a q/k head pair or of a run of
-// 32 NJ value channels; the last warps copy the low-rank rows and the write strengths ----
+// ---- several tokens of one sequence: convolutions, unit norms, write strengths ----
 constexpr int DR_ROWS = 16;
+
+// write strengths and low-rank rows [r0, r1)
+__device__ __forceinline__ void dl_aux_rows(const float *proj, int proj_stride, const DeltaShape &sh, const DeltaRows &out, int lane, int r0, int r1) {
+  for (int r = r0; r < r1; r++) {
+    const float *pr = proj + (size_t)r * proj_stride;
+    for (int i = lane; i < sh.heads; i += 32) out.beta[(size_t)r * sh.heads + i] = dl_sigmoid(pr[sh.beta_col() + i]);
+    if (out.a_low)
+#pragma unroll 4
+      for (int i = lane; i < out.a_low_stride; i += 32) out.a_low[(size_t)r * out.a_low_stride + i] = __float2bfloat16_rn(i < sh.decay_rank ? pr[sh.a1_col() + i] : 0.0f);
+    if (out.g_low)
+#pragma unroll 4
+      for (int i = lane; i < out.g_low_stride; i += 32) out.g_low[(size_t)r * out.g_low_stride + i] = __float2bfloat16_rn(i < sh.gate_rank ? pr[sh.g1_col() + i] : 0.0f);
+  }
+}
+constexpr int DR_AUX = 4;  // warps that share these rows of a block
+
+// Any sizes.  A warp owns 16 rows of a q/k head pair or of a run of 32 NJ value channels.
 template <int NJ>
 __global__ void __launch_bounds__(128) delta_rows_kernel(const float *__restrict__ proj, int proj_stride, const DeltaShape sh, const DeltaWeights w, const SsmState st,
                                                          const DeltaRows out, int v_units, int rows, int start_pos, int seq) {
@@ -266,7 +290,7 @@ __global__ void __launch_bounds__(128) delta_rows_kernel(const float *__restrict
   if (unit < G) {
     const float q_mul = 1.0f / sqrtf((float)D);
     for (int r = r0; r < r1; r++) {
-      float q[NJ], k[NJ], qq = 0.0f, kk = 0.0f, qk = 0.0f;
+      float q[NJ], k[NJ], qq = 0.0f, kk = 0.0f;
 #pragma unroll
       for (int j = 0; j < NJ; j++) {
         const int d = lane + 32 * j, cq = unit * D + d, ck = QK + cq;
@@ -279,10 +303,8 @@ __global__ void __launch_bounds__(128) delta_rows_kernel(const float *__restrict
         }
         qq = fmaf(q[j], q[j], qq);
         kk = fmaf(k[j], k[j], kk);
-        qk = fmaf(q[j], k[j], qk);
       }
-      qq = dl_warp_sum(qq); kk = dl_warp_sum(kk); qk = dl_warp_sum(qk);
-      const float qs = 1.0f / sqrtf(qq + 1e-6f) * q_mul, ks = 1.0f / sqrtf(kk + 1e-6f);
+      const float qs = 1.0f / sqrtf(dl_warp_sum(qq) + 1e-6f) * q_mul, ks = 1.0f / sqrtf(dl_warp_sum(kk) + 1e-6f);
 #pragma unroll
       for (int j = 0; j < NJ; j++) {
         const int d = lane + 32 * j;
@@ -291,7 +313,6 @@ __global__ void __launch_bounds__(128) delta_rows_kernel(const float *__restrict
           out.k[(size_t)r * QK + unit * D + d] = k[j] * ks;
         }
       }
-      if (lane == 0) out.qk[(size_t)r * G + unit] = qk * qs * ks;
     }
   } else if (unit < G + v_units) {
     for (int r = r0; r < r1; r++)
@@ -303,92 +324,362 @@ __global__ void __launch_bounds__(128) delta_rows_kernel(const float *__restrict
           keep(r, 2 * QK + e);
         }
       }
-  } else if (unit == G + v_units) {
-    for (int r = r0; r < r1; r++) {
-      const float *pr = proj + (size_t)r * proj_stride;
-      for (int i = lane; i < sh.heads; i += 32) out.beta[(size_t)r * sh.heads + i] = dl_sigmoid(pr[sh.beta_col() + i]);
-      if (out.a_low)
-        for (int i = lane; i < out.a_low_stride; i += 32) out.a_low[(size_t)r * out.a_low_stride + i] = __float2bfloat16_rn(i < sh.decay_rank ? pr[sh.a1_col() + i] : 0.0f);
-      if (out.g_low)
-        for (int i = lane; i < out.g_low_stride; i += 32) out.g_low[(size_t)r * out.g_low_stride + i] = __float2bfloat16_rn(i < sh.gate_rank ? pr[sh.g1_col() + i] : 0.0f);
-    }
+  } else if (unit < G + v_units + DR_AUX) {
+    const int step = DR_ROWS / DR_AUX, a0 = r0 + (unit - G - v_units) * step;
+    dl_aux_rows(proj, proj_stride, sh, out, lane, a0, min(a0 + step, r1));
   }
 }
 
-// ---- the recurrence, token by token: grid (heads, column tiles) ----
-constexpr int DS_TB = 16;  // tokens staged at a time
-template <int NV>
-__global__ void __launch_bounds__(DL_THREADS) delta_scan_kernel(const DeltaShape sh, const SsmState st, const DeltaRows in, float *__restrict__ out, int rows,
+// Up to four taps, sizes and strides that are multiples of four: a lane owns four neighbouring channels (times JV), the
+// rows a token reaches back to stay in registers, and four rows are fetched at a time.
+template <int TAPS>
+struct ConvWindow {
+  float w[4][TAPS];
+  float4 win[TAPS];  // the last TAPS rows, newest at the end
+  __device__ __forceinline__ void init(const float *conv, const float *proj, int proj_stride, const float *hist, int CH, int ch, int r0, int start_pos) {
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+#pragma unroll
+      for (int k = 0; k < TAPS; k++) w[i][k] = conv[(size_t)(ch + i) * TAPS + k];
+#pragma unroll
+    for (int k = 0; k + 1 < TAPS; k++) {
+      const int r = r0 - (TAPS - 1) + k, p = start_pos + r;
+      if (r >= 0) win[k + 1] = *reinterpret_cast<const float4 *>(proj + (size_t)r * proj_stride + ch);
+      else if (p >= 0) win[k + 1] = *reinterpret_cast<const float4 *>(hist + (size_t)(p % TAPS) * CH + ch);
+      else win[k + 1] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+  }
+  __device__ __forceinline__ float4 step(const float4 &x) {  // the row's convolution after silu
+#pragma unroll
+    for (int k = 0; k + 1 < TAPS; k++) win[k] = win[k + 1];
+    win[TAPS - 1] = x;
+    float4 o = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+    for (int k = 0; k < TAPS; k++) {
+      o.x = fmaf(w[0][k], win[k].x, o.x); o.y = fmaf(w[1][k], win[k].y, o.y);
+      o.z = fmaf(w[2][k], win[k].z, o.z); o.w = fmaf(w[3][k], win[k].w, o.w);
+    }
+    return make_float4(dl_silu(o.x), dl_silu(o.y), dl_silu(o.z), dl_silu(o.w));
+  }
+};
+
+template <int JV, int TAPS>
+__global__ void __launch_bounds__(128) delta_rows4_kernel(const float *__restrict__ proj, int proj_stride, const DeltaShape sh, const DeltaWeights w, const SsmState st,
+                                                          const DeltaRows out, int v_units, int rows, int start_pos, int seq) {
+  pdl_launch();
+  pdl_wait();
+  const int lane = threadIdx.x & 31, unit = blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int r0 = blockIdx.y * DR_ROWS, r1 = min(r0 + DR_ROWS, rows);
+  const int G = sh.kv_heads, D = sh.dim, QK = sh.qk(), CH = sh.channels(), inner = sh.inner();
+  const float *hist = st.hist + (size_t)seq * st.hist_seq;
+  constexpr int BATCH = 4;
+  auto keep = [&](int r, int ch, const float4 &x) {
+    if (TAPS > 1 && r >= rows - (TAPS - 1)) *reinterpret_cast<float4 *>(st.stage + (size_t)((start_pos + r) % TAPS) * CH + ch) = x;
+  };
+  if (unit < G) {
+    const float q_mul = 1.0f / sqrtf((float)D);
+    ConvWindow<TAPS> cq[JV], ck[JV];
+#pragma unroll
+    for (int j = 0; j < JV; j++) {
+      const int d = 4 * lane + 128 * j;
+      if (d < D) {
+        cq[j].init(w.conv, proj, proj_stride, hist, CH, unit * D + d, r0, start_pos);
+        ck[j].init(w.conv, proj, proj_stride, hist, CH, QK + unit * D + d, r0, start_pos);
+      }
+    }
+    for (int rb = r0; rb < r1; rb += BATCH) {
+      float4 xq[BATCH][JV], xk[BATCH][JV];
+#pragma unroll
+      for (int b = 0; b < BATCH; b++)
+#pragma unroll
+        for (int j = 0; j < JV; j++) {
+          const int d = 4 * lane + 128 * j;
+          if (d < D && rb + b < r1) {
+            xq[b][j] = *reinterpret_cast<const float4 *>(proj + (size_t)(rb + b) * proj_stride + unit * D + d);
+            xk[b][j] = *reinterpret_cast<const float4 *>(proj + (size_t)(rb + b) * proj_stride + QK + unit * D + d);
+          }
+        }
+#pragma unroll
+      for (int b = 0; b < BATCH; b++) {
+        const int r = rb + b;
+        if (r >= r1) break;  // warp-uniform
+        float qq = 0.0f, kk = 0.0f;
+        float4 q[JV], k[JV];
+#pragma unroll
+        for (int j = 0; j < JV; j++) {
+          const int d = 4 * lane + 128 * j;
+          q[j] = k[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+          if (d < D) {
+            q[j] = cq[j].step(xq[b][j]);
+            k[j] = ck[j].step(xk[b][j]);
+            keep(r, unit * D + d, xq[b][j]);
+            keep(r, QK + unit * D + d, xk[b][j]);
+          }
+          qq = fmaf(q[j].x, q[j].x, fmaf(q[j].y, q[j].y, fmaf(q[j].z, q[j].z, fmaf(q[j].w, q[j].w, qq))));
+          kk = fmaf(k[j].x, k[j].x, fmaf(k[j].y, k[j].y, fmaf(k[j].z, k[j].z, fmaf(k[j].w, k[j].w, kk))));
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+          qq += __shfl_xor_sync(0xffffffffu, qq, o);
+          kk += __shfl_xor_sync(0xffffffffu, kk, o);
+        }
+        const float qs = 1.0f / sqrtf(qq + 1e-6f) * q_mul, ks = 1.0f / sqrtf(kk + 1e-6f);
+#pragma unroll
+        for (int j = 0; j < JV; j++) {
+          const int d = 4 * lane + 128 * j;
+          if (d < D) {
+            *reinterpret_cast<float4 *>(out.q + (size_t)r * QK + unit * D + d) = make_float4(q[j].x * qs, q[j].y * qs, q[j].z * qs, q[j].w * qs);
+            *reinterpret_cast<float4 *>(out.k + (size_t)r * QK + unit * D + d) = make_float4(k[j].x * ks, k[j].y * ks, k[j].z * ks, k[j].w * ks);
+          }
+        }
+      }
+    }
+  } else if (unit < G + v_units) {
+    const int e = (unit - G) * 128 + 4 * lane;
+    if (e >= inner) return;
+    ConvWindow<TAPS> cv;
+    cv.init(w.conv, proj, proj_stride, hist, CH, 2 * QK + e, r0, start_pos);
+    for (int rb = r0; rb < r1; rb += BATCH) {
+      float4 x[BATCH];
+#pragma unroll
+      for (int b = 0; b < BATCH; b++)
+        if (rb + b < r1) x[b] = *reinterpret_cast<const float4 *>(proj + (size_t)(rb + b) * proj_stride + 2 * QK + e);
+#pragma unroll
+      for (int b = 0; b < BATCH; b++)
+        if (rb + b < r1) {
+          *reinterpret_cast<float4 *>(out.v + (size_t)(rb + b) * inner + e) = cv.step(x[b]);
+          keep(rb + b, 2 * QK + e, x[b]);
+        }
+    }
+  } else if (unit < G + v_units + DR_AUX) {
+    const int step = DR_ROWS / DR_AUX, a0 = r0 + (unit - G - v_units) * step;
+    dl_aux_rows(proj, proj_stride, sh, out, lane, a0, min(a0 + step, r1));
+  }
+}
+
+// ---- what a block of four tokens brings, without the state: one warp per (block, head) ----
+// A record: k and q decayed since the block's start, k decayed until its end (4 x NP each), the block's decay (NP), then
+// scalars: [k_1.k_0, k_2.k_0, k_2.k_1, k_3.k_0 | k_3.k_1, k_3.k_2, 0, 0 | beta_0..3 | q_t.k_s as rows t of four], decayed.
+constexpr int DB_T = 4, DB_SCALARS = 32;
+__host__ __device__ constexpr int db_record(int np) { return (3 * DB_T + 1) * np + DB_SCALARS; }
+
+template <int NP>
+__global__ void __launch_bounds__(128) delta_block_kernel(const DeltaShape sh, const DeltaRows in, int rows) {
+  pdl_launch();
+  pdl_wait();
+  constexpr int JB = NP >= 128 ? NP / 128 : 1;
+  const int lane = threadIdx.x & 31, unit = blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int H = sh.heads, D = sh.dim, QK = sh.qk(), HD = H * D, blocks = (rows + DB_T - 1) / DB_T;
+  if (unit >= blocks * H) return;
+  const int blk = unit / H, h = unit - blk * H, kvh = h / (H / sh.kv_heads), r0 = blk * DB_T;
+  const bool vec = (D & 3) == 0;
+  float4 k[DB_T][JB], q[DB_T][JB], g[DB_T][JB];
+  auto load = [&](const float *p, int d, bool ok, float fill) {
+    float4 v = make_float4(fill, fill, fill, fill);
+    if (!ok || d >= D) return v;
+    if (vec) return *reinterpret_cast<const float4 *>(p + d);
+    v.x = p[d];
+    if (d + 1 < D) v.y = p[d + 1];
+    if (d + 2 < D) v.z = p[d + 2];
+    if (d + 3 < D) v.w = p[d + 3];
+    return v;
+  };
+#pragma unroll
+  for (int t = 0; t < DB_T; t++)
+#pragma unroll
+    for (int j = 0; j < JB; j++) {
+      const int d = 4 * lane + 128 * j;
+      const bool ok = r0 + t < rows;
+      const size_t r = (size_t)(r0 + t);
+      k[t][j] = load(in.k + r * QK + kvh * D, d, ok, 0.0f);
+      q[t][j] = load(in.q + r * QK + kvh * D, d, ok, 0.0f);
+      g[t][j] = load(in.g + r * HD + h * D, d, ok, 1.0f);
+    }
+  const float beta = lane < DB_T && r0 + lane < rows ? in.beta[(size_t)(r0 + lane) * H + h] : 0.0f;
+  float *rec = in.records + (size_t)unit * db_record(NP);
+  auto mul = [](float4 &a, const float4 &b) { a.x *= b.x; a.y *= b.y; a.z *= b.z; a.w *= b.w; };
+  auto dot = [](const float4 &a, const float4 &b, float c) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, c)))); };
+  auto put = [&](int slot, int j, const float4 &v) {
+    const int d = 4 * lane + 128 * j;
+    if (d < NP) *reinterpret_cast<float4 *>(rec + slot * NP + d) = v;
+  };
+  // decayed since the start
+  float4 c[JB];
+#pragma unroll
+  for (int t = 0; t < DB_T; t++)
+#pragma unroll
+    for (int j = 0; j < JB; j++) {
+      if (t == 0) c[j] = g[0][j];
+      else mul(c[j], g[t][j]);
+      float4 a = k[t][j], b = q[t][j];
+      mul(a, c[j]);
+      mul(b, c[j]);
+      put(t, j, a);
+      put(DB_T + t, j, b);
+      if (t == DB_T - 1) put(3 * DB_T, j, c[j]);
+    }
+  // decayed from each token on, and the scalars between tokens
+  float sum[16];  // 0..5: k.k pairs in record order, 6 + 3 s - s (s - 1) / 2 ... : q_t . k_s for t >= s, s by s
+  int n = 6;
+#pragma unroll
+  for (int s = 0; s < DB_T; s++) {
+    float d0 = 0.0f;
+#pragma unroll
+    for (int j = 0; j < JB; j++) d0 = dot(k[s][j], q[s][j], d0);
+    sum[n++] = d0;
+#pragma unroll
+    for (int t = s + 1; t < DB_T; t++) {
+      float kk = 0.0f, kq = 0.0f;
+#pragma unroll
+      for (int j = 0; j < JB; j++) {
+        mul(k[s][j], g[t][j]);
+        kk = dot(k[s][j], k[t][j], kk);
+        kq = dot(k[s][j], q[t][j], kq);
+      }
+      sum[t == 1 ? 0 : t == 2 ? 1 + s : 3 + s] = kk;
+      sum[n++] = kq;
+    }
+#pragma unroll
+    for (int j = 0; j < JB; j++) put(2 * DB_T + s, j, k[s][j]);
+  }
+#pragma unroll
+  for (int i = 0; i < 16; i++) sum[i] = dl_warp_sum(sum[i]);
+  float out = 0.0f;  // lane i writes scalar i
+#pragma unroll
+  for (int i = 0; i < 6; i++)
+    if (lane == i) out = sum[i];
+  n = 6;
+#pragma unroll
+  for (int s = 0; s < DB_T; s++)
+#pragma unroll
+    for (int t = s; t < DB_T; t++) {
+      if (lane == 12 + 4 * t + s) out = sum[n];
+      n++;
+    }
+  const float b = __shfl_sync(0xffffffffu, beta, lane & 3);
+  if (lane >= 8 && lane < 12) out = b;
+  rec[(3 * DB_T + 1) * NP + lane] = out;
+}
+
+// ---- the recurrence: grid (heads, column tiles), a warp per eight columns ----
+// LN lanes share LN / 4 columns, a lane holds NP / LN channels of each (4 l + 4 LN i + {0..3}).  The sums of a block (columns x
+// tokens x {k, q}) are reduced and scattered at once: lane l of the warp ends up with both sums of column l / 4 and token l % 4.
+constexpr int DS_COLS = 32, DS_THREADS = 128, DS_STAGES = 4;
+template <int NP, int LN>
+__global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaShape sh, const SsmState st, const DeltaRows in, float *__restrict__ out, int rows,
                                                                 int start_pos, int seq) {
   pdl_launch();
   pdl_wait();
-  constexpr int NP = NV * 32, TOK = 3 * NP + DL_COLS + 4;  // floats staged per token: k, q, g, v, beta, q . k
-  extern __shared__ __align__(16) float ds_smem[];          // [2][DS_TB][TOK], then o [DS_TB][DL_COLS]
-  float *so = ds_smem + 2 * DS_TB * TOK;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, p0 = blockIdx.y * DL_COLS;
-  const int D = sh.dim, V = sh.vdim, G = sh.kv_heads, kvh = h / (sh.heads / G), QK = sh.qk(), inner = sh.inner(), HD = sh.heads * D;
-  const int cols = min(DL_COLS, V - p0), col = tid / DL_LANES, sub = tid % DL_LANES;
-  for (int i = tid; i < 2 * DS_TB * TOK; i += DL_THREADS) ds_smem[i] = 0.0f;  // padded channels and columns stay zero
-  __syncthreads();
-  const bool vec = (D & 3) == 0 && (V & 3) == 0;
-  auto cp = [](float *dst, const float *src, bool wide) {
-    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
-    if (wide) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
-    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
-  };
+  constexpr int R4 = NP / LN / 4, C = LN / 4, REC = db_record(NP);
+  extern __shared__ __align__(16) float ds_smem[];  // [DS_STAGES][REC]
+  __shared__ __align__(16) float su[DS_THREADS / 32][8][DB_T];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, li = lane & (LN - 1), grp = lane / LN;
+  const int V = sh.vdim, inner = sh.inner(), H = sh.heads;
+  const int c0 = blockIdx.y * DS_COLS + warp * 8;       // the warp's first column
+  const int my_col = c0 + (lane >> 2), my_t = lane & 3;  // what this lane finishes
+  const int blocks = (rows + DB_T - 1) / DB_T;
   auto stage = [&](int blk) {
-    const int r0 = blk * DS_TB, n = min(DS_TB, rows - r0);
-    const int unit = vec ? 4 : 1;
-    for (int t = warp; t < n; t += DL_THREADS / 32) {
-      float *d = ds_smem + ((blk & 1) * DS_TB + t) * TOK;
-      const size_t r = (size_t)(r0 + t);
-      const float *k = in.k + r * QK + kvh * D, *q = in.q + r * QK + kvh * D, *g = in.g + r * HD + h * D, *v = in.v + r * inner + h * V + p0;
-      for (int e = lane * unit; e < D; e += 32 * unit) {
-        cp(d + e, k + e, vec);
-        cp(d + NP + e, q + e, vec);
-        cp(d + 2 * NP + e, g + e, vec);
-      }
-      for (int e = lane * unit; e < cols; e += 32 * unit) cp(d + 3 * NP + e, v + e, vec);
-      if (lane == 0) cp(d + 3 * NP + DL_COLS, in.beta + r * sh.heads + h, false);
-      if (lane == 1) cp(d + 3 * NP + DL_COLS + 1, in.qk + r * G + kvh, false);
+    if (blk < blocks) {
+      const float *src = in.records + ((size_t)blk * H + h) * REC;
+      const uint32_t dst = (uint32_t)__cvta_generic_to_shared(ds_smem + (blk % DS_STAGES) * REC);
+      for (int i = tid; i < REC / 4; i += DS_THREADS)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + 16 * i), "l"(src + 4 * i) : "memory");
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  float *S = st.s + (size_t)seq * st.s_seq + ((size_t)h * V + p0 + col) * NP + 4 * sub;
-  f32x2 s[2 * NV];
+  f32x2 s[C][2 * R4];
+  float *S = st.s + (size_t)seq * st.s_seq + ((size_t)h * V + c0 + grp * C) * NP + 4 * li;
 #pragma unroll
-  for (int i = 0; i < NV; i++) {
-    if (col < cols && start_pos > 0) x2_load4(S + 32 * i, s[2 * i], s[2 * i + 1]);
-    else s[2 * i] = s[2 * i + 1] = 0ull;
-  }
-  const int blocks = (rows + DS_TB - 1) / DS_TB;
-  stage(0);
+  for (int c = 0; c < C; c++)
+#pragma unroll
+    for (int i = 0; i < R4; i++) {
+      if (c0 + grp * C + c < V && start_pos > 0) x2_load4(S + (size_t)c * NP + 4 * LN * i, s[c][2 * i], s[c][2 * i + 1]);
+      else s[c][2 * i] = s[c][2 * i + 1] = 0ull;
+    }
+  const size_t my_off = (size_t)h * V + my_col;
+  auto value = [&](int blk) { return my_col < V && blk * DB_T + my_t < rows ? in.v[(size_t)(blk * DB_T + my_t) * inner + my_off] : 0.0f; };
+#pragma unroll
+  for (int i = 0; i < DS_STAGES - 1; i++) stage(i);
+  float v_next = value(0);
   for (int blk = 0; blk < blocks; blk++) {
-    if (blk + 1 < blocks) {
-      stage(blk + 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    __syncthreads();
-    const float *src = ds_smem + (blk & 1) * DS_TB * TOK;
-    const int r0 = blk * DS_TB, n = min(DS_TB, rows - r0);
-#pragma unroll 2
-    for (int t = 0; t < n; t++) {
-      const float *d = src + t * TOK;
-      const float2 bq = *reinterpret_cast<const float2 *>(d + 3 * NP + DL_COLS);
-      const float o = dl_token<NV>(s, d, d + NP, d + 2 * NP, sub, d[3 * NP + col], bq.x, bq.y, 1.0f, 1.0f);
-      if (sub == 0) so[t * DL_COLS + col] = o;
-    }
-    __syncthreads();
-    for (int i = tid; i < n * DL_COLS; i += DL_THREADS) {
-      const int t = i / DL_COLS, c = i - t * DL_COLS;
-      if (c < cols) out[(size_t)(r0 + t) * inner + h * V + p0 + c] = so[i];
-    }
-  }
-  if (col < cols)
+    asm volatile("cp.async.wait_group %0;" ::"n"(DS_STAGES - 2) : "memory");
+    __syncthreads();  // this record is there, and every warp is done with the one before it
+    stage(blk + DS_STAGES - 1);
+    const float *rec = ds_smem + (blk % DS_STAGES) * REC, *vec = rec + 4 * li, *sc = rec + (3 * DB_T + 1) * NP;
+    const float v = v_next;
+    v_next = value(blk + 1);
+    float val[C * 2 * DB_T];
 #pragma unroll
-    for (int i = 0; i < NV; i++) x2_store4(S + 32 * i, s[2 * i], s[2 * i + 1]);
+    for (int t = 0; t < DB_T; t++)
+#pragma unroll
+      for (int kq = 0; kq < 2; kq++) {
+        f32x2 x[2 * R4], acc[C];
+#pragma unroll
+        for (int i = 0; i < R4; i++) x2_load4(vec + (kq * DB_T + t) * NP + 4 * LN * i, x[2 * i], x[2 * i + 1]);
+#pragma unroll
+        for (int c = 0; c < C; c++) {
+          acc[c] = x2_mul(s[c][0], x[0]);
+#pragma unroll
+          for (int i = 1; i < 2 * R4; i++) acc[c] = x2_fma(s[c][i], x[i], acc[c]);
+        }
+#pragma unroll
+        for (int c = 0; c < C; c++) val[(c * DB_T + t) * 2 + kq] = x2_sum(acc[c]);
+      }
+    int n = C * 2 * DB_T;
+#pragma unroll
+    for (int o = LN / 2; o > 0; o >>= 1) {
+      n >>= 1;
+      const bool upper = li & o;
+#pragma unroll
+      for (int i = 0; i < C * DB_T; i++)
+        if (i < n) {
+          const float send = upper ? val[i] : val[i + n], keep = upper ? val[i + n] : val[i];
+          val[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
+    }
+    const float4 a0 = *reinterpret_cast<const float4 *>(sc), a1 = *reinterpret_cast<const float4 *>(sc + 4), be = *reinterpret_cast<const float4 *>(sc + 8);
+    const float4 b = *reinterpret_cast<const float4 *>(sc + 12 + 4 * my_t);
+    const float e = v - val[0];
+    const float e0 = __shfl_sync(0xffffffffu, e, lane & ~3), e1 = __shfl_sync(0xffffffffu, e, lane & ~3 | 1), e2 = __shfl_sync(0xffffffffu, e, lane & ~3 | 2),
+                e3 = __shfl_sync(0xffffffffu, e, lane | 3);
+    const float u0 = be.x * e0, u1 = be.y * fmaf(-a0.x, u0, e1), u2 = be.z * fmaf(-a0.z, u1, fmaf(-a0.y, u0, e2)),
+                u3 = be.w * fmaf(-a1.y, u2, fmaf(-a1.x, u1, fmaf(-a0.w, u0, e3)));
+    su[warp][lane >> 2][my_t] = my_t == 0 ? u0 : my_t == 1 ? u1 : my_t == 2 ? u2 : u3;
+    __syncwarp();
+    if (my_col < V && blk * DB_T + my_t < rows)
+      out[(size_t)(blk * DB_T + my_t) * inner + my_off] = fmaf(b.w, u3, fmaf(b.z, u2, fmaf(b.y, u1, fmaf(b.x, u0, val[1]))));
+    {
+      f32x2 g[2 * R4];
+#pragma unroll
+      for (int i = 0; i < R4; i++) x2_load4(vec + 3 * DB_T * NP + 4 * LN * i, g[2 * i], g[2 * i + 1]);
+#pragma unroll
+      for (int c = 0; c < C; c++)
+#pragma unroll
+        for (int i = 0; i < 2 * R4; i++) s[c][i] = x2_mul(s[c][i], g[i]);
+    }
+    float4 u[C];
+#pragma unroll
+    for (int c = 0; c < C; c++) u[c] = *reinterpret_cast<const float4 *>(su[warp][grp * C + c]);
+#pragma unroll
+    for (int t = 0; t < DB_T; t++) {
+      f32x2 x[2 * R4];
+#pragma unroll
+      for (int i = 0; i < R4; i++) x2_load4(vec + (2 * DB_T + t) * NP + 4 * LN * i, x[2 * i], x[2 * i + 1]);
+#pragma unroll
+      for (int c = 0; c < C; c++) {
+        const float ut = t == 0 ? u[c].x : t == 1 ? u[c].y : t == 2 ? u[c].z : u[c].w;
+        const f32x2 uu = x2_pack(ut, ut);
+#pragma unroll
+        for (int i = 0; i < 2 * R4; i++) s[c][i] = x2_fma(x[i], uu, s[c][i]);
+      }
+    }
+    __syncwarp();  // su is rewritten by the next block
+  }
+#pragma unroll
+  for (int c = 0; c < C; c++)
+#pragma unroll
+    for (int i = 0; i < R4; i++)
+      if (c0 + grp * C + c < V) x2_store4(S + (size_t)c * NP + 4 * LN * i, s[c][2 * i], s[c][2 * i + 1]);
 }
 
 template <int NV>
@@ -409,20 +700,41 @@ dp_status launch_step(dp_ctx *ctx, const float *proj, int proj_stride, const Del
 
 template <int NV>
 dp_status launch_scan(dp_ctx *ctx, const DeltaShape &sh, const SsmState &st, const DeltaRows &r, float *out, int rows, const RowMap &map) {
-  const size_t smem = (size_t)(2 * DS_TB * (3 * NV * 32 + DL_COLS + 4) + DS_TB * DL_COLS) * 4;
+  constexpr int NP = 32 * NV, LN = NP == 32 ? 8 : NP <= 128 ? 16 : 32;
+  const size_t smem = (size_t)DS_STAGES * db_record(NP) * 4;
   static dp_per_device_once attr;
   if (attr.pending(ctx->device)) {
-    DP_CUDA(ctx, cudaFuncSetAttribute(delta_scan_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    DP_CUDA(ctx, cudaFuncSetAttribute((delta_scan_kernel<NP, LN>), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     attr.done(ctx->device);
   }
-  DP_LAUNCH(ctx, delta_scan_kernel<NV>, dim3(sh.heads, (sh.vdim + DL_COLS - 1) / DL_COLS), DL_THREADS, smem, sh, st, r, out, rows, map.start_pos, map.seq);
+  const int units = (rows + DB_T - 1) / DB_T * sh.heads;
+  DP_LAUNCH(ctx, delta_block_kernel<NP>, (units + 3) / 4, 128, 0, sh, r, rows);
+  DP_LAUNCH(ctx, (delta_scan_kernel<NP, LN>), dim3(sh.heads, (sh.vdim + DS_COLS - 1) / DS_COLS), DS_THREADS, smem, sh, st, r, out, rows, map.start_pos, map.seq);
+  return DP_OK;
+}
+
+template <int JV>
+dp_status launch_rows4(dp_ctx *ctx, const float *proj, int proj_stride, const DeltaShape &sh, const DeltaWeights &w, const SsmState &st, const DeltaRows &r, int rows,
+                       const RowMap &map) {
+  const int v_units = (sh.inner() + 127) / 128, units = sh.kv_heads + v_units + DR_AUX;
+  const dim3 grid((units + 3) / 4, (rows + DR_ROWS - 1) / DR_ROWS);
+#define DP_ROWS4(T) DP_LAUNCH(ctx, (delta_rows4_kernel<JV, T>), grid, 128, 0, proj, proj_stride, sh, w, st, r, v_units, rows, map.start_pos, map.seq)
+  switch (sh.taps) {
+    case 1: DP_ROWS4(1); break;
+    case 2: DP_ROWS4(2); break;
+    case 3: DP_ROWS4(3); break;
+    default: DP_ROWS4(4); break;
+  }
+#undef DP_ROWS4
   return DP_OK;
 }
 
 template <int NJ>
 dp_status launch_rows(dp_ctx *ctx, const float *proj, int proj_stride, const DeltaShape &sh, const DeltaWeights &w, const SsmState &st, const DeltaRows &r, int rows,
                       const RowMap &map) {
-  const int v_units = (sh.inner() + 32 * NJ - 1) / (32 * NJ), units = sh.kv_heads + v_units + 1;
+  if (sh.taps <= 4 && sh.dim % 4 == 0 && sh.inner() % 4 == 0 && proj_stride % 4 == 0 && NJ <= 8)
+    return launch_rows4<(NJ > 4 ? 2 : 1)>(ctx, proj, proj_stride, sh, w, st, r, rows, map);
+  const int v_units = (sh.inner() + 32 * NJ - 1) / (32 * NJ), units = sh.kv_heads + v_units + DR_AUX;
   DP_LAUNCH(ctx, delta_rows_kernel<NJ>, dim3((units + 3) / 4, (rows + DR_ROWS - 1) / DR_ROWS), 128, 0, proj, proj_stride, sh, w, st, r, v_units, rows, map.start_pos,
             map.seq);
   return DP_OK;
@@ -451,3 +763,4 @@ dp_status dpk_delta_rows(dp_ctx *ctx, const float *proj, int proj_stride, const 
 dp_status dpk_delta_scan(dp_ctx *ctx, const DeltaShape &sh, const SsmState &st, const DeltaRows &r, float *out, int rows, const RowMap &map) {
   DP_BY_STRIDE(launch_scan, ctx, sh, st, r, out, rows, map);
 }
+size_t dpk_delta_record_floats(const DeltaShape &sh, int rows) { return (size_t)((rows + DB_T - 1) / DB_T) * sh.heads * db_record(sh.state_stride); }

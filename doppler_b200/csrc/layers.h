@@ -179,10 +179,10 @@ struct DeltaWeights {
 // what a portion's tokens bring to the recurrence, f32
 struct DeltaRows {
   float *q, *k;     // [rows][kv_heads * dim] unit vectors, q also / sqrt(dim)
-  float *qk;        // [rows][kv_heads] q . k
   float *v;         // [rows][heads * vdim]
   float *beta;      // [rows][heads]
   const float *g;   // [rows][heads * dim] decays
+  float *records;   // dpk_delta_record_floats: the same, arranged for the recurrence
   __nv_bfloat16 *a_low = nullptr, *g_low = nullptr;  // low-rank rows as bf16, strides multiples of 8 (null: not wanted)
   int a_low_stride = 0, g_low_stride = 0;
 };
@@ -193,6 +193,7 @@ dp_status dpk_delta_step(dp_ctx *ctx, const float *proj, int proj_stride, const 
 // consecutive tokens of one sequence: convolutions, unit norms, write strengths; then the recurrence over them
 dp_status dpk_delta_rows(dp_ctx *ctx, const float *proj, int proj_stride, const DeltaShape &sh, const DeltaWeights &w, const SsmState &st, const DeltaRows &r,
                          int rows, const RowMap &map);
+size_t dpk_delta_record_floats(const DeltaShape &sh, int rows);
 dp_status dpk_delta_scan(dp_ctx *ctx, const DeltaShape &sh, const SsmState &st, const DeltaRows &r, float *out, int rows, const RowMap &map);
 
 // ---- latent attention (latent.cu) ----

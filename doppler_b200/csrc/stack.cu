@@ -45,6 +45,8 @@ struct StackLayer {
   Mat proj, o, gateup, down;
   Mat a2, g2;      // delta rule: second matrices of decay and gate
   Mat uq, uk, uv;  // latent attention
+  Mat ukv;         // latent attention: uk and uv together in f16, heads padded to eight rows (bf16 mode)
+  bool up_exact = true;  // every value fits f16
   __nv_bfloat16 *norm[2] = {}, *conv[2] = {}, *post[2] = {}, *mix_norm = nullptr, *dq_norm = nullptr, *dkv_norm = nullptr;
   float *hc_in[2] = {}, *hc_out[2] = {}, *hc_mix[2] = {};
   float *conv_w = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *d = nullptr;
@@ -84,6 +86,8 @@ struct dp_stack {
   dp_stack_cfg cfg;
   bool f32 = false;
   std::vector<StackLayer> layers;
+  dp_buf expanded = nullptr;   // latent attention: keys and values of a sequence's tokens, [token][ukv.N] f16
+
   Mat embed;
   __nv_bfloat16 *final_norm = nullptr;
   uint64_t missing = 0;
@@ -113,6 +117,25 @@ dp_status mat_alloc(dp_model *m, Mat *t, int N, int K, const char *label) {
 dp_status mat_upload(dp_ctx *ctx, const Mat &t, int row0, const void *host, int rows, int cols) {
   DP_CUDA(ctx, cudaMemcpy2DAsync((char *)t.buf->dptr + (size_t)row0 * t.stride * 2, (size_t)t.stride * 2, host, (size_t)cols * 2, (size_t)cols * 2, (size_t)rows,
                                  cudaMemcpyHostToDevice, ctx->stream));
+  DP_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
+  return DP_OK;
+}
+
+// bf16 rows of all heads into a matrix of f16, a head's rows padded to whole groups of eight; *exact is cleared where a value
+// does not fit
+dp_status mat_upload_f16(dp_ctx *ctx, const Mat &t, int row0, const void *host, int heads, int rows, int cols, bool *exact) {
+  const size_t padded = up((size_t)rows, 8);
+  std::vector<__half> stage(heads * padded * t.stride, __half(0.0f));
+  for (int h = 0; h < heads; h++)
+    for (int r = 0; r < rows; r++)
+      for (int c = 0; c < cols; c++) {
+        const uint32_t bits = (uint32_t)((const uint16_t *)host)[((size_t)h * rows + r) * cols + c] << 16;
+        float v;
+        memcpy(&v, &bits, 4);
+        if (!(fabsf(v) <= 65504.0f)) *exact = false;
+        stage[(h * padded + r) * t.stride + c] = __float2half_rn(v);
+      }
+  DP_CUDA(ctx, cudaMemcpyAsync((char *)t.buf->dptr + (size_t)row0 * t.stride * 2, stage.data(), stage.size() * 2, cudaMemcpyHostToDevice, ctx->stream));
   DP_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
   return DP_OK;
 }
@@ -199,7 +222,7 @@ void carve_acts(dp_model *m, Carver &c) {
   dp_stack *s = m->stack;
   const size_t T = m->T, H = s->cfg.width, S = s->cfg.streams;
   size_t proj = 0, q = 1, xbc = 1, heads = 1, mix = 1, k = up(H, 8), ff = 1;
-  size_t dl_qk = 0, dl_heads = 0, dl_inner = 0, dl_hd = 0, low_a = 0, low_g = 0, q_abs = 0, ctx = 0;
+  size_t dl_qk = 0, dl_heads = 0, dl_inner = 0, dl_hd = 0, low_a = 0, low_g = 0, records = 0, q_abs = 0, ctx = 0;
   auto most = [](size_t &a, size_t b) { if (b > a) a = b; };
   for (const StackLayer &L : s->layers) {
     most(proj, L.proj.N);
@@ -210,7 +233,7 @@ void carve_acts(dp_model *m, Carver &c) {
     if (L.mamba() || L.lightning()) { most(xbc, L.channels()); most(heads, L.c.heads); }
     if (L.is_delta()) {
       most(dl_qk, L.delta.qk()); most(dl_heads, L.c.heads); most(dl_inner, L.inner()); most(dl_hd, (size_t)L.c.heads * L.c.dim);
-      most(low_a, L.a2.stride); most(low_g, L.g2.stride);
+      most(low_a, L.a2.stride); most(low_g, L.g2.stride); most(records, dpk_delta_record_floats(L.delta, (int)T));
     }
     if (L.latent()) {
       most(q, L.uq.N); most(k, L.uq.stride);
@@ -219,8 +242,9 @@ void carve_acts(dp_model *m, Carver &c) {
   }
   c.take(&s->x[0], T * S * H); c.take(&s->x[1], T * S * H); c.take(&s->y, T * H); c.take(&m->h, T * H);
   c.take(&s->proj, T * proj); c.take(&s->q, T * q); c.take(&s->xbc, T * xbc); c.take(&s->dt, T * heads); c.take(&s->mix, T * mix);
-  c.take(&s->dl.q, T * dl_qk); c.take(&s->dl.k, T * dl_qk); c.take(&s->dl.qk, T * dl_heads); c.take(&s->dl.beta, T * dl_heads);
+  c.take(&s->dl.q, T * dl_qk); c.take(&s->dl.k, T * dl_qk); c.take(&s->dl.beta, T * dl_heads);
   c.take(&s->dl.v, T * dl_inner); c.take(&s->gate, T * dl_inner); c.take(&s->dl_g, T * dl_hd);
+  c.take(&s->dl.records, records);
   c.take(&s->dl.a_low, T * low_a); c.take(&s->dl.g_low, T * low_g);
   c.take(&s->q_abs, T * q_abs); c.take(&s->ctx, T * ctx);
   const size_t e = s->f32 ? 4 : 2;
@@ -446,6 +470,38 @@ dp_status delta_portion(dp_model *m, StackLayer &L, int rows, const RowMap &map)
   return dpk_delta_scan(m->ctx, L.delta, L.st, r, s->mix, rows, map);
 }
 
+// Keys and values of all heads formed from the cached latents (portions of many rows): what `expanded` must be able to hold,
+// and where it pays: forming them costs as much per token as `rows` queries save against the absorbed form, whose products
+// run at about a quarter of the rate.
+bool expand_pays(const dp_stack *s, const StackLayer &L, int rows, int kv_len) {
+  const LatentShape &sh = L.lat;
+  if (s->f32 || !s->expanded || !L.up_exact || rows < 16 || (size_t)kv_len * L.ukv.N * 2 > s->expanded->bytes) return false;
+  const long saved = 2l * sh.kv_rank + sh.rot_dim - (sh.dim + sh.rot_dim + sh.vdim);
+  return saved > 0 ? saved * 4 * rows >= (long)sh.kv_rank * (sh.dim + sh.vdim) : true;
+}
+
+dp_status latent_expanded(dp_model *m, int l, int rows, int seq, int start_pos, int ks) {
+  dp_stack *s = m->stack;
+  StackLayer &L = s->layers[l];
+  const LatentShape &sh = L.lat;
+  const LatentCache cache = latent_cache(m, l);
+  const int kv_len = start_pos + rows, N = L.ukv.N;
+  const __half *lat = (const __half *)cache.rows + (size_t)seq * cache.seq;
+  __half *kv = (__half *)s->expanded->dptr;
+  DP_TRY(dpk_gemm_f16_tc(m->ctx, (const __half *)L.ukv.w(), L.ukv.stride, lat, sh.cols(), kv, N, kv_len, N, sh.kv_rank));
+  dpk_attn_params p{};
+  p.q = s->q;
+  p.scale = L.c.scale;
+  p.num_heads = p.num_kv_heads = sh.heads; p.head_dim = sh.dim + sh.rot_dim; p.v_dim = sh.vdim;
+  p.k = kv; p.k_dim = sh.dim; p.k_row_stride = N;
+  p.v = kv + (size_t)sh.heads * up(sh.dim, 8); p.v_row_stride = N;
+  p.k2 = lat + sh.c_pad(); p.k2_dim = sh.rot_dim; p.k2_row_stride = sh.cols();
+  p.batch = 1; p.seq_len = rows; p.kv_len = kv_len; p.causal = 1; p.start_pos = start_pos;
+  p.out_bf16 = (__nv_bfloat16 *)s->a; p.out_stride = ks;
+  if (L.c.head_gate) { p.gate = s->proj + sh.gate_col(); p.gate_stride = L.proj.N; }
+  return dpk_attention_with_scratch(m->ctx, p, nullptr, 1);
+}
+
 // Latent attention of several rows: s->proj -> head outputs in s->a (rows of `ks` elements).
 dp_status latent_rows(dp_model *m, int l, int rows, bool decode, int seq, int start_pos, int ks, const RowMap &map) {
   dp_ctx *ctx = m->ctx;
@@ -457,7 +513,9 @@ dp_status latent_rows(dp_model *m, int l, int rows, bool decode, int seq, int st
   const int qs = a_stride(s, L.uq.K);
   DP_TRY(dpk_group_norm(ctx, s->proj, L.proj.N, n, sh.q_rank, s->a, !s->f32, qs, rows));
   DP_TRY(product(m, L.uq, s->a, qs, s->q, rows));
-  DP_TRY(dpk_latent_append(ctx, s->proj, L.proj.N, sh, L.dkv_norm, L.rot, latent_cache(m, l), s->q, s->q_abs, rows, map));
+  const bool expand = !decode && expand_pays(s, L, rows, start_pos + rows);
+  DP_TRY(dpk_latent_append(ctx, s->proj, L.proj.N, sh, L.dkv_norm, L.rot, latent_cache(m, l), s->q, expand ? nullptr : s->q_abs, rows, map));
+  if (expand) return latent_expanded(m, l, rows, seq, start_pos, ks);
   GroupedProduct p;
   p.w = L.uk.w(); p.w_z = (size_t)sh.dim * L.uk.stride; p.w_n = 1; p.w_k = L.uk.stride;
   p.x = s->q; p.x_row = L.uq.N; p.x_z = sh.dim + sh.rot_dim;
@@ -467,7 +525,7 @@ dp_status latent_rows(dp_model *m, int l, int rows, bool decode, int seq, int st
   dpk_attn_params ap = attn_params(m, l, rows, decode, seq, start_pos);
   ap.out = s->ctx;
   int splits = 1;
-  if (decode) dpk_attention_scratch_bytes(ctx, ap, &splits);
+  if (dpk_attention_scratch_bytes(ctx, ap, &splits) > m->attn_scratch->bytes) splits = 1;
   DP_TRY(dpk_attention_with_scratch(ctx, ap, (float *)m->attn_scratch->dptr, splits));
   p = GroupedProduct();
   p.w = L.uv.w(); p.w_z = (size_t)sh.vdim * L.uv.stride; p.w_n = L.uv.stride; p.w_k = 1;
@@ -659,6 +717,7 @@ extern "C" dp_status dp_model_create_stack(dp_ctx *ctx, const dp_stack_cfg *cfg,
     DP_TRY(mat_alloc(m, &s->embed, c.vocab, c.width, "embedding_bf16"));
     s->missing = one << DP_T_EMBED | one << DP_T_FINAL_NORM;
     const size_t e = s->f32 ? 4 : 2;
+    size_t expand_cols = 0;
     auto miss = [](StackLayer &L, std::initializer_list<int> ids) { for (int id : ids) L.missing |= (uint64_t)1 << id; };
     for (int l = 0; l < c.n_layers; l++) {
       StackLayer &L = s->layers[l];
@@ -694,6 +753,11 @@ extern "C" dp_status dp_model_create_stack(dp_ctx *ctx, const dp_stack_cfg *cfg,
         DP_TRY(mat_alloc(m, &L.uq, L.c.heads * (L.c.dim + L.c.rot_dim), L.c.q_rank, "w_uq_bf16"));
         DP_TRY(mat_alloc(m, &L.uk, L.c.heads * L.c.dim, L.c.kv_rank, "w_uk_bf16"));
         DP_TRY(mat_alloc(m, &L.uv, L.c.heads * L.c.vdim, L.c.kv_rank, "w_uv_bf16"));
+        if (!s->f32) {
+          DP_TRY(mat_alloc(m, &L.ukv, (int)(L.c.heads * (up(L.c.dim, 8) + up(L.c.vdim, 8))), L.c.kv_rank, "w_ukv_f16"));
+          m->weight_bytes -= (size_t)L.ukv.N * L.ukv.stride * 2;  // a copy; a decode step reads uk and uv
+          if (up(L.c.dim, 8) + up(L.c.rot_dim, 8) <= 192 && L.c.vdim <= 128 && (size_t)L.ukv.N > expand_cols) expand_cols = L.ukv.N;
+        }
         DP_TRY(rope_table(m, L.c.rot_dim, L.c.rot_base, &L.rot));
       }
       DP_TRY(mat_alloc(m, &L.o, c.width, L.inner(), "w_o_bf16"));
@@ -736,9 +800,14 @@ extern "C" dp_status dp_model_create_stack(dp_ctx *ctx, const dp_stack_cfg *cfg,
         DP_TRY(dp_buf_acquire(ctx, bytes, "latent_cache", &m->kc[l]));
         DP_TRY(dp_buf_fill(ctx, m->kc[l], 0, 0, m->kc[l]->bytes));  // the padding of its rows stays zero
         s->state_bytes += bytes;
-        const size_t need = (size_t)B * L.c.heads * 32 * (L.lat.c_pad() + 2) * 4;
+        // a wave of CTAs beside the rows: short portions split their keys too
+        const size_t need = ((size_t)B * 32 + ctx->sm_count + 64) * L.c.heads * (L.lat.c_pad() + 2) * 4;
         if (need > scratch) scratch = need;
       }
+    }
+    if (expand_cols) {
+      const size_t most = (size_t)4 << 30, bytes = (size_t)c.max_seq * expand_cols * 2;  // longer sequences take the absorbed form
+      DP_TRY(dp_buf_acquire(ctx, bytes < most ? bytes : most, "latent_expanded", &s->expanded));
     }
     DP_TRY(carve(&s->state, "sequence_state", [&](Carver &k) { carve_state(s, k); }));
     s->state_bytes += s->state->bytes;
@@ -796,7 +865,8 @@ void dp_stack_destroy(dp_model *m) {
   auto rel = [&](dp_buf b) { if (b) dp_buf_release(m->ctx, b); };
   for (StackLayer &L : s->layers)
     if (L.owner < 0)
-      for (const Mat *t : {&L.proj, &L.o, &L.gateup, &L.down, &L.a2, &L.g2, &L.uq, &L.uk, &L.uv}) rel(t->buf);
+      for (const Mat *t : {&L.proj, &L.o, &L.gateup, &L.down, &L.a2, &L.g2, &L.uq, &L.uk, &L.uv, &L.ukv}) rel(t->buf);
+  rel(s->expanded);
   for (RopeTable &t : s->ropes) rel(t.buf);
   rel(s->embed.buf); rel(s->vectors); rel(s->state); rel(s->acts); rel(s->entries);
   delete s;
@@ -925,8 +995,18 @@ extern "C" dp_status dp_model_load_tensor(dp_model *m, int layer, dp_tensor_id i
     case DP_T_DQ_NORM: st = vec_bf16(L.dq_norm, 1, L.c.q_rank); break;
     case DP_T_DKV_NORM: st = vec_bf16(L.dkv_norm, 1, L.c.kv_rank); break;
     case DP_T_UQ: st = part(lat, L.uq, 0, L.uq.N, L.c.q_rank); break;
-    case DP_T_UK: st = part(lat, L.uk, 0, L.uk.N, L.c.kv_rank); break;
-    case DP_T_UV: st = part(lat, L.uv, 0, L.uv.N, L.c.kv_rank); break;
+    case DP_T_UK:
+    case DP_T_UV: {
+      const bool is_v = id == DP_T_UV;
+      const Mat &w = is_v ? L.uv : L.uk;
+      st = part(lat, w, 0, w.N, L.c.kv_rank);
+      if (st == DP_OK && L.ukv.buf) {
+        st = mat_upload_f16(ctx, L.ukv, is_v ? (int)(L.c.heads * up(L.c.dim, 8)) : 0, host, L.c.heads, is_v ? L.c.vdim : L.c.dim, L.c.kv_rank, &L.up_exact);
+        for (StackLayer &o : s->layers)
+          if (o.owner == layer) o.up_exact = L.up_exact;
+      }
+      break;
+    }
     case DP_T_FF_GATE:
     case DP_T_FF_UP:
       DP_CHECK(ctx, L.c.ff > 0, "loadTensor: layer %d has no %s", layer, tensor_name(id));
