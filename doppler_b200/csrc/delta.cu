@@ -561,29 +561,34 @@ __global__ void __launch_bounds__(128) delta_block_kernel(const DeltaShape sh, c
   rec[(3 * DB_T + 1) * NP + lane] = out;
 }
 
-// ---- the recurrence: grid (heads, column tiles), a warp per eight columns ----
-// LN lanes share LN / 4 columns, a lane holds NP / LN channels of each (4 l + 4 LN i + {0..3}).  The sums of a block (columns x
-// tokens x {k, q}) are reduced and scattered at once: lane l of the warp ends up with both sums of column l / 4 and token l % 4.
-constexpr int DS_COLS = 32, DS_THREADS = 128, DS_STAGES = 4;
+// ---- the recurrence: grid (heads, column tiles), a warp per four columns ----
+// LN lanes share LN / 8 columns, a lane holds NP / LN channels of each (4 l + 4 LN i + {0..3}).  The sums of a block (columns x
+// tokens x {k, q}) are reduced and scattered at once: lane 8 c + 2 t + {0, 1} of the warp ends up with the sums of column c and
+// token t, the even lane with the one for k, the odd lane with the one for q.
+constexpr int DS_COLS = 32, DS_WARPS = 8, DS_THREADS = DS_WARPS * 32, DS_STAGES = 4;
 template <int NP, int LN>
 __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaShape sh, const SsmState st, const DeltaRows in, float *__restrict__ out, int rows,
                                                                 int start_pos, int seq) {
   pdl_launch();
   pdl_wait();
-  constexpr int R4 = NP / LN / 4, C = LN / 4, REC = db_record(NP);
+  constexpr int R4 = NP / LN / 4, C = LN / 8, REC = db_record(NP);
   extern __shared__ __align__(16) float ds_smem[];  // [DS_STAGES][REC]
-  __shared__ __align__(16) float su[DS_THREADS / 32][8][DB_T];
+  __shared__ __align__(16) float su[DS_WARPS][4][DB_T];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, li = lane & (LN - 1), grp = lane / LN;
   const int V = sh.vdim, inner = sh.inner(), H = sh.heads;
-  const int c0 = blockIdx.y * DS_COLS + warp * 8;       // the warp's first column
-  const int my_col = c0 + (lane >> 2), my_t = lane & 3;  // what this lane finishes
+  const int c0 = blockIdx.y * DS_COLS + warp * 4;                                       // the warp's first column
+  const int my_col = c0 + (lane >> 3), my_t = (lane >> 1) & 3, first = lane & ~7;  // what this lane finishes
+  const bool is_q = lane & 1;
   const int blocks = (rows + DB_T - 1) / DB_T;
   auto stage = [&](int blk) {
     if (blk < blocks) {
       const float *src = in.records + ((size_t)blk * H + h) * REC;
       const uint32_t dst = (uint32_t)__cvta_generic_to_shared(ds_smem + (blk % DS_STAGES) * REC);
-      for (int i = tid; i < REC / 4; i += DS_THREADS)
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + 16 * i), "l"(src + 4 * i) : "memory");
+#pragma unroll
+      for (int k = 0; k < (REC / 4 + DS_THREADS - 1) / DS_THREADS; k++) {
+        const int i = tid + k * DS_THREADS;
+        if (i < REC / 4) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + 16 * i), "l"(src + 4 * i) : "memory");
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -597,7 +602,7 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaShape
       else s[c][2 * i] = s[c][2 * i + 1] = 0ull;
     }
   const size_t my_off = (size_t)h * V + my_col;
-  auto value = [&](int blk) { return my_col < V && blk * DB_T + my_t < rows ? in.v[(size_t)(blk * DB_T + my_t) * inner + my_off] : 0.0f; };
+  auto value = [&](int blk) { return !is_q && my_col < V && blk * DB_T + my_t < rows ? in.v[(size_t)(blk * DB_T + my_t) * inner + my_off] : 0.0f; };
 #pragma unroll
   for (int i = 0; i < DS_STAGES - 1; i++) stage(i);
   float v_next = value(0);
@@ -637,17 +642,18 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaShape
           val[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
         }
     }
-    const float4 a0 = *reinterpret_cast<const float4 *>(sc), a1 = *reinterpret_cast<const float4 *>(sc + 4), be = *reinterpret_cast<const float4 *>(sc + 8);
+    const float4 a0 = *reinterpret_cast<const float4 *>(sc), be = *reinterpret_cast<const float4 *>(sc + 8);
+    const float2 a1 = *reinterpret_cast<const float2 *>(sc + 4);
     const float4 b = *reinterpret_cast<const float4 *>(sc + 12 + 4 * my_t);
     const float e = v - val[0];
-    const float e0 = __shfl_sync(0xffffffffu, e, lane & ~3), e1 = __shfl_sync(0xffffffffu, e, lane & ~3 | 1), e2 = __shfl_sync(0xffffffffu, e, lane & ~3 | 2),
-                e3 = __shfl_sync(0xffffffffu, e, lane | 3);
+    const float e0 = __shfl_sync(0xffffffffu, e, first), e1 = __shfl_sync(0xffffffffu, e, first + 2), e2 = __shfl_sync(0xffffffffu, e, first + 4),
+                e3 = __shfl_sync(0xffffffffu, e, first + 6);
     const float u0 = be.x * e0, u1 = be.y * fmaf(-a0.x, u0, e1), u2 = be.z * fmaf(-a0.z, u1, fmaf(-a0.y, u0, e2)),
                 u3 = be.w * fmaf(-a1.y, u2, fmaf(-a1.x, u1, fmaf(-a0.w, u0, e3)));
-    su[warp][lane >> 2][my_t] = my_t == 0 ? u0 : my_t == 1 ? u1 : my_t == 2 ? u2 : u3;
+    if ((lane & 7) == 0) *reinterpret_cast<float4 *>(su[warp][lane >> 3]) = make_float4(u0, u1, u2, u3);
     __syncwarp();
-    if (my_col < V && blk * DB_T + my_t < rows)
-      out[(size_t)(blk * DB_T + my_t) * inner + my_off] = fmaf(b.w, u3, fmaf(b.z, u2, fmaf(b.y, u1, fmaf(b.x, u0, val[1]))));
+    if (is_q && my_col < V && blk * DB_T + my_t < rows)
+      out[(size_t)(blk * DB_T + my_t) * inner + my_off] = fmaf(b.w, u3, fmaf(b.z, u2, fmaf(b.y, u1, fmaf(b.x, u0, val[0]))));
     {
       f32x2 g[2 * R4];
 #pragma unroll
@@ -673,7 +679,7 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaShape
         for (int i = 0; i < 2 * R4; i++) s[c][i] = x2_fma(x[i], uu, s[c][i]);
       }
     }
-    __syncwarp();  // su is rewritten by the next block
+    // (su is rewritten behind the next block's barrier)
   }
 #pragma unroll
   for (int c = 0; c < C; c++)
@@ -700,7 +706,7 @@ dp_status launch_step(dp_ctx *ctx, const float *proj, int proj_stride, const Del
 
 template <int NV>
 dp_status launch_scan(dp_ctx *ctx, const DeltaShape &sh, const SsmState &st, const DeltaRows &r, float *out, int rows, const RowMap &map) {
-  constexpr int NP = 32 * NV, LN = NP == 32 ? 8 : NP <= 128 ? 16 : 32;
+  constexpr int NP = 32 * NV, LN = NP >= 128 ? 32 : NP / 4;
   const size_t smem = (size_t)DS_STAGES * db_record(NP) * 4;
   static dp_per_device_once attr;
   if (attr.pending(ctx->device)) {

@@ -146,7 +146,6 @@ constexpr int LV_ROWS = 32;
 __global__ void __launch_bounds__(256) latent_values_step_kernel(const float *__restrict__ part, int splits, const LatentShape sh, const __nv_bfloat16 *__restrict__ wuv,
                                                                  int wuv_stride, const float *__restrict__ gate, float *__restrict__ out) {
   extern __shared__ __align__(16) float lv_ctx[];  // [wuv_stride]
-  __shared__ float s_w[32];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, v0 = blockIdx.y * LV_ROWS;
   const int pieces = wuv_stride / 8, CP = sh.c_pad(), row = CP + 2;
   constexpr int PER = LV_ROWS / 8, PRE = 2;  // rows per warp, pieces asked for before the wait
@@ -162,28 +161,30 @@ __global__ void __launch_bounds__(256) latent_values_step_kernel(const float *__
   pdl_launch();
   const float *pp = part + (size_t)h * splits * (splits > 1 ? row : CP);
   if (splits > 1) {
-    if (warp == 0) {
-      const float m = lane < splits ? pp[(size_t)lane * row + CP] : -FLT_MAX, l = lane < splits ? pp[(size_t)lane * row + CP + 1] : 0.0f;
-      float mm = m;
+    // every warp works out what each split counts for, a lane per split
+    const float m = lane < splits ? pp[(size_t)lane * row + CP] : -FLT_MAX, l = lane < splits ? pp[(size_t)lane * row + CP + 1] : 0.0f;
+    float mm = m;
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, o));
-      const float c = m == -FLT_MAX ? 0.0f : exp2f(m - mm);
-      float ll = l * c;
+    for (int o = 16; o > 0; o >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, o));
+    const float c = m == -FLT_MAX ? 0.0f : exp2f(m - mm);
+    float ll = l * c;
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) ll += __shfl_xor_sync(0xffffffffu, ll, o);
-      s_w[lane] = ll > 0.0f ? c / ll : 0.0f;
+    for (int o = 16; o > 0; o >>= 1) ll += __shfl_xor_sync(0xffffffffu, ll, o);
+    const float wt = ll > 0.0f ? c / ll : 0.0f;
+    for (int c0 = 0; c0 < CP; c0 += 512) {  // two columns per thread, c_pad is a multiple of sixteen
+      const int k = c0 + 2 * tid;
+      float2 acc = make_float2(0.0f, 0.0f);
+#pragma unroll 16
+      for (int s = 0; s < splits; s++) {
+        const float f = __shfl_sync(0xffffffffu, wt, s);
+        const float2 x = k < CP ? *reinterpret_cast<const float2 *>(pp + (size_t)s * row + k) : make_float2(0.0f, 0.0f);
+        acc.x = fmaf(x.x, f, acc.x);
+        acc.y = fmaf(x.y, f, acc.y);
+      }
+      if (k < wuv_stride) *reinterpret_cast<float2 *>(lv_ctx + k) = acc;
     }
-    __syncthreads();
-  }
-  for (int c = tid; c < wuv_stride; c += 256) {
-    float v = 0.0f;
-    if (c < sh.kv_rank) {
-      if (splits > 1) {
-#pragma unroll 8
-        for (int s = 0; s < splits; s++) v = fmaf(pp[(size_t)s * row + c], s_w[s], v);
-      } else v = pp[c];
-    }
-    lv_ctx[c] = v;
+  } else {
+    for (int c = tid; c < wuv_stride; c += 256) lv_ctx[c] = pp[c];
   }
   __syncthreads();
   const float g = gate ? lt_sigmoid(gate[h]) : 1.0f;

@@ -424,6 +424,47 @@ __global__ void __launch_bounds__(256) group_norm_warp_kernel(const float *__res
   }
 }
 
+// short parts (at most 128 values): a warp takes four of them, so that enough loads are under way
+template <typename OutT>
+__global__ void __launch_bounds__(256) group_norm_short_kernel(const float *__restrict__ x, int x_stride, const GroupNorm n, int gs, OutT *__restrict__ dst,
+                                                               int dst_stride, int rows) {
+  pdl_launch();
+  pdl_wait();
+  constexpr int PARTS = 4;
+  const int lane = threadIdx.x & 31, part0 = (blockIdx.x * 8 + (threadIdx.x >> 5)) * PARTS, c = lane * 4;
+  FV<4> v[PARTS], gate[PARTS];
+  int row[PARTS], at[PARTS];
+#pragma unroll
+  for (int i = 0; i < PARTS; i++) {
+    const int part = part0 + i;
+    row[i] = part / n.groups;
+    at[i] = (part - row[i] * n.groups) * gs + c;
+    const bool ok = part < rows * n.groups && c < gs;
+    if (!ok) row[i] = -1;
+    v[i] = ok ? ldv<4>(x + (size_t)row[i] * x_stride + at[i]) : FV<4>{};
+    gate[i] = ok && n.gate ? ldv<4>(n.gate + (size_t)row[i] * n.gate_stride + at[i]) : FV<4>{};
+  }
+  float ss[PARTS];
+#pragma unroll
+  for (int i = 0; i < PARTS; i++) ss[i] = fmaf(v[i].v[0], v[i].v[0], fmaf(v[i].v[1], v[i].v[1], fmaf(v[i].v[2], v[i].v[2], v[i].v[3] * v[i].v[3])));
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+    for (int i = 0; i < PARTS; i++) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+#pragma unroll
+  for (int i = 0; i < PARTS; i++) {
+    if (row[i] < 0) continue;
+    const float inv = 1.0f / sqrtf(ss[i] / (float)gs + n.eps);
+    const FV<4> w = ldw<4>(n.w + (n.w_shared ? c : at[i]));
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+      v[i].v[j] = v[i].v[j] * inv * w.v[j];
+      if (n.gate) v[i].v[j] *= 1.0f / (1.0f + expf(-gate[i].v[j]));
+    }
+    stv<4>(dst + (size_t)row[i] * dst_stride + at[i], v[i]);
+  }
+}
+
 template <int V, typename OutT>
 __global__ void __launch_bounds__(256) group_norm_kernel(const float *__restrict__ x, int x_stride, const GroupNorm n, int gs, OutT *__restrict__ dst,
                                                          int dst_stride) {
@@ -531,6 +572,12 @@ dp_status dpk_group_norm(dp_ctx *ctx, const float *x, int x_stride, const GroupN
   const int gs = width / n.groups;
   const bool aligned = ((uintptr_t)x & 15) == 0 && (!n.gate || (((uintptr_t)n.gate & 15) == 0 && n.gate_stride % 4 == 0));
   const bool vec = gs % 4 == 0 && x_stride % 4 == 0 && dst_stride % 4 == 0 && aligned;
+  if (vec && gs <= 128) {
+    const unsigned blocks = (unsigned)(((size_t)rows * n.groups + 31) / 32);
+    if (dst_bf16) DP_LAUNCH(ctx, group_norm_short_kernel<__nv_bfloat16>, blocks, 256, 0, x, x_stride, n, gs, (__nv_bfloat16 *)dst, dst_stride, rows);
+    else DP_LAUNCH(ctx, group_norm_short_kernel<float>, blocks, 256, 0, x, x_stride, n, gs, (float *)dst, dst_stride, rows);
+    return DP_OK;
+  }
   if (vec && gs <= 1024) {
     const unsigned blocks = (unsigned)(((size_t)rows * n.groups + 7) / 8);
     if (dst_bf16) DP_LAUNCH(ctx, (group_norm_warp_kernel<8, __nv_bfloat16>), blocks, 256, 0, x, x_stride, n, gs, (__nv_bfloat16 *)dst, dst_stride, rows);

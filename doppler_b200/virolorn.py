@@ -66,6 +66,8 @@ def layer_config(entries: List[dict], index: int, shape: Callable[[str], Optiona
     """Entry ``index`` of config 'layers' -> the fields of dp_layer_cfg.  ``shape(name)``: a tensor's shape."""
     where, entry = f"layer {index}", entries[index]
     owner = _owner(entries, index)
+    if owner != index and {k: v for k, v in entry.items() if k != "weights_of"} != {k: v for k, v in entries[owner].items() if k != "weights_of"}:
+        raise ConfigError(f"{where}: uses the weights of layer {owner} but differs from it")
     kind, m = st.need(entry, where, "type", "mixer")
     if kind not in MIXERS:
         raise ConfigError(f"{where}: unknown type '{kind}'")
@@ -86,8 +88,6 @@ def layer_config(entries: List[dict], index: int, shape: Callable[[str], Optiona
         _positive(where + " mlp", ff=ff)
         out.update(ff=ff, ff_limit=0.0, ff_slope=1.0, ff_shift=0.0)
     if owner != index:
-        if {k: v for k, v in entry.items() if k != "weights_of"} != {k: v for k, v in entries[owner].items() if k != "weights_of"}:
-            raise ConfigError(f"{where}: uses the weights of layer {owner} but differs from it")
         out["share"] = owner + 1
     return out
 
