@@ -114,21 +114,20 @@ __device__ __forceinline__ float dl_conv(const float *proj, int proj_stride, con
 // What earlier steps left (state, convolution histories, positions) and the matrices of decay and gate are read before
 // griddepcontrol.wait; after it only this token's projections are.
 struct DeltaStepSmem {  // offsets in floats; the weight tiles behind them in bytes
-  int q, k, v, g, low, red, weights;
+  int q, k, v, g, low, weights;
   int w_rows_a, w_rows_g, pitch_a, pitch_g;  // staged rows (0: read from global memory), bytes per staged row
   int total;
 };
 
-__host__ __device__ inline DeltaStepSmem delta_step_smem(const DeltaShape &sh, int a2_stride, int g2_stride, int limit) {
+__host__ __device__ inline DeltaStepSmem delta_step_smem(const DeltaShape &sh, int a2_stride, int g2_stride, int limit, bool staged) {
   DeltaStepSmem m;
   const int NP = sh.state_stride;
   m.q = 0; m.k = NP; m.g = 2 * NP; m.v = 3 * NP; m.low = m.v + DL_COLS;
-  m.red = m.low + a2_stride + g2_stride;
-  m.weights = (m.red + 16 + 3) / 4 * 4;
+  m.weights = m.low + a2_stride + g2_stride;  // (a multiple of four)
   m.pitch_a = a2_stride * 2 + 16; m.pitch_g = g2_stride * 2 + 16;
   m.w_rows_a = sh.dim; m.w_rows_g = DL_COLS;
   m.total = m.weights * 4 + m.w_rows_a * m.pitch_a + m.w_rows_g * m.pitch_g;
-  if (m.total > limit) { m.w_rows_a = m.w_rows_g = 0; m.total = m.weights * 4; }
+  if (!staged || m.total > limit) { m.w_rows_a = m.w_rows_g = 0; m.total = m.weights * 4; }
   return m;
 }
 
@@ -146,14 +145,44 @@ __device__ __forceinline__ float dl_dot_row(const __nv_bfloat16 *w, const float 
   return acc;
 }
 
-template <int NV>
+// product of one 16-byte piece of a row with eight values
+__device__ __forceinline__ float dl_piece(const uint4 &r, const float (&x)[8]) {
+  float acc = __uint_as_float(r.x << 16) * x[0];
+  acc = fmaf(__uint_as_float(r.x & 0xffff0000u), x[1], acc);
+  acc = fmaf(__uint_as_float(r.y << 16), x[2], acc); acc = fmaf(__uint_as_float(r.y & 0xffff0000u), x[3], acc);
+  acc = fmaf(__uint_as_float(r.z << 16), x[4], acc); acc = fmaf(__uint_as_float(r.z & 0xffff0000u), x[5], acc);
+  acc = fmaf(__uint_as_float(r.w << 16), x[6], acc); acc = fmaf(__uint_as_float(r.w & 0xffff0000u), x[7], acc);
+  return acc;
+}
+// sums over sixteen lanes of N values each (N a power of two up to sixteen): the lane ends up with the sum of value (lane & 15) / (16 / N)
+template <int N> __device__ __forceinline__ float dl_sum_scatter16(float (&v)[N], int lane) {
+  int n = N;
+#pragma unroll
+  for (int o = 8; o > 0; o >>= 1) {
+    if (n > 1) {
+      n >>= 1;
+      const bool upper = lane & o;
+#pragma unroll
+      for (int i = 0; i < (N > 1 ? N / 2 : 1); i++)
+        if (i < n) {
+          const float send = upper ? v[i] : v[i + n], keep = upper ? v[i + n] : v[i];
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+    }
+  }
+  return v[0];
+}
+
+// SMALL: low-rank sizes up to 128.  The matrices' rows are then fetched straight into registers, sixteen lanes to a row.
+template <int NV, bool SMALL>
 __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(const float *__restrict__ proj, int proj_stride, const DeltaShape sh, const DeltaWeights w,
                                                                 const SsmState st, float *__restrict__ out, float *__restrict__ gate,
                                                                 const int *__restrict__ pos_arr, const DeltaStepSmem m) {
   constexpr int NP = NV * 32, CHANNELS = 2 * NP + DL_COLS, PER = (CHANNELS + DL_THREADS - 1) / DL_THREADS;
   extern __shared__ __align__(16) float dl_smem[];
   float *sq = dl_smem + m.q, *sk = dl_smem + m.k, *sv = dl_smem + m.v, *sg = dl_smem + m.g, *low_a = dl_smem + m.low, *low_g = low_a + w.a2_stride;
-  float *red = dl_smem + m.red;
   unsigned char *s_wa = reinterpret_cast<unsigned char *>(dl_smem + m.weights), *s_wg = s_wa + m.w_rows_a * m.pitch_a;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.x, p0 = blockIdx.y * DL_COLS, row = blockIdx.z;
   const int D = sh.dim, V = sh.vdim, per = sh.heads / sh.kv_heads, kvh = h / per, CH = sh.channels(), taps = sh.taps, QK = sh.qk(), inner = sh.inner();
@@ -166,7 +195,21 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(const float *__r
   // rows of the decay's and the gate's second matrix
   const __nv_bfloat16 *wa = w.a2 + (size_t)h * D * w.a2_stride, *wg = w.g2 + ((size_t)h * V + p0) * w.g2_stride;
   const int pa = w.a2_stride / 8, pg = w.g2_stride / 8;
-  if (m.w_rows_a) {
+  constexpr int IT = SMALL ? NP / 16 : 1, GT = 2;  // rows per half-warp: key channels, value columns
+  const int half = lane >> 4, piece = lane & 15;
+  uint4 ra[IT], rg[GT];
+  if constexpr (SMALL) {
+#pragma unroll
+    for (int i = 0; i < IT; i++) {
+      const int c = warp * (NP / 8) + 2 * i + half;
+      ra[i] = c < D && piece < pa ? __ldg(reinterpret_cast<const uint4 *>(wa + (size_t)c * w.a2_stride) + piece) : make_uint4(0, 0, 0, 0);
+    }
+#pragma unroll
+    for (int i = 0; i < GT; i++) {
+      const int c = warp * 4 + 2 * i + half;
+      rg[i] = c < cols && piece < pg ? __ldg(reinterpret_cast<const uint4 *>(wg + (size_t)c * w.g2_stride) + piece) : make_uint4(0, 0, 0, 0);
+    }
+  } else if (m.w_rows_a) {
     for (int i = tid; i < D * pa; i += DL_THREADS)
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(s_wa + (i / pa) * m.pitch_a + (i % pa) * 16)), "l"(wa + 8 * (size_t)i) : "memory");
     for (int i = tid; i < cols * pg; i += DL_THREADS)
@@ -199,56 +242,86 @@ __global__ void __launch_bounds__(DL_THREADS) delta_step_kernel(const float *__r
         if (pos - k >= 0) acc[j] = fmaf(cw[taps - 1 - k], hist[(size_t)((pos - k) % taps) * CH + ch], acc[j]);
     }
   }
+  // the decay this lane will finish (SMALL): its constants
+  const int my_c = warp * (NP / 8) + 2 * (piece / (16 / IT)) + half;
+  const float rate = SMALL && my_c < D ? w.rate[h * D + my_c] : 0.0f, bias = SMALL && my_c < D ? w.bias[h * D + my_c] : 0.0f;
   const bool keep_qk = blockIdx.y == 0 && h == kvh * per;  // one head of the group appends its q and k
   pdl_wait();
   pdl_launch();
   const float beta = dl_sigmoid(pr[sh.beta_col() + h]);
-  for (int i = tid; i < w.a2_stride; i += DL_THREADS) low_a[i] = i < sh.decay_rank ? pr[sh.a1_col() + i] : 0.0f;
-  for (int i = tid; i < w.g2_stride; i += DL_THREADS) low_g[i] = i < sh.gate_rank ? pr[sh.g1_col() + i] : 0.0f;
+  float xa[8], xg[8], cur[PER];
+  if constexpr (SMALL) {
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+      const int i = piece * 8 + j;
+      xa[j] = i < sh.decay_rank ? pr[sh.a1_col() + i] : 0.0f;
+      xg[j] = i < sh.gate_rank ? pr[sh.g1_col() + i] : 0.0f;
+    }
+  } else {
+    for (int i = tid; i < w.a2_stride; i += DL_THREADS) low_a[i] = i < sh.decay_rank ? pr[sh.a1_col() + i] : 0.0f;
+    for (int i = tid; i < w.g2_stride; i += DL_THREADS) low_g[i] = i < sh.gate_rank ? pr[sh.g1_col() + i] : 0.0f;
+  }
+#pragma unroll
+  for (int j = 0; j < PER; j++) cur[j] = chan[j] >= 0 ? pr[chan[j]] : 0.0f;
 #pragma unroll
   for (int j = 0; j < PER; j++) {
     const int i = tid + j * DL_THREADS;
     if (i < CHANNELS) {
       float val = 0.0f;
       if (chan[j] >= 0) {
-        const float cur = pr[chan[j]];
-        val = dl_silu(fmaf(last[j], cur, acc[j]));
-        if (taps > 1 && (i >= 2 * NP || keep_qk)) slot[chan[j]] = cur;
+        val = dl_silu(fmaf(last[j], cur[j], acc[j]));
+        if (taps > 1 && (i >= 2 * NP || keep_qk)) slot[chan[j]] = cur[j];
       }
       if (i < NP) sq[i] = val;
       else if (i < 2 * NP) sk[i - NP] = val;
       else sv[i - 2 * NP] = val;
     }
   }
-  if (m.w_rows_a) asm volatile("cp.async.wait_group 0;" ::: "memory");
-  __syncthreads();
-  // two threads per key channel: its decay
-  for (int c0 = 0; c0 < NP; c0 += DL_THREADS / 2) {
-    const int c = c0 + (tid >> 1);
-    float d = 0.0f;
-    if (c < D) d = dl_dot_row(m.w_rows_a ? reinterpret_cast<const __nv_bfloat16 *>(s_wa + c * m.pitch_a) : wa + (size_t)c * w.a2_stride, low_a, pa, tid & 1, 2);
-    d += __shfl_xor_sync(0xffffffffu, d, 1);
-    if (c < NP && (tid & 1) == 0) sg[c] = c < D ? expf(-w.rate[h * D + c] * dl_softplus(d + w.bias[h * D + c])) : 0.0f;
-  }
-  // eight threads per value column: the output gate
-  {
+  if constexpr (SMALL) {
+    float va[IT], vg[GT];
+#pragma unroll
+    for (int i = 0; i < IT; i++) va[i] = dl_piece(ra[i], xa);
+#pragma unroll
+    for (int i = 0; i < GT; i++) vg[i] = dl_piece(rg[i], xg);
+    const float a = dl_sum_scatter16<IT>(va, lane), g = dl_sum_scatter16<GT>(vg, lane);
+    if (piece % (16 / IT) == 0) sg[my_c] = my_c < D ? expf(-rate * dl_softplus(a + bias)) : 0.0f;
+    const int gc = warp * 4 + 2 * (piece / (16 / GT)) + half;
+    if (piece % (16 / GT) == 0 && gc < cols) gate[(size_t)row * inner + h * V + p0 + gc] = g;
+    __syncthreads();
+  } else {
+    if (m.w_rows_a) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    // two threads per key channel: its decay
+    for (int c0 = 0; c0 < NP; c0 += DL_THREADS / 2) {
+      const int c = c0 + (tid >> 1);
+      float d = 0.0f;
+      if (c < D) d = dl_dot_row(m.w_rows_a ? reinterpret_cast<const __nv_bfloat16 *>(s_wa + c * m.pitch_a) : wa + (size_t)c * w.a2_stride, low_a, pa, tid & 1, 2);
+      d += __shfl_xor_sync(0xffffffffu, d, 1);
+      if (c < NP && (tid & 1) == 0) sg[c] = c < D ? expf(-w.rate[h * D + c] * dl_softplus(d + w.bias[h * D + c])) : 0.0f;
+    }
+    // eight threads per value column: the output gate
     float d = 0.0f;
     if (col < cols) d = dl_dot_row(m.w_rows_a ? reinterpret_cast<const __nv_bfloat16 *>(s_wg + col * m.pitch_g) : wg + (size_t)col * w.g2_stride, low_g, pg, sub, DL_LANES);
 #pragma unroll
     for (int o = 4; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
     if (sub == 0 && col < cols) gate[(size_t)row * inner + h * V + p0 + col] = d;
+    __syncthreads();
   }
-  if (warp < 3) {  // q.q, k.k, q.k
-    const float *a = warp == 1 ? sk : sq, *b = warp == 0 ? sq : sk;
-    float d = 0.0f;
+  // q.q, k.k, q.k, by every warp for itself
+  float qq = 0.0f, kk = 0.0f, qk = 0.0f;
 #pragma unroll
-    for (int i = 0; i < NV; i++) d = fmaf(a[lane + 32 * i], b[lane + 32 * i], d);
-    d = dl_warp_sum(d);
-    if (lane == 0) red[warp] = d;
+  for (int i = 0; i < NV; i++) {
+    const float a = sq[lane + 32 * i], b = sk[lane + 32 * i];
+    qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); qk = fmaf(a, b, qk);
   }
-  __syncthreads();
-  const float q_scale = 1.0f / sqrtf(red[0] + 1e-6f) / sqrtf((float)D), k_scale = 1.0f / sqrtf(red[1] + 1e-6f);
-  const float o = dl_token<NV>(s, sk, sq, sg, sub, sv[col], beta, red[2], k_scale, q_scale);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    qq += __shfl_xor_sync(0xffffffffu, qq, o);
+    kk += __shfl_xor_sync(0xffffffffu, kk, o);
+    qk += __shfl_xor_sync(0xffffffffu, qk, o);
+  }
+  const float q_scale = 1.0f / sqrtf(qq + 1e-6f) / sqrtf((float)D), k_scale = 1.0f / sqrtf(kk + 1e-6f);
+  const float o = dl_token<NV>(s, sk, sq, sg, sub, sv[col], beta, qk, k_scale, q_scale);
   if (col < cols) {
 #pragma unroll
     for (int i = 0; i < NV; i++) x2_store4(S + 32 * i, s[2 * i], s[2 * i + 1]);
@@ -720,15 +793,21 @@ template <int NV>
 dp_status launch_step(dp_ctx *ctx, const float *proj, int proj_stride, const DeltaShape &sh, const DeltaWeights &w, const SsmState &st, float *out, float *gate,
                       int rows, const int *pos) {
   const int limit = 100 * 1024;  // two CTAs per SM
+  const dim3 grid(sh.heads, (sh.vdim + DL_COLS - 1) / DL_COLS, rows);
+  if constexpr (NV <= 4)
+    if (w.a2_stride <= 128 && w.g2_stride <= 128) {
+      const DeltaStepSmem m = delta_step_smem(sh, w.a2_stride, w.g2_stride, limit, false);
+      DP_LAUNCH(ctx, (delta_step_kernel<NV, true>), grid, DL_THREADS, (size_t)m.total, proj, proj_stride, sh, w, st, out, gate, pos, m);
+      return DP_OK;
+    }
   static dp_per_device_once attr;
   if (attr.pending(ctx->device)) {
-    DP_CUDA(ctx, cudaFuncSetAttribute(delta_step_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, limit));
+    DP_CUDA(ctx, cudaFuncSetAttribute((delta_step_kernel<NV, false>), cudaFuncAttributeMaxDynamicSharedMemorySize, limit));
     attr.done(ctx->device);
   }
-  const DeltaStepSmem m = delta_step_smem(sh, w.a2_stride, w.g2_stride, limit);
+  const DeltaStepSmem m = delta_step_smem(sh, w.a2_stride, w.g2_stride, limit, true);
   if (m.total > limit) return dp_fail(ctx, DP_ERR_UNSUPPORTED, "delta: low-rank sizes %d and %d exceed shared memory", sh.decay_rank, sh.gate_rank);
-  DP_LAUNCH(ctx, delta_step_kernel<NV>, dim3(sh.heads, (sh.vdim + DL_COLS - 1) / DL_COLS, rows), DL_THREADS, (size_t)m.total, proj, proj_stride, sh, w, st, out, gate,
-            pos, m);
+  DP_LAUNCH(ctx, (delta_step_kernel<NV, false>), grid, DL_THREADS, (size_t)m.total, proj, proj_stride, sh, w, st, out, gate, pos, m);
   return DP_OK;
 }
 

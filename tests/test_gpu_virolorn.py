@@ -29,6 +29,8 @@ CASES = {
     "delta odd sizes": config([delta(heads=6, kv_heads=3, dim=5, vdim=11, conv=3, ranks=(17, 5))], width=51),
     "delta wide keys": config([delta(heads=2, kv_heads=1, dim=200, vdim=40)]),
     "delta wider keys": config([delta(heads=2, kv_heads=2, dim=260, vdim=9)]),
+    "delta wide low ranks": config([delta(ranks=(150, 3)), delta(dim=40, ranks=(5, 200))]),
+    "delta wider low ranks": config([delta(heads=2, kv_heads=2, dim=256, vdim=9, ranks=(300, 140))]),
     "delta with feed-forward": config([delta(mlp=FF)]),
     "latent": config([latent()]),
     "latent one head": config([latent(heads=1, dim=6, rot_dim=2, vdim=5, kv_rank=9, q_rank=3)]),
