@@ -404,9 +404,11 @@ __global__ void __launch_bounds__(128) delta_rows_kernel(const float *__restrict
 }
 
 // Up to four taps, sizes and strides that are multiples of four: a lane owns four neighbouring channels (times JV), the
-// rows a token reaches back to stay in registers, and four rows are fetched at a time.
-template <int TAPS>
+// rows a token reaches back to stay in registers, and four rows are fetched at a time.  FAST: the approximate exponential and
+// quotient (the bf16 mode, in which these activations need no more than sixteen bits).
+template <int TAPS, bool FAST>
 struct ConvWindow {
+  static __device__ __forceinline__ float silu(float v) { return FAST ? __fdividef(v, 1.0f + __expf(-v)) : dl_silu(v); }
   float w[4][TAPS];
   float4 win[TAPS];  // the last TAPS rows, newest at the end
   __device__ __forceinline__ void init(const float *conv, const float *proj, int proj_stride, const float *hist, int CH, int ch, int r0, int start_pos) {
@@ -432,11 +434,11 @@ struct ConvWindow {
       o.x = fmaf(w[0][k], win[k].x, o.x); o.y = fmaf(w[1][k], win[k].y, o.y);
       o.z = fmaf(w[2][k], win[k].z, o.z); o.w = fmaf(w[3][k], win[k].w, o.w);
     }
-    return make_float4(dl_silu(o.x), dl_silu(o.y), dl_silu(o.z), dl_silu(o.w));
+    return make_float4(silu(o.x), silu(o.y), silu(o.z), silu(o.w));
   }
 };
 
-template <int JV, int TAPS>
+template <int JV, int TAPS, bool FAST>
 __global__ void __launch_bounds__(128) delta_rows4_kernel(const float *__restrict__ proj, int proj_stride, const DeltaShape sh, const DeltaWeights w, const SsmState st,
                                                           const DeltaRows out, int v_units, int rows, int start_pos, int seq) {
   pdl_launch();
@@ -451,7 +453,7 @@ __global__ void __launch_bounds__(128) delta_rows4_kernel(const float *__restric
   };
   if (unit < G) {
     const float q_mul = 1.0f / sqrtf((float)D);
-    ConvWindow<TAPS> cq[JV], ck[JV];
+    ConvWindow<TAPS, FAST> cq[JV], ck[JV];
 #pragma unroll
     for (int j = 0; j < JV; j++) {
       const int d = 4 * lane + 128 * j;
@@ -510,7 +512,7 @@ __global__ void __launch_bounds__(128) delta_rows4_kernel(const float *__restric
   } else if (unit < G + v_units) {
     const int e = (unit - G) * 128 + 4 * lane;
     if (e >= inner) return;
-    ConvWindow<TAPS> cv;
+    ConvWindow<TAPS, FAST> cv;
     cv.init(w.conv, proj, proj_stride, hist, CH, 2 * QK + e, r0, start_pos);
     for (int rb = r0; rb < r1; rb += BATCH) {
       float4 x[BATCH];
@@ -831,7 +833,10 @@ dp_status launch_rows4(dp_ctx *ctx, const float *proj, int proj_stride, const De
                        const RowMap &map) {
   const int v_units = (sh.inner() + 127) / 128, units = sh.kv_heads + v_units + DR_AUX;
   const dim3 grid((units + 3) / 4, (rows + DR_ROWS - 1) / DR_ROWS);
-#define DP_ROWS4(T) DP_LAUNCH(ctx, (delta_rows4_kernel<JV, T>), grid, 128, 0, proj, proj_stride, sh, w, st, r, v_units, rows, map.start_pos, map.seq)
+#define DP_ROWS4(T) do { \
+    if (r.a_low) DP_LAUNCH(ctx, (delta_rows4_kernel<JV, T, true>), grid, 128, 0, proj, proj_stride, sh, w, st, r, v_units, rows, map.start_pos, map.seq); \
+    else DP_LAUNCH(ctx, (delta_rows4_kernel<JV, T, false>), grid, 128, 0, proj, proj_stride, sh, w, st, r, v_units, rows, map.start_pos, map.seq); \
+  } while (0)
   switch (sh.taps) {
     case 1: DP_ROWS4(1); break;
     case 2: DP_ROWS4(2); break;
