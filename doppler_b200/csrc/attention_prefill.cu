@@ -50,14 +50,15 @@ __device__ __forceinline__ uint32_t apf_pack(float a, float b) {
 }
 
 // grid: (query tiles, KV heads, batch); G = num_heads / num_kv_heads in {1, 2, 4, 8}
-template <int DK, int DV>
+// EXACT: one-part keys and values of just these sizes, heads side by side
+template <int DK, int DV, bool EXACT>
 __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_attn_params p, int G) {
   pdl_launch();
   pdl_wait();
   using L = ApfLayout<DK, DV>;
   constexpr int KS = DK / 16, NV = DV / 8;
-  const int D = p.head_dim, V = p.v_dim ? p.v_dim : D;  // sizes of a query and of a value; keys: k_dim + k2_dim
-  const int kd = p.k2 ? p.k_dim : D, k_pieces = (kd + 7) / 8, k2_pieces = p.k2 ? (p.k2_dim + 7) / 8 : 0, v_pieces = (V + 7) / 8;
+  const int D = EXACT ? DK : p.head_dim, V = EXACT ? DV : (p.v_dim ? p.v_dim : D);  // sizes of a query and of a value; keys: k_dim + k2_dim
+  const int kd = !EXACT && p.k2 ? p.k_dim : D, k_pieces = (kd + 7) / 8, k2_pieces = !EXACT && p.k2 ? (p.k2_dim + 7) / 8 : 0, v_pieces = (V + 7) / 8;
   extern __shared__ __align__(128) unsigned char apf_smem[];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g = lane >> 2, t = lane & 3;
@@ -87,7 +88,7 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
   const __half *vbase = p.v + (size_t)b * (p.v_batch_stride ? p.v_batch_stride : p.kv_batch_stride) + (size_t)kvh * v_pieces * 8;
   const __half *k2base = p.k2 + (size_t)b * p.k2_batch_stride;
   // elements between consecutive keys
-  const size_t key_stride = p.k_row_stride ? (size_t)p.k_row_stride : (size_t)p.num_kv_heads * D, val_stride = p.v_row_stride ? (size_t)p.v_row_stride : (size_t)p.num_kv_heads * V;
+  const size_t key_stride = !EXACT && p.k_row_stride ? (size_t)p.k_row_stride : (size_t)p.num_kv_heads * D, val_stride = !EXACT && p.v_row_stride ? (size_t)p.v_row_stride : (size_t)p.num_kv_heads * V;
   const uint32_t smem0 = (uint32_t)__cvta_generic_to_shared(apf_smem);
 
   auto issue_tile = [&](int tile) {
@@ -128,6 +129,7 @@ __global__ void __launch_bounds__(APF_THREADS, 1) attn_prefill_tc_kernel(dpk_att
     auto pair = [&](const float *q, bool ok, int d) {
       float2 v = make_float2(0.0f, 0.0f);
       if (!ok) return v;
+      if (EXACT) return *reinterpret_cast<const float2 *>(q + d);
       const int at = d < k_pieces * 8 ? d : kd + (d - k_pieces * 8), end = d < k_pieces * 8 ? kd : D;
       if (at + 1 < end && (((D | at) & 1) == 0)) return *reinterpret_cast<const float2 *>(q + at);
       if (at < end) v.x = q[at];
@@ -283,24 +285,25 @@ bool dpk_attention_prefill_eligible(const dpk_attn_params &p) {
   return true;
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool EXACT>
 static dp_status launch_prefill(dp_ctx *ctx, const dpk_attn_params &p, int G) {
   const int QT = 16 * APF_WARPS / G;
   const size_t smem = 2 * ApfLayout<DK, DV>::STAGE;
   static dp_per_device_once attr;
   if (attr.pending(ctx->device)) {
-    DP_CUDA(ctx, cudaFuncSetAttribute((attn_prefill_tc_kernel<DK, DV>), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    DP_CUDA(ctx, cudaFuncSetAttribute((attn_prefill_tc_kernel<DK, DV, EXACT>), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     attr.done(ctx->device);
   }
   dim3 grid((p.seq_len + QT - 1) / QT, p.num_kv_heads, p.batch);
-  DP_LAUNCH(ctx, (attn_prefill_tc_kernel<DK, DV>), grid, APF_THREADS, smem, p, G);
+  DP_LAUNCH(ctx, (attn_prefill_tc_kernel<DK, DV, EXACT>), grid, APF_THREADS, smem, p, G);
   return DP_OK;
 }
 
 dp_status dpk_attention_prefill(dp_ctx *ctx, const dpk_attn_params &p) {
   const int G = p.num_heads / p.num_kv_heads;
   const int dk = p.k2 ? (p.k_dim + 7) / 8 * 8 + (p.k2_dim + 7) / 8 * 8 : p.head_dim, dv = p.v_dim ? p.v_dim : p.head_dim;
-  if (dk <= 64 && dv <= 64) return launch_prefill<64, 64>(ctx, p, G);
-  if (dk <= 128) return launch_prefill<128, 128>(ctx, p, G);
-  return launch_prefill<192, 128>(ctx, p, G);
+  if (!p.k2) return launch_prefill<128, 128, true>(ctx, p, G);
+  if (dk <= 64 && dv <= 64) return launch_prefill<64, 64, false>(ctx, p, G);
+  if (dk <= 128) return launch_prefill<128, 128, false>(ctx, p, G);
+  return launch_prefill<192, 128, false>(ctx, p, G);
 }
